@@ -646,6 +646,130 @@ class TorchOps:
             out[b] = (p @ v).reshape(-1).to(q.dtype)
         return out
 
+    # ------------------------------------------------------------- latent attention, output norms, experts
+    # Rows may be padded on the right with zeros (``width`` is the true size).  The residual stream ``x`` is fp32 and
+    # updated in place; what the next product reads is returned in the activation dtype.
+    def flash_latent(self, dtype: torch.dtype) -> bool:
+        """Whether prompts may expand keys and values and use :meth:`attention_context` in this dtype."""
+        return True
+
+    def latent_multiple(self, dtype: torch.dtype) -> int:
+        """What the cached latent's size is padded to."""
+        return 8
+
+    def embed_pairs(self, ids, prev, table, bigram, consts):
+        """``x = table[id] (+ bigram[row])`` with ``row = (prev * mul_prev + id * mul_cur) mod buckets``, or row
+        ``buckets`` where ``prev < 0``; ``consts = (buckets, mul_prev, mul_cur)``.  Returns ``x`` fp32 and its rounding to the table's dtype."""
+        x = _f(table[ids]).clone()
+        if bigram is not None:
+            n, a, c = consts
+            row = torch.where(prev < 0, torch.full_like(ids, n), (prev.long() * a + ids * c) % n)
+            x = x + _f(bigram[row])
+        return x, x.to(table.dtype, copy=True)
+
+    def latent_append(self, rows, w, width, eps, pages, slots):
+        """RMS norm of ``rows[N, R]`` (mean over ``width``), written to cache slots ``slots`` of ``pages[P, 16, R]``
+        (negative: nowhere) and returned."""
+        r = _f(rows)
+        c = (r * torch.rsqrt(r.pow(2).sum(-1, keepdim=True) / width + eps) * w).to(pages.dtype)
+        ok = slots >= 0
+        pages[slots[ok] // 16, slots[ok] % 16] = c[ok]
+        return c
+
+    def latent_gather(self, pages, page_table, cu_context, total):
+        """The cached latents of every sequence, packed: ``[total, R]``."""
+        cu = cu_context.tolist()
+        return torch.cat([pages[page_table[b, : (n + 15) // 16].long()].flatten(0, 1)[:n]
+                          for b, n in enumerate(j - i for i, j in zip(cu, cu[1:]))])
+
+    def latent_attention(self, q, pages, page_table, ctx_lens, cu_seqlens, max_q, max_ctx, scale):
+        """``q[N, H, R]`` against the cached latents, which serve as keys and values of every head.  Sequence ``b`` owns
+        rows ``cu_seqlens[b:b+2]`` (None: row ``b``), the last of its ``ctx_lens[b]`` tokens; causal."""
+        N, H, R = q.shape
+        out = torch.empty_like(q)
+        cu = cu_seqlens.tolist() if cu_seqlens is not None else list(range(N + 1))
+        for b, n in enumerate(ctx_lens.tolist()):
+            lo, hi = cu[b], cu[b + 1]
+            c = _f(pages[page_table[b, : (n + 15) // 16].long()].flatten(0, 1)[:n])
+            s = torch.einsum("nhr,tr->nht", _f(q[lo:hi]), c) * scale
+            seen = torch.arange(n, device=q.device)[None, :] <= torch.arange(n - (hi - lo), n, device=q.device)[:, None]
+            p = torch.softmax(s.masked_fill(~seen[:, None, :], float("-inf")), -1)
+            out[lo:hi] = torch.einsum("nht,tr->nhr", p, c).to(q.dtype)
+        return out
+
+    def attention_context(self, q, k, v, cu_seqlens, cu_context, max_q, scale):
+        """Causal attention of packed query rows ``q[Nq, H, d]`` against packed contexts ``k, v[Nk, H, d]``: the queries
+        of sequence ``b`` are the last of its ``cu_context[b+1] - cu_context[b]`` positions."""
+        out = torch.empty(q.shape[0], q.shape[1], v.shape[2], device=q.device, dtype=q.dtype)
+        cq, ck = cu_seqlens.tolist(), cu_context.tolist()
+        for b in range(len(cq) - 1):
+            qb, kb, vb = _f(q[cq[b]:cq[b + 1]]), _f(k[ck[b]:ck[b + 1]]), _f(v[ck[b]:ck[b + 1]])
+            n, t = qb.shape[0], kb.shape[0]
+            s = torch.einsum("nhd,thd->hnt", qb, kb) * scale
+            seen = torch.arange(t, device=q.device)[None, :] <= torch.arange(t - n, t, device=q.device)[:, None]
+            p = torch.softmax(s.masked_fill(~seen, float("-inf")), -1)
+            out[cq[b]:cq[b + 1]] = torch.einsum("hnt,thd->nhd", p, vb).to(q.dtype)
+        return out
+
+    def head_gemm(self, a, w, transposed: bool = False):
+        """One product per head: ``a[N, H, K]`` with ``w[H, M, K]`` (``transposed``: ``w[H, K, M]``) -> ``[N, H, M]``."""
+        return torch.einsum("nhk,hkm->nhm" if transposed else "nhk,hmk->nhm", a, w)
+
+    def activate(self, u, kind: str):
+        """``relu2``: squared ReLU; ``gelu``: the exact (erf) GELU."""
+        z = _f(u)
+        return (F.relu(z).square() if kind == "relu2" else F.gelu(z)).to(u.dtype)
+
+    def norm_add(self, x, y, g, width, eps):
+        """``x += rms(y) * g`` in place; returns ``x`` in ``y``'s dtype."""
+        z = _f(y)
+        x += z * torch.rsqrt(z.pow(2).sum(-1, keepdim=True) / width + eps) * g
+        return x.to(y.dtype, copy=True)
+
+    def norm_rows(self, x, rows, w, width, eps, dtype):
+        z = x[rows]
+        return (z * torch.rsqrt(z.pow(2).sum(-1, keepdim=True) / width + eps) * w).to(dtype)
+
+    def moe_route(self, h, router, experts, top, scale, groups, keep):
+        """Softmax router with group-limited top-k.  ``router[E (+ 1), D]``: an extra row is the shared expert's gate.
+        Returns expert ids ``[N, top]`` int32, weights ``[N, top]`` fp32 (score * scale) and the gate's sigmoid ``[N]`` or None."""
+        z = _f(h) @ _f(router).t()
+        s = torch.softmax(z[:, :experts], -1)
+        elig = s
+        if keep < groups:
+            best = s.view(-1, groups, experts // groups).amax(-1).topk(keep, -1).indices
+            ok = torch.zeros(s.shape[0], groups, dtype=torch.bool, device=s.device).scatter_(1, best, True)
+            elig = s.masked_fill(~ok.repeat_interleave(experts // groups, 1), -1.0)
+        w, ids = elig.topk(top, -1)
+        return ids.to(torch.int32), w * scale, torch.sigmoid(z[:, experts]) if router.shape[0] > experts else None
+
+    def moe_experts(self, h, ids, up, down, kind):
+        """Every token through its chosen experts (``up[E, ff, D]``, ``down[E, D, ff]``).  Returns the outputs as rows
+        grouped by expert, and ``at[N, top]``: the row of each (token, choice)."""
+        flat = ids.flatten().long()
+        order = torch.argsort(flat, stable=True)
+        at = torch.empty_like(order)
+        at[order] = torch.arange(order.numel(), device=order.device)
+        src = h[order // ids.shape[1]]
+        out = torch.empty(order.numel(), down.shape[1], device=h.device, dtype=h.dtype)
+        lo = 0
+        for e, n in enumerate(torch.bincount(flat, minlength=up.shape[0]).tolist()):
+            if n:
+                out[lo:lo + n] = self.activate(src[lo:lo + n] @ up[e].t(), kind) @ down[e].t()
+            lo += n
+        return out, at.view(ids.shape).to(torch.int32)
+
+    def moe_combine_norm_add(self, x, ye, at, wts, ys, gate, g, width, eps, dtype):
+        """``y = sum_k wts * ye[at] (+ gate * ys)``, then :meth:`norm_add`."""
+        y = (_f(ye)[at.long()] * wts.unsqueeze(-1)).sum(1)
+        if ys is not None:
+            y = y + gate.unsqueeze(-1) * _f(ys)
+        return self.norm_add(x, y, g, width, eps).to(dtype)
+
+    def softcap_(self, logits, cap: float):
+        """``cap * tanh(logits / cap)`` in place."""
+        return logits.div_(cap).tanh_().mul_(cap)
+
     def argmax(self, logits: torch.Tensor) -> torch.Tensor:
         return logits.float().argmax(-1)
 

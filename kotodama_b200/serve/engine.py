@@ -13,8 +13,12 @@ AttnRes needs no cross-token state at inference: the sources of a routing call a
 token's own block summaries, rebuilt layer by layer (``src/model/llama.py:718-763``), so only
 keys and values are cached.
 
-The layer pipeline is the executor's forward schedule (same ops backend: PyTorch on CPU,
-sm_100a kernels on CUDA); sampling follows the reference order repetition penalty ->
+The engine is the scheduler, the page accounting, the decode graphs and the sampling; the layer pipeline and
+the contents of the cache belong to the model family's runner (``serve/runners.py``, chosen by
+``models/registry.py``).  A family that can continue a cached sequence also takes prompts in portions
+(``prefill_portion``) and sequences whose tokens the caller supplies (``open`` / ``feed`` / ``close``): both
+go through the same two passes as generation, ``_extend`` (several tokens per request) and ``_decode_pass``
+(one token per request).  Sampling follows the reference order repetition penalty ->
 temperature -> top-k -> top-p -> multinomial, greedy at temperature 0 (``serve.py:266-304``).
 """
 from __future__ import annotations
@@ -26,12 +30,9 @@ from typing import Any, Optional
 import numpy as np
 import torch
 
-from ..config import ModelConfig
-from ..engine import ParamArena
-from ..models.llama import KotodamaModel
 from ..ops import get_ops
-
-PAGE = 16
+from .cache import PAGE, PagedKVCache, PagePool  # noqa: F401  (the engine module re-exports its cache)
+from .runners import Batch, make_runner
 
 
 @dataclass
@@ -56,35 +57,7 @@ class Request:
     finished: bool = False
     finish_reason: str = ""
     slot: int = -1                       # row of the engine's seen-token bitmap (repetition penalty)
-
-
-class PagedKVCache:
-    """Per-layer key/value page pools and a free list shared by all layers (a page index means
-    the same slot in every layer)."""
-
-    def __init__(self, cfg: ModelConfig, num_pages: int, device: torch.device, dtype: torch.dtype,
-                 n_kv_local: Optional[int] = None) -> None:
-        self.n_kv = n_kv_local or cfg.num_kv_heads
-        self.hd = cfg.head_dim
-        self.num_pages = num_pages
-        shape = (cfg.num_layers, num_pages, self.n_kv, PAGE, self.hd)      # 16 rows of one (page, head) are contiguous
-        self.k = torch.zeros(shape, device=device, dtype=dtype)
-        self.v = torch.zeros(shape, device=device, dtype=dtype)
-        self.free = list(range(num_pages - 1, -1, -1))
-
-    def pages_for(self, tokens: int) -> int:
-        return (tokens + PAGE - 1) // PAGE
-
-    def can_allocate(self, n: int) -> bool:
-        return len(self.free) >= n
-
-    def allocate(self, n: int) -> list[int]:
-        if len(self.free) < n:
-            raise RuntimeError("KV cache exhausted")
-        return [self.free.pop() for _ in range(n)]
-
-    def release(self, pages: list[int]) -> None:
-        self.free.extend(reversed(pages))
+    prev: int = -1                       # the last token that is in the cache (-1: none): part of the sequence's state
 
 
 def request_seed(r: Request) -> int:
@@ -115,27 +88,26 @@ def sample_tokens(logits: torch.Tensor, reqs: list[Request], ops: Any, seen: Opt
 
 
 class ServingEngine:
-    def __init__(self, model: KotodamaModel, *, device: torch.device | str = "cpu",
+    def __init__(self, model: Any, *, device: torch.device | str = "cpu",
                  dtype: torch.dtype = torch.float32, max_batch: int = 64, num_pages: Optional[int] = None,
                  max_ctx: Optional[int] = None, ops: Any = None, tp: Any = None,
-                 prefill_batch_tokens: int = 8192) -> None:
+                 prefill_batch_tokens: int = 8192, prefill_portion: int = 0) -> None:
         self.device = torch.device(device)
         self.dtype = dtype
         self.model = model.eval()
-        self.cfg: ModelConfig = model.config
+        self.cfg = model.config
         self.ops = ops or get_ops(self.device)
         self.tp = tp                                  # tensor-parallel helper (``serve.tp``) or None
-        if tp is not None:
-            tp.prepare_model(model)
-        self.arena = ParamArena(model, self.device, dtype, with_grads=False)
+        self.runner = make_runner(self)
+        self.arena = getattr(self.runner, "arena", None)
         cfg = self.cfg
         self.max_ctx = max_ctx or cfg.max_position_embeddings
         self.max_batch = max_batch
-        tpn = tp.size if tp is not None else 1
-        self.H, self.KV = cfg.num_attention_heads // tpn, cfg.num_kv_heads // tpn
-        self.hd, self.D = cfg.head_dim, cfg.hidden_size
+        if prefill_portion and not self.runner.continues:
+            raise ValueError(f"{type(self.runner).__name__} prefills whole prompts only")
+        self.prefill_portion = prefill_portion        # most tokens of one prompt per prefill pass; 0: the whole prompt
         pages = num_pages or max_batch * ((self.max_ctx + PAGE - 1) // PAGE)
-        self.cache = PagedKVCache(cfg, pages, self.device, dtype, n_kv_local=self.KV)
+        self.cache = self.runner.make_cache(pages)
         self.max_pages_per_req = (self.max_ctx + PAGE - 1) // PAGE
         self.waiting: list[Request] = []
         self.running: list[Request] = []
@@ -159,19 +131,6 @@ class ServingEngine:
         self.prefill_batch_tokens = prefill_batch_tokens     # tokens of one packed prefill pass over several prompts; 0: one prompt per pass
         self.stats = {"prefill_tokens": 0, "decode_tokens": 0, "prefill_s": 0.0, "decode_s": 0.0, "steps": 0,
                       "prefill_passes": 0}
-        ar = self.arena
-        self.layers = []
-        for i in range(cfg.num_layers):
-            p = f"layers.{i}."
-            g = lambda n: ar.view(p + n) if (p + n) in ar.by_name else None
-            dw = self.ops.decode_weight          # on CUDA: adds the tile-major copy that decode-size products stream
-            self.layers.append(dict(
-                wqkv=dw(ar.fused(p + "attn.q_proj.weight", p + "attn.v_proj.weight")), wo=dw(ar.view(p + "attn.o_proj.weight")),
-                wgu=dw(ar.fused(p + "ffn.gate_proj.weight", p + "ffn.up_proj.weight")), wd=dw(ar.view(p + "ffn.down_proj.weight")),
-                attn_norm=g("attn_norm.weight"), ffn_norm=g("ffn_norm.weight"), qn=g("attn.q_norm.weight"),
-                kn=g("attn.k_norm.weight"), aq=g("attn_res_query"), an=g("attn_res_norm.weight"),
-                mq=g("mlp_res_query"), mn=g("mlp_res_norm.weight")))
-        self.boundaries = frozenset(cfg.boundaries()) if cfg.attn_res else frozenset()
 
     # ------------------------------------------------------------------ requests
     def add_request(self, prompt: list[int], params: Optional[SamplingParams] = None) -> Request:
@@ -203,90 +162,72 @@ class ServingEngine:
     def has_work(self) -> bool:
         return bool(self.waiting or self.running)
 
-    # ------------------------------------------------------------------ model pass
+    # ------------------------------------------------------------------ model passes
     @torch.no_grad()
-    def _forward(self, ids: torch.Tensor, positions: torch.Tensor, slots: torch.Tensor, decode: Optional[dict],
-                 last_rows: torch.Tensor, seqs: Optional[dict] = None) -> torch.Tensor:
-        """Runs all layers on ``ids[N]``; keys/values go to ``slots`` (negative = padding, dropped).
-        ``decode`` holds the page table and context lengths for paged attention; ``None`` means a
-        causal prefill of ``prompts`` requests, each padded to ``N / prompts`` rows.
-        Returns logits for ``last_rows``."""
-        ops, cfg, ar = self.ops, self.cfg, self.arena
-        H, KV, hd = self.H, self.KV, self.hd
-        eps = cfg.norm_eps
-        cos, sin = self.model.rope_cos, self.model.rope_sin
-        N = ids.numel()
-        x = ops.embedding_fwd(ids, ar.view("embed_tokens.weight"))
-        committed: list[torch.Tensor] = []
-        partial: Optional[torch.Tensor] = x
-        for i, lw in enumerate(self.layers):
-            xn, _ = ops.route_norm_fwd(committed + [partial], lw["aq"], lw["an"], lw["attn_norm"], eps)
-            if i in self.boundaries:
-                committed = committed + [partial]
-                partial = None
-            qkv = ops.gemm_nt(xn, lw["wqkv"])
-            # QK-norm + RoPE; the same launch puts the new keys and values into their cache slots
-            qk, _ = ops.qknorm_rope_fwd(qkv, lw["qn"], lw["kn"], cos, sin, N, H, KV, hd, eps, positions=positions,
-                                        append=(self.cache.k[i], self.cache.v[i], slots))
-            k_rows = qk[:, H * hd:]
-            v_rows = qkv[:, (H + KV) * hd:]
-            if decode is None:
-                o, _ = ops.attention_fwd(qk[:, : H * hd].view(1, N, H, hd), k_rows.view(1, N, KV, hd),
-                                         v_rows.view(1, N, KV, hd), need_grad=False, **seqs)
-                attn = o.reshape(N, H * hd)
-            else:
-                attn = ops.paged_decode_attention(qk[:, : H * hd], self.cache.k[i], self.cache.v[i],
-                                                  decode["page_table"], decode["ctx_lens"], decode["max_ctx"], H, KV, hd)
-            partial = self._row_linear(attn, lw["wo"], partial)
-            xn2, _ = ops.route_norm_fwd(committed + [partial], lw["mq"], lw["mn"], lw["ffn_norm"], eps)
-            act = ops.swiglu_fwd(ops.gemm_nt(xn2, lw["wgu"]))
-            partial = self._row_linear(act, lw["wd"], partial)
-        g = lambda n: ar.view(n) if n in ar.by_name else None
-        xf, _ = ops.route_norm_fwd([s[last_rows] for s in committed + [partial]], g("final_res_query"),
-                                   g("final_res_norm.weight"), ar.view("norm.weight"), eps)
-        return ops.gemm_nt(xf, self.model.get_lm_head_weight())
-
-    def _row_linear(self, x: torch.Tensor, w: torch.Tensor, residual: Optional[torch.Tensor]) -> torch.Tensor:
-        if self.tp is None:
-            return self.ops.gemm_nt(x, w, residual=residual)
-        return self.tp.row_linear(self.ops, x, w, residual)
-
-    # ------------------------------------------------------------------ scheduling
-    def _prefill(self, reqs: list[Request]) -> None:
-        """One pass over the prompts of ``reqs``, packed back to back (no padding): the attention kernel
-        takes the sequence boundaries (``cu_seqlens``), every other op is per token."""
-        ns = [len(r.prompt) for r in reqs]
+    def _extend(self, parts: list[tuple[Request, list[int]]], rows: Optional[list[int]] = None) -> torch.Tensor:
+        """One pass over the next tokens of several requests (a prompt, or a portion of one), packed back to back
+        (no padding): the attention takes the sequence boundaries, every other op is per token.  Returns the logits
+        at ``rows`` of the packed tokens (default: each request's last)."""
+        ns = [len(t) for _, t in parts]
         total = sum(ns)
         ids = torch.empty(total, dtype=torch.long)
         slots = torch.empty(total, dtype=torch.long)
         pos = torch.empty(total, dtype=torch.int32)
+        prev = torch.empty(total, dtype=torch.int32)
         cu = [0]
-        for r, n in zip(reqs, ns):
+        for (r, toks), n in zip(parts, ns):
             at = cu[-1]
-            ids[at:at + n] = torch.tensor(r.prompt, dtype=torch.long)
-            t = torch.arange(n)
+            ids[at:at + n] = torch.tensor(toks, dtype=torch.long)
+            prev[at] = r.prev
+            prev[at + 1:at + n] = ids[at:at + n - 1].to(torch.int32)
+            t = torch.arange(r.ctx_len, r.ctx_len + n)
             slots[at:at + n] = torch.tensor(r.pages, dtype=torch.long)[t // PAGE] * PAGE + t % PAGE
             pos[at:at + n] = t.to(torch.int32)
             cu.append(at + n)
-        last = torch.tensor([c - 1 for c in cu[1:]])
         dev = self.device
-        seqs = {"cu_seqlens": torch.tensor(cu, dtype=torch.int32).to(dev), "max_seqlen": max(ns)}
-        logits = self._forward(ids.to(dev), pos.to(dev), slots.to(dev), None, last.to(dev), seqs=seqs)
+        last = torch.tensor(rows if rows is not None else [c - 1 for c in cu[1:]], dtype=torch.long)
+        batch = Batch(ids=ids.to(dev), positions=pos.to(dev), slots=slots.to(dev), rows=last.to(dev), prev=prev.to(dev),
+                      cu_seqlens=torch.tensor(cu, dtype=torch.int32).to(dev), max_seqlen=max(ns))
+        if self.runner.continues:
+            ctx = [r.ctx_len + n for (r, _), n in zip(parts, ns)]
+            table = np.zeros((len(parts), self.max_pages_per_req), dtype=np.int32)
+            for i, (r, _) in enumerate(parts):
+                table[i, : len(r.pages)] = r.pages
+            batch.page_table = torch.from_numpy(table).to(dev)
+            batch.ctx_lens = torch.tensor(ctx, dtype=torch.int32).to(dev)
+            batch.cu_context = torch.tensor([0] + np.cumsum(ctx).tolist(), dtype=torch.int32).to(dev)
+            batch.total_context = sum(ctx)
+            batch.max_ctx = max(ctx)
+        logits = self.runner.forward(batch)
+        for (r, toks), n in zip(parts, ns):
+            r.ctx_len += n
+            r.prev = int(toks[-1])
+        self.stats["prefill_tokens"] += total
+        self.stats["prefill_passes"] += 1
+        return logits
+
+    # ------------------------------------------------------------------ scheduling
+    def _prefill(self, parts: list[tuple[Request, list[int]]]) -> None:
+        """One prefill pass; requests whose prompt it completes get their first token."""
+        logits = self._extend(parts)
+        done = [i for i, (r, _) in enumerate(parts) if r.ctx_len >= len(r.prompt)]
+        if not done:
+            return
+        if len(done) < len(parts):
+            logits = logits[torch.tensor(done, device=logits.device)]
+        reqs = [parts[i][0] for i in done]
         if self.logit_trace is not None:
             self.logit_trace.append(([r.rid for r in reqs], logits.float().cpu()))
         toks = sample_tokens(logits, reqs, self.ops, self.seen).tolist()
         if self.tp is not None:
             toks = self.tp.sync_tokens(toks, self.device)
-        for r, n, tok in zip(reqs, ns, toks):
-            r.ctx_len = n
+        for r, tok in zip(reqs, toks):
             self._accept(r, int(tok))
-        self.stats["prefill_tokens"] += total
-        self.stats["prefill_passes"] += 1
 
-    def _admit(self) -> list[list[Request]]:
-        """Moves the waiting requests that fit (batch slots, pages) to ``running`` and groups them
-        into prefill passes of at most ``prefill_batch_tokens`` packed tokens (0: one prompt per pass)."""
-        admitted: list[Request] = []
+    def _admit(self) -> list[list[tuple[Request, list[int]]]]:
+        """Moves the waiting requests that fit (batch slots, pages) to ``running`` and groups the prompt tokens that
+        are due - the next portion of every request that is not prefilled yet - into passes of at most
+        ``prefill_batch_tokens`` packed tokens (0: one request per pass)."""
         while self.waiting and len(self.running) < self.max_batch:
             r = self.waiting[0]
             need = self.cache.pages_for(min(len(r.prompt) + r.params.max_new_tokens, self.max_ctx))
@@ -300,14 +241,18 @@ class ServingEngine:
                 self._init_seen(r)
             self.waiting.pop(0)
             self.running.append(r)
-            admitted.append(r)
-        groups: list[list[Request]] = []
-        cur: list[Request] = []
-        for r in admitted:
-            if cur and sum(len(q.prompt) for q in cur) + len(r.prompt) > self.prefill_batch_tokens:
+        groups: list[list[tuple[Request, list[int]]]] = []
+        cur: list[tuple[Request, list[int]]] = []
+        for r in self.running:
+            if r.ctx_len >= len(r.prompt):
+                continue
+            n = len(r.prompt) - r.ctx_len
+            if self.prefill_portion:
+                n = min(n, self.prefill_portion)
+            if cur and sum(len(t) for _, t in cur) + n > self.prefill_batch_tokens:
                 groups.append(cur)
                 cur = []
-            cur.append(r)
+            cur.append((r, r.prompt[r.ctx_len: r.ctx_len + n]))
         if cur:
             groups.append(cur)
         return groups
@@ -339,26 +284,30 @@ class ServingEngine:
         elif r.ctx_len + 1 >= self.max_ctx:
             r.finished, r.finish_reason = True, "context"
 
-    def _decode_inputs(self, reqs: list[Request]):
+    def _decode_inputs(self, reqs: list[Request], tokens: list[int]):
         """Static device buffers for a decode step; the page table is rebuilt only when the set of
-        running requests changes (pages are assigned once, at admission)."""
+        running requests (or the pages they hold) changes."""
         B = len(reqs)
-        key = tuple(r.rid for r in reqs)
+        key = tuple((r.rid, len(r.pages)) for r in reqs)
         # static buffers and captured graphs are kept per batch size: a batch size that comes back
         # (requests of unequal length retire one by one) replays its old graphs
         st = self._dec_states.get(B)
         if st is None:
-            # ids | slots (int64), pos | ctx (int32) live in ONE device buffer with a pinned host twin: a decode
-            # step costs one host -> device copy of 24 bytes per request
+            # ids | slots (int64), pos | ctx (int32) and, for families whose embedding looks at it, the token before
+            # (int32) live in ONE device buffer with a pinned host twin: a decode step costs one host -> device copy
+            # of 24 (28) bytes per request
             dev = self.device
-            packed = torch.zeros(24 * B, dtype=torch.uint8, device=dev)
-            host = torch.zeros(24 * B, dtype=torch.uint8, pin_memory=dev.type == "cuda")
+            width = 28 if self.runner.needs_prev else 24
+            packed = torch.zeros(width * B, dtype=torch.uint8, device=dev)
+            host = torch.zeros(width * B, dtype=torch.uint8, pin_memory=dev.type == "cuda")
             cut = lambda t, lo, hi, dt: t[lo * B: hi * B].view(dt)
             st = {"B": B, "key": None, "packed": packed, "host": host,
                   "ids": cut(packed, 0, 8, torch.long), "slots": cut(packed, 8, 16, torch.long),
                   "pos": cut(packed, 16, 20, torch.int32), "ctx": cut(packed, 20, 24, torch.int32),
                   "h_ids": cut(host, 0, 8, torch.long).numpy(), "h_slots": cut(host, 8, 16, torch.long).numpy(),
                   "h_pos": cut(host, 16, 20, torch.int32).numpy(), "h_ctx": cut(host, 20, 24, torch.int32).numpy(),
+                  "prev": cut(packed, 24, 28, torch.int32) if width == 28 else None,
+                  "h_prev": cut(host, 24, 28, torch.int32).numpy() if width == 28 else None,
                   "table": torch.zeros(B, self.max_pages_per_req, dtype=torch.int32, device=dev),
                   "rows": torch.arange(B, device=dev), "idx": np.arange(B), "graphs": {}}
             self._dec_states[B] = st
@@ -370,31 +319,37 @@ class ServingEngine:
             st["host_table"] = table
             st["key"] = key
         lens = np.fromiter((r.ctx_len for r in reqs), dtype=np.int64, count=B)
-        st["h_ids"][:] = np.fromiter((r.generated[-1] for r in reqs), dtype=np.int64, count=B)
+        st["h_ids"][:] = tokens
         st["h_slots"][:] = st["host_table"][st["idx"], lens // PAGE].astype(np.int64) * PAGE + lens % PAGE
         st["h_pos"][:] = lens
         st["h_ctx"][:] = lens + 1
+        if st["h_prev"] is not None:
+            st["h_prev"][:] = np.fromiter((r.prev for r in reqs), dtype=np.int32, count=B)
         st["packed"].copy_(st["host"], non_blocking=True)
         return st
 
-    def _decode(self) -> None:
-        reqs = self.running
-        B = len(reqs)
-        st = self._decode_inputs(reqs)
+    @torch.no_grad()
+    def _decode_pass(self, reqs: list[Request], tokens: list[int]) -> tuple[torch.Tensor, Optional[torch.Tensor]]:
+        """One token per request against the cache, on CUDA as the replay of a captured graph.  Returns the logits and
+        (from a graph) the argmax tokens.  The caller reads something back before the next pass (the host
+        twin of the inputs is reused)."""
+        st = self._decode_inputs(reqs, tokens)
         max_ctx = max(r.ctx_len for r in reqs) + 1
-        bucket = min(self.max_ctx, ((max_ctx + 511) // 512) * 512)       # grid of the split-KV kernel
-        decode = {"page_table": st["table"], "ctx_lens": st["ctx"], "max_ctx": bucket}
-        greedy = all(r.params.temperature == 0 and r.params.repetition_penalty == 1.0 for r in reqs)
+        # grid of the split-KV kernel, where the family's attention kernel is launched for a context size
+        bucket = min(self.max_ctx, ((max_ctx + 511) // 512) * 512) if self.runner.context_buckets else self.max_ctx
+        batch = Batch(ids=st["ids"], positions=st["pos"], slots=st["slots"], rows=st["rows"], prev=st["prev"],
+                      page_table=st["table"], ctx_lens=st["ctx"], max_ctx=bucket, decode=True)
+        toks = None
         if self.device.type == "cuda" and self.use_cuda_graphs:
             g = st["graphs"].get(bucket)
             if g is None:
                 # one eager pass first: lazy initialisation must not happen under capture
-                self._forward(st["ids"], st["pos"], st["slots"], decode, st["rows"])
+                self.runner.forward(batch)
                 torch.cuda.synchronize()
                 graph = torch.cuda.CUDAGraph()
                 # the captured launches are programmatic dependents of one another (the graph keeps the edges)
                 with torch.cuda.graph(graph), self.ops.dependent_launch(self.dependent_launch):
-                    logits = self._forward(st["ids"], st["pos"], st["slots"], decode, st["rows"])
+                    logits = self.runner.forward(batch)
                     toks = self.ops.argmax(logits)
                 g = st["graphs"][bucket] = (graph, logits, toks)
             if self.graph_ms is not None:            # device time of the replay alone (what the host adds is wall - this)
@@ -406,9 +361,19 @@ class ServingEngine:
             else:
                 g[0].replay()
             logits, toks = g[1], g[2]
-            toks = toks if greedy else sample_tokens(logits, reqs, self.ops, self.seen)
         else:
-            logits = self._forward(st["ids"], st["pos"], st["slots"], decode, st["rows"])
+            logits = self.runner.forward(batch)
+        for r, t in zip(reqs, tokens):
+            r.ctx_len += 1
+            r.prev = int(t)
+        self.stats["decode_tokens"] += len(reqs)
+        return logits, toks
+
+    def _decode(self, reqs: list[Request]) -> None:
+        B = len(reqs)
+        greedy = all(r.params.temperature == 0 and r.params.repetition_penalty == 1.0 for r in reqs)
+        logits, toks = self._decode_pass(reqs, [r.generated[-1] for r in reqs])
+        if toks is None or not greedy:
             toks = sample_tokens(logits, reqs, self.ops, self.seen)
         if self.logit_trace is not None:
             self.logit_trace.append(([r.rid for r in reqs], logits[:B].float().cpu()))
@@ -418,9 +383,60 @@ class ServingEngine:
             self.graph_ms += [a.elapsed_time(b) for a, b in self._graph_events]     # the token read above synchronised
             self._graph_events.clear()
         for r, t in zip(reqs, toks):
-            r.ctx_len += 1
             self._accept(r, int(t))
-        self.stats["decode_tokens"] += B
+
+    # ------------------------------------------------------------------ sequences fed by the caller
+    def open(self) -> Request:
+        """A sequence whose tokens the caller supplies through :meth:`feed`; it holds cache pages until :meth:`close`."""
+        if not self.runner.continues:
+            raise ValueError(f"{type(self.runner).__name__} cannot continue a cached sequence token by token")
+        r = Request(self._next_id, [], SamplingParams())
+        self._next_id += 1
+        return r
+
+    def feed(self, entries: list[tuple[Request, list[int], list[int]]]) -> list[torch.Tensor]:
+        """Advances opened sequences by their next tokens, from the cache that earlier calls left.  An entry is
+        ``(sequence, tokens, places)``; returns per entry the fp32 logits on the host, ``[len(places), vocab]``.  A single
+        further token takes the decode pass, anything else the packed pass of a prompt."""
+        for r, toks, places in entries:
+            if not toks:
+                raise ValueError("an entry without tokens")
+            bad = [t for t in toks if not 0 <= t < self.cfg.vocab_size]
+            if bad or any(not 0 <= p < len(toks) for p in places):
+                raise ValueError(f"token ids outside the vocabulary ({bad[:3]}) or places outside the tokens")
+            n = r.ctx_len + len(toks)
+            if n > self.max_ctx:
+                raise ValueError(f"sequence of {n} tokens does not fit the context of {self.max_ctx}")
+            more = self.cache.pages_for(n) - len(r.pages)
+            if more > 0:
+                r.pages = r.pages + self.cache.allocate(more)
+        out: list[Any] = [None] * len(entries)
+        single = [i for i, (r, toks, _) in enumerate(entries) if len(toks) == 1 and r.ctx_len > 0]
+        packed = [i for i in range(len(entries)) if i not in set(single)]
+        if single:
+            logits, _ = self._decode_pass([entries[i][0] for i in single], [entries[i][1][0] for i in single])
+            logits = logits.float().cpu()
+            for k, i in enumerate(single):
+                out[i] = logits[k:k + 1][[0] * len(entries[i][2])]
+        while packed:
+            group = [packed.pop(0)]
+            while packed and sum(len(entries[i][1]) for i in group + packed[:1]) <= self.prefill_batch_tokens:
+                group.append(packed.pop(0))
+            rows, at = [], 0
+            for i in group:
+                rows += [at + p for p in entries[i][2]]
+                at += len(entries[i][1])
+            logits = self._extend([entries[i][:2] for i in group], rows or [at - 1]).float().cpu()
+            at = 0
+            for i in group:
+                n = len(entries[i][2])
+                out[i] = logits[at:at + n]
+                at += n
+        return out
+
+    def close(self, r: Request) -> None:
+        self._release(r)
+        r.finished, r.finish_reason = True, "closed"
 
     def step(self) -> list[Request]:
         """Admit and prefill what fits, advance every running request by one token, retire the
@@ -430,11 +446,11 @@ class ServingEngine:
         for group in self._admit():
             self._prefill(group)
         t1 = time.perf_counter()
-        live = [r for r in self.running if not r.finished]
         done = [r for r in self.running if r.finished]
-        self.running = live
-        if live:
-            self._decode()
+        self.running = [r for r in self.running if not r.finished]
+        ready = [r for r in self.running if r.generated]            # the others are still being prefilled
+        if ready:
+            self._decode(ready)
         done += [r for r in self.running if r.finished]
         self.running = [r for r in self.running if not r.finished]
         for r in done:
