@@ -45,6 +45,8 @@ constexpr int FWD_THREADS = 320;                   // 8 softmax warps, MMA warp,
 struct FlashParams {
     int B, T, H, KV;
     const int* cu_seqlens;                         // [B + 1] token offsets, or null: sequence b = rows [b*T, (b+1)*T)
+    const int* cu_keys;                            // [B + 1] key offsets when keys and queries differ in number: the
+                                                   // queries of a sequence are then the last of its key positions
     float scale_log2;                              // softmax scale * log2(e)
     __nv_bfloat16* out;                            // token-major, heads side by side
     long long out_stride;                          // elements between tokens of `out`
@@ -115,8 +117,14 @@ flash_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant_
         seq_row0 = b * p.T;
         Tb = p.T;
     }
+    int key_row0 = seq_row0, ahead = 0;            // first key row; keys in front of the first query
+    if (p.cu_keys) {
+        key_row0 = p.cu_keys[b];
+        ahead = p.cu_keys[b + 1] - key_row0 - Tb;
+    }
     // key tiles of this query tile; a tile that starts past the sequence end has none
-    const int n = qt * BT < Tb ? qt + 1 : 0;
+    const int n = qt * BT < Tb ? (ahead + min(qt * BT + BT, Tb) + BT - 1) / BT : 0;
+    const int qpos = ahead + qt * BT;              // key position of the tile's first query
 
     if (threadIdx.x == 0) {
         tc::mbar_init(q_ready, 8);
@@ -155,7 +163,7 @@ flash_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant_
                 const int ks = j % KST;
                 if (!tc::mbar_wait(k_empty + ks, ((j / KST) & 1) ^ 1, abort_flag)) return false;
                 tc::mbar_expect_tx(k_full + ks, TB);
-                load_tile<HD>(sK + ks * TB, &tmK, k_full + ks, kx, seq_row0 + j * BT);
+                load_tile<HD>(sK + ks * TB, &tmK, k_full + ks, kx, key_row0 + j * BT);
                 return true;
             };
             bool ok = load_k(0) && (n < 2 || load_k(1));
@@ -163,7 +171,7 @@ flash_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant_
                 const int vs = j % VST;
                 if (!tc::mbar_wait(v_empty + vs, ((j / VST) & 1) ^ 1, abort_flag)) { ok = false; break; }
                 tc::mbar_expect_tx(v_full + vs, TB);
-                load_tile<HD>(sV + vs * TB, &tmV, v_full + vs, vx, seq_row0 + j * BT);
+                load_tile<HD>(sV + vs * TB, &tmV, v_full + vs, vx, key_row0 + j * BT);
                 if (j + 2 < n) ok = load_k(j + 2);
             }
             if (!ok) atomicMax(p.status, (int)KB_TIMEOUT_TMA);
@@ -253,8 +261,8 @@ flash_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant_
             tc::tmem_ld32(tmem_s + hf * 64 + 32, reinterpret_cast<uint32_t*>(s + 32));
             tc::tmem_ld_wait();
             KB_TICK(2, tk)                                              // tensor-memory load
-            if (j == qt) {                                          // diagonal tile: causal mask
-                const int cmax = r - hf * 64;
+            if (j * BT + BT - 1 > qpos) {                           // tile on the diagonal: causal mask
+                const int cmax = qpos - j * BT + r - hf * 64;
 #pragma unroll
                 for (int c = 0; c < 64; ++c) s[c] = c <= cmax ? s[c] : -INFINITY;
             }
@@ -373,7 +381,7 @@ flash_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant_
                         }
                     }
                 }
-                if (valid && hf == 0) {
+                if (valid && hf == 0 && p.lse) {
                     const long long base = p.cu_seqlens ? (long long)seq_row0 : (long long)b * p.lse_bs;
                     p.lse[(long long)head * p.lse_hs + base + qt * BT + r] = (m_used + log2f(l) - TRUNC_BIAS_LOG2) * LN2;
                 }
@@ -422,28 +430,27 @@ KB_API int kb_attn_dbg_read(long long* host16) {
 }
 #endif
 
-// q/k/v: token-major matrices [total tokens, *] whose rows hold the heads side by side (row strides
-// in elements; *_col0 = column of head 0).  out: token-major with `out_stride` elements per token.
-// Fixed-length batches: cu_seqlens null, B sequences of T tokens, lse[B, H, T].  Packed sequences:
-// cu_seqlens[B + 1] (device), `total` tokens, max_T the longest sequence, lse[H, total].
-KB_API int kb_flash_fwd(const void* q, long long q_stride, int q_cols, int q_col0, const void* k, long long k_stride,
-                        int k_cols, int k_col0, const void* v, long long v_stride, int v_cols, int v_col0, void* out,
-                        long long out_stride, float* lse, const int* cu_seqlens, long long total, int B, int max_T, int H,
-                        int KV, int hd, float scale, int* status, cudaStream_t st) {
+static int flash_fwd_impl(const void* q, long long q_stride, int q_cols, int q_col0, const void* k, long long k_stride,
+                          int k_cols, int k_col0, const void* v, long long v_stride, int v_cols, int v_col0, void* out,
+                          long long out_stride, float* lse, const int* cu_seqlens, long long total, const int* cu_keys,
+                          long long total_keys, int B, int max_T, int H, int KV, int hd, float scale, int* status, cudaStream_t st) {
     if ((hd != 128 && hd != 64) || max_T < 1 || B < 1 || KV < 1 || H % KV != 0) return 5;
     if (!operand_ok(q, q_stride, q_col0) || !operand_ok(k, k_stride, k_col0) || !operand_ok(v, v_stride, v_col0)) return 6;
     if (((uintptr_t)out & 15) || (out_stride & 7)) return 6;
+    if ((cu_keys != nullptr) && !cu_seqlens) return 5;
     const long long rows = cu_seqlens ? total : (long long)B * max_T;
+    const long long key_rows = cu_keys ? total_keys : rows;
     CUtensorMap tmQ, tmK, tmV;
     int r = make_rows_tmap(&tmQ, q, rows, q_cols, q_stride);
     if (r) return r;
-    r = make_rows_tmap(&tmK, k, rows, k_cols, k_stride);
+    r = make_rows_tmap(&tmK, k, key_rows, k_cols, k_stride);
     if (r) return r;
-    r = make_rows_tmap(&tmV, v, rows, v_cols, v_stride);
+    r = make_rows_tmap(&tmV, v, key_rows, v_cols, v_stride);
     if (r) return r;
     FlashParams p;
     p.B = B; p.T = max_T; p.H = H; p.KV = KV;
     p.cu_seqlens = cu_seqlens;
+    p.cu_keys = cu_keys;
     p.scale_log2 = scale * LOG2E;
     p.out = (__nv_bfloat16*)out;
     p.out_stride = out_stride;
@@ -457,4 +464,27 @@ KB_API int kb_flash_fwd(const void* q, long long q_stride, int q_cols, int q_col
     p.n_tiles = (max_T + BT - 1) / BT;
     p.status = status;
     return hd == 128 ? launch_fwd<128>(tmQ, tmK, tmV, p, max_T, st) : launch_fwd<64>(tmQ, tmK, tmV, p, max_T, st);
+}
+
+// q/k/v: token-major matrices [total tokens, *] whose rows hold the heads side by side (row strides
+// in elements; *_col0 = column of head 0).  out: token-major with `out_stride` elements per token.
+// Fixed-length batches: cu_seqlens null, B sequences of T tokens, lse[B, H, T].  Packed sequences:
+// cu_seqlens[B + 1] (device), `total` tokens, max_T the longest sequence, lse[H, total].
+KB_API int kb_flash_fwd(const void* q, long long q_stride, int q_cols, int q_col0, const void* k, long long k_stride,
+                        int k_cols, int k_col0, const void* v, long long v_stride, int v_cols, int v_col0, void* out,
+                        long long out_stride, float* lse, const int* cu_seqlens, long long total, int B, int max_T, int H,
+                        int KV, int hd, float scale, int* status, cudaStream_t st) {
+    return flash_fwd_impl(q, q_stride, q_cols, q_col0, k, k_stride, k_cols, k_col0, v, v_stride, v_cols, v_col0, out, out_stride,
+                          lse, cu_seqlens, total, nullptr, 0, B, max_T, H, KV, hd, scale, status, st);
+}
+
+// Packed queries against packed contexts: the queries of sequence b (rows cu_seqlens[b] .. cu_seqlens[b + 1] of q) are
+// the last of its key positions (rows cu_keys[b] .. cu_keys[b + 1] of k and v); max_T bounds the queries of a sequence.
+KB_API int kb_flash_fwd_context(const void* q, long long q_stride, int q_cols, const void* k, long long k_stride, int k_cols,
+                                const void* v, long long v_stride, int v_cols, void* out, long long out_stride,
+                                const int* cu_seqlens, long long total, const int* cu_keys, long long total_keys, int B, int max_T,
+                                int H, int KV, int hd, float scale, int* status, cudaStream_t st) {
+    if (!cu_seqlens || !cu_keys) return 5;
+    return flash_fwd_impl(q, q_stride, q_cols, 0, k, k_stride, k_cols, 0, v, v_stride, v_cols, 0, out, out_stride, nullptr, cu_seqlens,
+                          total, cu_keys, total_keys, B, max_T, H, KV, hd, scale, status, st);
 }

@@ -1014,14 +1014,17 @@ KB_API int kb_paged_decode_merged(const void* q, long long q_stride, const void*
 }
 
 // Greedy sampling: out[row] = argmax_j logits[row][j] (first index on ties).
-__global__ void argmax_kernel(const bf16* __restrict__ logits, long long stride, int V, long long* __restrict__ out) {
+__device__ __forceinline__ float logit_f(bf16 v) { return __bfloat162float(v); }
+__device__ __forceinline__ float logit_f(float v) { return v; }
+template <typename T>
+__global__ void argmax_kernel(const T* __restrict__ logits, long long stride, int V, long long* __restrict__ out) {
     __shared__ float bv[32];
     __shared__ int bi[32];
-    const bf16* lg = logits + (size_t)blockIdx.x * stride;
+    const T* lg = logits + (size_t)blockIdx.x * stride;
     float best = -INFINITY;
     int idx = 0x7fffffff;
     for (int j = threadIdx.x; j < V; j += blockDim.x) {
-        const float v = __bfloat162float(lg[j]);
+        const float v = logit_f(lg[j]);
         if (v > best || (v == best && j < idx)) { best = v; idx = j; }
     }
 #pragma unroll
@@ -1045,8 +1048,10 @@ __global__ void argmax_kernel(const bf16* __restrict__ logits, long long stride,
         if (lane == 0) out[blockIdx.x] = idx;
     }
 }
-KB_API int kb_argmax(const void* logits, long long stride, int rows, int V, long long* out, cudaStream_t st) {
-    argmax_kernel<<<rows, 512, 0, st>>>((const bf16*)logits, stride, V, out);
+// type: 0 bf16, 1 fp32 logits
+KB_API int kb_argmax(const void* logits, long long stride, int rows, int V, long long* out, int type, cudaStream_t st) {
+    if (type == 1) argmax_kernel<float><<<rows, 512, 0, st>>>((const float*)logits, stride, V, out);
+    else argmax_kernel<bf16><<<rows, 512, 0, st>>>((const bf16*)logits, stride, V, out);
     return kb_launch_status();
 }
 

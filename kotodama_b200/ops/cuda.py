@@ -24,6 +24,7 @@ _LL = ctypes.c_longlong
 _F = ctypes.c_float
 
 _FMT = {torch.float16: 0, torch.bfloat16: 1}
+_TYPE = {torch.bfloat16: 0, torch.float32: 1}      # activation type of kernels that exist for both
 _OUT = {torch.float16: 0, torch.bfloat16: 1, torch.float32: 2}
 
 
@@ -69,7 +70,8 @@ class CudaOps(TorchOps):
         self.fp8_pair = int(os.environ.get("KOTODAMA_FP8_PAIR", "0"))       # mx kernel: 1 = SM-pair tiles, 0 = one CTA per tile (faster, default)
         for name in ("kb_route_bwd_grid", "kb_qknorm_grid_warps", "kb_route_pipe_grid", "kb_route_blocked_ok",
                      "kb_route_blocked_grid"):
-            getattr(self.lib, name).restype = _I
+            if hasattr(self.lib, name):          # a library of the serving kernels alone does not have the training ones
+                getattr(self.lib, name).restype = _I
 
     # ------------------------------------------------------------------ utils
     def _rc(self, rc: int, what: str) -> None:
@@ -110,6 +112,8 @@ class CudaOps(TorchOps):
         decode-size product launched as a dependent may fetch it before the kernels ahead have finished.
         ``diag`` is added to the diagonal of the result (fused into the CTA-pair kernel's epilogue when
         there is an addend, a separate in-place add otherwise)."""
+        if a.dtype == torch.float32:
+            return self._gemm_f32(a, b, M, N, K, a_mn, b_mn, out, cin, alpha, beta, batch)
         out_dtype = out_dtype or (out.dtype if out is not None else a.dtype)
         lead = (batch,) if batch > 1 else ()
         if out is None:
@@ -204,6 +208,20 @@ class CudaOps(TorchOps):
         self._rc(rc, "kb_gemm")
         if diag:
             out.diagonal(dim1=-2, dim2=-1).add_(diag)
+        return out
+
+    def _gemm_f32(self, a, b, M, N, K, a_mn, b_mn, out, cin, alpha, beta, batch):
+        """The 32-bit mode: plain fp32 products (no reduced-precision matrix mode)."""
+        if a_mn or alpha != 1.0 or (cin is not None and beta != 1.0) or b.dtype != torch.float32:
+            raise KernelError(f"fp32 products take K-major fp32 operands and alpha = beta = 1, got {a.dtype}, {b.dtype}")
+        if out is None:
+            out = torch.empty(*((batch,) if batch > 1 else ()), M, N, device=a.device, dtype=torch.float32)
+        if a.stride(-1) != 1 or b.stride(-1) != 1 or out.stride(-1) != 1 or out.dtype != torch.float32 or (
+                cin is not None and cin.stride() != out.stride()):
+            raise KernelError("fp32 products take row-major operands; the addend is laid out like the output")
+        bs = lambda t: t.stride(0) if batch > 1 else 0
+        self._call("kb_gemm_f32", _p(a), _p(b), _p(out), _p(cin), _I(M), _I(N), _I(K), _I(batch), _LL(a.stride(-2)),
+                   _LL(b.stride(-2)), _LL(out.stride(-2)), _LL(bs(a)), _LL(bs(b)), _LL(bs(out)), _I(int(b_mn)), _p(None), _st())
         return out
 
     # ------------------------------------------------------------------ block-scaled fp8
@@ -661,8 +679,157 @@ class CudaOps(TorchOps):
         self.launches += 1
         return out
 
+    # ------------------------------------------------------------------ latent attention, output norms, experts
+    def flash_latent(self, dtype):
+        return dtype == torch.bfloat16
+
+    def latent_multiple(self, dtype):
+        return 128 if dtype == torch.bfloat16 else 8       # 128-row blocks of the tensor-core kernel
+
+    def embed_pairs(self, ids, prev, table, bigram, consts):
+        N, D = ids.numel(), table.shape[1]
+        x = torch.empty(N, D, device=table.device, dtype=torch.float32)
+        h = x if table.dtype == torch.float32 else torch.empty(N, D, device=table.device, dtype=table.dtype)
+        self._call("kb_embed_pairs", _p(ids), _p(prev), _p(table), _p(bigram), _LL(consts[0]), _LL(consts[1]), _LL(consts[2]),
+                   _p(x), _p(h), _I(N), _I(D), _I(table.shape[0]), _I(_TYPE[table.dtype]), _p(self.status(table.device)), _st())
+        return x, h
+
+    def latent_append(self, rows, w, width, eps, pages, slots):
+        N, R = rows.shape
+        out = torch.empty(N, R, device=rows.device, dtype=rows.dtype)
+        self._call("kb_latent_append", _p(rows), _LL(rows.stride(0)), _p(w), _I(width), _F(eps), _p(pages), _p(slots), _p(out),
+                   _I(N), _I(R), _LL(pages.shape[0] * pages.shape[1]), _I(_TYPE[rows.dtype]), _p(self.status(rows.device)), _st())
+        return out
+
+    def latent_gather(self, pages, page_table, cu_context, total):
+        R = pages.shape[-1]
+        out = torch.empty(total, R, device=pages.device, dtype=pages.dtype)
+        self._call("kb_latent_gather", _p(pages), _p(page_table), _I(page_table.shape[1]), _p(cu_context), _I(page_table.shape[0]),
+                   _p(out), _I(total), _I(R), _I(pages.shape[0]), _I(_TYPE[pages.dtype]), _p(self.status(pages.device)), _st())
+        return out
+
+    def latent_attention(self, q, pages, page_table, ctx_lens, cu_seqlens, max_q, max_ctx, scale):
+        """bf16: the tensor-core kernel (``csrc/latent_attn_sm100.cu``); the 32-bit mode, and latents too large for its
+        ring, take the plain kernel (``csrc/latent_attn.cu``)."""
+        N, H, R = q.shape
+        B = page_table.shape[0]
+        dev = q.device
+        out = torch.empty(N, H, R, device=dev, dtype=q.dtype)
+        if not q.is_contiguous():
+            raise KernelError("latent queries must be dense")
+        if q.dtype == torch.bfloat16 and self.lib.kb_latent_ok(_I(B), _I(max_q), _I(H), _I(R)):
+            cols = self.lib.kb_latent_cols(_I(max_q), _I(H))
+            slots = self.lib.kb_latent_partials(_I(B), _I(max_q), _I(H))
+            part_o = torch.empty(slots * cols * R, device=dev, dtype=torch.float32)
+            part_ml = torch.empty(slots * cols * 2, device=dev, dtype=torch.float32)
+            unit_off = torch.empty(2049, device=dev, dtype=torch.int32)
+            self._call("kb_latent_attn", _p(q), _p(pages), _p(page_table), _I(page_table.shape[1]), _I(pages.shape[0]), _p(ctx_lens),
+                       _p(cu_seqlens), _I(B), _I(max_q), _I(N), _I(H), _I(R), _F(scale), _p(part_o), _p(part_ml), _p(unit_off),
+                       _p(out), _p(self.status(dev)), _st())
+            self.launches += 1
+            return out
+        self._call("kb_latent_attn_plain", _p(q), _p(pages), _p(page_table), _I(page_table.shape[1]), _I(pages.shape[0]), _p(ctx_lens),
+                   _p(cu_seqlens), _I(B), _p(out), _I(N), _I(H), _I(R), _F(scale), _I(_TYPE[q.dtype]), _p(self.status(dev)), _st())
+        return out
+
+    def attention_context(self, q, k, v, cu_seqlens, cu_context, max_q, scale):
+        Nq, H, hd = q.shape
+        Nk, KV = k.shape[0], k.shape[1]
+        if q.dtype != torch.bfloat16 or hd not in (64, 128) or v.shape[2] != hd:
+            raise KernelError(f"flash attention takes bf16 heads of 64 or 128, got {q.dtype} {tuple(q.shape)} {tuple(v.shape)}")
+        for t in (q, k, v):
+            if t.stride(2) != 1 or t.stride(1) != hd:
+                raise KernelError("attention operands are token-major rows with the heads side by side")
+        out = torch.empty(Nq, H, hd, device=q.device, dtype=q.dtype)
+        self._call("kb_flash_fwd_context", _p(q), _LL(q.stride(0)), _I(H * hd), _p(k), _LL(k.stride(0)), _I(KV * hd), _p(v),
+                   _LL(v.stride(0)), _I(KV * hd), _p(out), _LL(H * hd), _p(cu_seqlens), _LL(Nq), _p(cu_context), _LL(Nk),
+                   _I(cu_seqlens.numel() - 1), _I(max_q), _I(H), _I(KV), _I(hd), _F(scale), _p(self.status(q.device)), _st())
+        return out
+
+    def head_gemm(self, a, w, transposed=False):
+        N, H, K = a.shape
+        M = w.shape[2] if transposed else w.shape[1]
+        out = torch.empty(N, H, M, device=a.device, dtype=a.dtype)
+        if H == 1:
+            self._gemm(a[:, 0], w[0], N, M, K, False, transposed, out=out[:, 0])
+        else:
+            self._gemm(a.transpose(0, 1), w, N, M, K, False, transposed, out=out.transpose(0, 1), batch=H)
+        return out
+
+    def activate(self, u, kind):
+        out = torch.empty_like(u)
+        self._call("kb_activate", _p(u), _p(out), _LL(u.numel()), _I({"gelu": 1, "relu2": 2}[kind]), _I(_TYPE[u.dtype]), _st())
+        return out
+
+    def _norm_add(self, x, y, ys, g, width, eps, at, wts, gate, dtype):
+        N, D = x.shape
+        h = x if dtype == torch.float32 else torch.empty(N, D, device=x.device, dtype=dtype)
+        self._call("kb_norm_add", _p(x), _p(y), _p(ys), _p(g), _p(h), _I(N), _I(D), _I(width), _F(eps), _p(at), _p(wts), _p(gate),
+                   _I(at.shape[1] if at is not None else 0), _LL(y.shape[0]), _I(_TYPE[y.dtype]), _p(self.status(x.device)), _st())
+        return h
+
+    def norm_add(self, x, y, g, width, eps):
+        return self._norm_add(x, y, None, g, width, eps, None, None, None, y.dtype)
+
+    def moe_combine_norm_add(self, x, ye, at, wts, ys, gate, g, width, eps, dtype):
+        return self._norm_add(x, ye, ys, g, width, eps, at, wts, gate, dtype)
+
+    def norm_rows(self, x, rows, w, width, eps, dtype):
+        out = torch.empty(rows.numel(), x.shape[1], device=x.device, dtype=dtype)
+        self._call("kb_norm_rows", _p(x), _p(rows), _p(w), _p(out), _I(rows.numel()), _I(x.shape[0]), _I(x.shape[1]), _I(width),
+                   _F(eps), _I(_TYPE[dtype]), _p(self.status(x.device)), _st())
+        return out
+
+    def moe_route(self, h, router, experts, top, scale, groups, keep):
+        N, D = h.shape
+        E = router.shape[0]
+        dev = h.device
+        logits = torch.empty(N, E, device=dev, dtype=torch.float32)
+        if N <= 256:
+            self._call("kb_router_dot", _p(h), _p(router), _p(logits), _I(N), _I(E), _I(D), _I(_TYPE[h.dtype]), _st())
+        else:
+            self.gemm_nt(h, router, out=logits)
+        gated = E > experts
+        ids = torch.empty(N, top, device=dev, dtype=torch.int32)
+        wts = torch.empty(N, top, device=dev, dtype=torch.float32)
+        gate = torch.empty(N, device=dev, dtype=torch.float32) if gated else None
+        self._call("kb_moe_select", _p(logits), _I(E), _I(N), _I(experts), _I(top), _F(scale), _I(groups), _I(keep), _I(int(gated)),
+                   _p(ids), _p(wts), _p(gate), _st())
+        return ids, wts, gate
+
+    def moe_experts(self, h, ids, up, down, kind):
+        N, top = ids.shape
+        E, ff, D = up.shape
+        A = N * top
+        dev = h.device
+        at = torch.empty(N, top, device=dev, dtype=torch.int32)
+        tok = torch.empty(A, device=dev, dtype=torch.int32)
+        offsets = torch.empty(E + 1, device=dev, dtype=torch.int32)
+        rows = torch.empty(A, D, device=dev, dtype=h.dtype)
+        self._call("kb_moe_group", _p(h), _p(ids), _I(N), _I(top), _I(E), _I(D * h.element_size()), _p(at), _p(tok), _p(offsets),
+                   _p(rows), _st())
+        self.launches += 1
+        u = self._grouped(rows, up, offsets, kind)
+        return self._grouped(u, down, offsets, None), at
+
+    def _grouped(self, rows, w, offsets, kind):
+        A, K = rows.shape
+        E, M, _ = w.shape
+        out = torch.empty(A, M, device=rows.device, dtype=rows.dtype)
+        if rows.dtype == torch.float32:
+            self._call("kb_gemm_f32", _p(rows), _p(w), _p(out), _p(None), _I(A), _I(M), _I(K), _I(E), _LL(K), _LL(K), _LL(M), _LL(0),
+                       _LL(M * K), _LL(0), _I(0), _p(offsets), _st())
+            return self.activate(out, kind) if kind else out
+        self._call("kb_gemm_grouped", _p(rows), _p(w), _p(out), _p(offsets), _I(A), _I(E), _I(M), _I(K), _LL(M),
+                   _I({None: 0, "gelu": 1, "relu2": 2}[kind]), _I(int(A <= 24 * E)), _p(self.status(rows.device)), _st())
+        return out
+
+    def softcap_(self, logits, cap):
+        self._call("kb_softcap", _p(logits), _LL(logits.numel()), _F(cap), _st())
+        return logits
+
     def argmax(self, logits):
         out = torch.empty(logits.shape[0], device=logits.device, dtype=torch.long)
         self._rc(self.lib.kb_argmax(_p(logits), _LL(logits.stride(0)), _I(logits.shape[0]), _I(logits.shape[1]),
-                                    _p(out), _st()), "kb_argmax")
+                                    _p(out), _I(_TYPE[logits.dtype]), _st()), "kb_argmax")
         return out
