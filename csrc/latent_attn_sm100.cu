@@ -156,8 +156,9 @@ latent_attn_sm100_kernel(const __grid_constant__ CUtensorMap tmC, const __grid_c
     const uint32_t tmem = *tmem_slot;
     const uint32_t tmem_s = tmem, tmem_o = tmem + 32;          // S^T: HG columns; O^T: HG columns per 128-row block
     const long long T = uoff[U];
-    const int g = blockIdx.x, G = gridDim.x;
-    const int t_begin = (int)(T * g / G), t_end = (int)(T * (g + 1) / G);
+    // pieces: no more than tiles, so that no piece is empty (the merge walks the pieces of a unit)
+    const int g = blockIdx.x, G = (int)(T < (long long)gridDim.x ? T : (long long)gridDim.x);
+    const int t_begin = g < G ? (int)(T * g / G) : 0, t_end = g < G ? (int)(T * (g + 1) / G) : 0;
     int u0 = 0;
     if (t_begin < t_end) {
         int hi = U;
@@ -393,13 +394,14 @@ latent_attn_sm100_kernel(const __grid_constant__ CUtensorMap tmC, const __grid_c
 // One block per (unit, column): weighs the pieces of the unit and writes the column's latent-space output.
 __global__ void __launch_bounds__(128)
 latent_merge_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml, const int* __restrict__ unit_off,
-                    const int* __restrict__ cu, bf16* __restrict__ out, int units, int cgs, int HG, int H, int R, int G) {
+                    const int* __restrict__ cu, bf16* __restrict__ out, int units, int cgs, int HG, int H, int R, int ctas) {
     kb_dep_trigger();
     kb_dep_wait();
     const int u = blockIdx.x, j = blockIdx.y, b = u / cgs, col = (u % cgs) * HG + j;
     const int q0 = cu ? cu[b] : b, nq = cu ? cu[b + 1] - q0 : 1;
     if (col >= nq * H) return;
     const long long T = unit_off[units];
+    const int G = (int)(T < (long long)ctas ? T : (long long)ctas);
     const int lo = unit_off[u], hi = unit_off[u + 1];
     bf16* dst = out + ((long long)q0 * H + col) * R;
     const int g0 = hi > lo ? (int)(((lo + 1ll) * G - 1) / T) : 0, g1 = hi > lo ? (int)(((long long)hi * G - 1) / T) : -1;
