@@ -61,8 +61,9 @@ def expert_ff(h, up, down):
     return gelu_erf(h @ up.t()) @ down.t()
 
 
-def route(h, w_router, r):
-    """Chosen experts and weights per token: [(expert, weight), ...]."""
+def route(h, w_router, r, margins=None):
+    """Chosen experts and weights per token: [(expert, weight), ...].  ``margins`` collects, per token, by how much (in
+    logits) the closest decision was taken."""
     picks = []
     for z in h @ w_router.t():
         s = torch.softmax(z, 0)
@@ -71,16 +72,24 @@ def route(h, w_router, r):
         g = r.get("groups")
         if g:
             size = E // g["count"]
-            best = sorted(range(g["count"]), key=lambda i: -float(s[i * size:(i + 1) * size].max()))[: g["keep"]]
+            ranked = sorted(range(g["count"]), key=lambda i: -float(s[i * size:(i + 1) * size].max()))
+            best = ranked[: g["keep"]]
             allowed = {e for i in best for e in range(i * size, (i + 1) * size)}
-        order = sorted(allowed, key=lambda e: -float(s[e]))[: r["top"]]
+        ordered = sorted(allowed, key=lambda e: -float(s[e]))
+        order = ordered[: r["top"]]
+        if margins is not None:
+            gap = float(z[order[-1]] - z[ordered[len(order)]]) if len(ordered) > len(order) else math.inf
+            if g and g["keep"] < g["count"]:
+                top = lambda i: float(z[i * size:(i + 1) * size].max())
+                gap = min(gap, top(best[-1]) - top(ranked[g["keep"]]))
+            margins.append(gap)
         picks.append([(e, s[e] * r["scale"]) for e in order])
     return picks
 
 
-def moe_ff(h, w, mlp):
+def moe_ff(h, w, mlp, margins=None):
     rows = []
-    for x, pick in zip(h, route(h, w["router"], mlp["router"])):
+    for x, pick in zip(h, route(h, w["router"], mlp["router"], margins)):
         y = torch.zeros_like(x)
         for e, g in pick:
             y = y + g * expert_ff(x[None], w[f"e{e}.up"], w[f"e{e}.down"])[0]
@@ -98,8 +107,9 @@ def sub(weights, prefix):
     return {k[len(prefix):]: v for k, v in weights.items() if k.startswith(prefix)}
 
 
-def forward(cfg, weights, tokens, layers_out=None):
-    """Logits [tokens, vocab]; ``layers_out`` collects the residual stream after every layer."""
+def forward(cfg, weights, tokens, layers_out=None, margins_out=None):
+    """Logits [tokens, vocab]; ``layers_out`` collects the residual stream after every layer, ``margins_out`` the routers'
+    margins per expert layer."""
     eps = cfg["norm"]["eps"]
     x = embed(tokens, weights["embed"], weights.get("bigram"), (cfg.get("embedding") or {}).get("bigram"))
     for i, layer in enumerate(cfg["layers"]):
@@ -107,7 +117,10 @@ def forward(cfg, weights, tokens, layers_out=None):
         x = x + rms(latent_attention(x, sub(w, "mix."), layer["mixer"], eps), w["norm1"], eps) * w["ls1"]
         mlp = layer["mlp"]
         if mlp is not None:
-            y = dense_ff(x, sub(w, "mlp.")) if mlp["kind"] == "dense" else moe_ff(x, sub(w, "mlp."), mlp)
+            margins = []
+            y = dense_ff(x, sub(w, "mlp.")) if mlp["kind"] == "dense" else moe_ff(x, sub(w, "mlp."), mlp, margins)
+            if margins and margins_out is not None:
+                margins_out.append(margins)
             x = x + rms(y, w["norm2"], eps) * w["ls2"]
         if layers_out is not None:
             layers_out.append(x.clone())
