@@ -104,7 +104,7 @@ def kernels(name: str, z: dict, batch: int = 64, ctx: int = 1280, tokens: int = 
     sets = max(2, int(400e6 // (B * ctx * R * 2)) + 1)
     lens = torch.full((B,), ctx, dtype=torch.int32, device=dev)
     tables = torch.randperm(B * mp, device=dev).to(torch.int32).view(B, mp).contiguous()
-    pages = [bf(B * mp, 16, R) for _ in range(sets)]
+    pages = [bf(B * mp, R // 64, 16, 64) for _ in range(sets)]
     q = bf(B, H, R)
     ms = timed([lambda i=i: ops.latent_attention(q, pages[i], tables, lens, None, 1, ctx, 0.088) for i in range(sets)])
     add("latent decode attention + merge", "decode attention", ms, B * ctx * R * 2 + 2 * B * H * R * 2, 4.0 * B * ctx * H * R)
@@ -162,19 +162,17 @@ def kernels(name: str, z: dict, batch: int = 64, ctx: int = 1280, tokens: int = 
             hs = [bf(n, D) for _ in range(4)]
             ms = timed([lambda x=x: ops.moe_route(x, router, E, top, 1.0, 8, 4) for x in hs])
             add(f"router + selection ({tag})", "row kernel", ms, (n * D + (E + 1) * D) * 2, 2.0 * n * D * (E + 1))
-            tmp = [torch.empty(n, top, device=dev, dtype=torch.int32) for _ in range(2)]
-            tok, o2, gr = torch.empty(A, device=dev, dtype=torch.int32), torch.empty(E + 1, device=dev, dtype=torch.int32), bf(A, D)
-            import ctypes
-            P, I = (lambda t: ctypes.c_void_p(t.data_ptr())), ctypes.c_int
-            st = lambda: ctypes.c_void_p(torch.cuda.current_stream().cuda_stream)
-            ms = timed([lambda x=x: ops._call("kb_moe_group", P(x), P(ids), I(n), I(top), I(E), I(D * 2), P(tmp[0]), P(tok), P(o2), P(gr), st())
-                        for x in hs])
+            plans = [ops.moe_route(x, router, E, top, 1.0, 8, 4) for x in hs]
+            # grouping turns the plan's ranks into places: every replay starts from a copy of the ranks
+            keep = [(p[3][0], p[3][1].clone()) if p[3] is not None else None for p in plans]
+            group = lambda x, p, k: ops._moe_group(x, p[0], E, None if k is None else (k[0], k[1].clone()))
+            ms = timed([lambda x=x, p=p, k=k: group(x, p, k) for x, p, k in zip(hs, plans, keep)])
             add(f"grouping + row gather ({tag})", "row kernel", ms, (n * D + A * D) * 2)
             xs = [torch.randn(n, D, device=dev) for _ in range(4)]
             ye, ys, wts, gate, g = bf(A, D), bf(n, D), torch.rand(n, top, device=dev), torch.rand(n, device=dev), torch.ones(D, device=dev)
             ms = timed([lambda x=x: ops.moe_combine_norm_add(x, ye, at, wts, ys, gate, g, D, 1e-5, torch.bfloat16) for x in xs])
             add(f"combine + norm + residual ({tag})", "row kernel", ms, A * D * 2 + n * D * (2 + 4 + 4 + 2))
-            del up, rows, u, ye, gr
+            del up, rows, u, ye
     # ---- prefill: attention, dense product, row kernels
     n = tokens
     qf, kf, vf = bf(n, H, 128), bf(n, H, 128), bf(n, H, 128)
@@ -209,7 +207,7 @@ def kernels(name: str, z: dict, batch: int = 64, ctx: int = 1280, tokens: int = 
     ms = timed([lambda x=x: ops.route_norm_fwd([x], None, None, nw, 1e-5) for x in xb])
     add("llama: RMS norm (prefill)", "row kernel", ms, n * D * 4)
     qc = [bf(n, H * 128 + R) for _ in range(3)]
-    pg = torch.zeros(n // 16, 16, R, device=dev, dtype=torch.bfloat16)
+    pg = torch.zeros(n // 16, R // 64, 16, 64, device=dev, dtype=torch.bfloat16)
     sl, cw = torch.arange(n, device=dev), torch.ones(R, device=dev)
     ms = timed([lambda x=x: ops.latent_append(x[:, H * 128:], cw, R, 1e-5, pg, sl) for x in qc])
     add("latent norm + cache append (prefill)", "row kernel", ms, n * R * 6)

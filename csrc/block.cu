@@ -3,6 +3,7 @@
 // The residual stream is fp32; T (bf16 or fp32) is the activation type.  Rows may be padded with zeros on the
 // right up to a multiple of 8 elements: `width` is the true size that means are taken over.
 // Compiled without fast-math: the fp32 mode is meant to be exact to fp32 rounding.
+#include "act.cuh"
 #include "vec.cuh"
 
 namespace {
@@ -43,7 +44,7 @@ __global__ void embed_pairs_kernel(const long long* __restrict__ ids, const int*
 template <typename T>
 __global__ void __launch_bounds__(256)
 latent_append_kernel(const T* __restrict__ rows, long long stride, const float* __restrict__ w, int width, float eps,
-                     T* __restrict__ pages, const long long* __restrict__ slots, T* __restrict__ out, int N, int R,
+                     T* __restrict__ pages, int W, const long long* __restrict__ slots, T* __restrict__ out, int N, int R,
                      long long num_slots, int* __restrict__ status) {
     kb_dep_trigger();
     kb_dep_wait();
@@ -70,13 +71,13 @@ latent_append_kernel(const T* __restrict__ rows, long long stride, const float* 
 #pragma unroll
         for (int j = 0; j < 8; ++j) v[j] = v[j] * r * g[j];
         if (out) store8(out + (long long)row * R + c, v);
-        if (s >= 0) store8(pages + s * R + c, v);
+        if (s >= 0) store8(pages + (s / PAGE) * PAGE * R + ((long long)(c / W) * PAGE + s % PAGE) * W + c % W, v);
     }
 }
 
 // Packed copy of the cached rows of every sequence; row -> sequence by binary search in the prefix sums.
 template <typename T>
-__global__ void latent_gather_kernel(const T* __restrict__ pages, const int* __restrict__ table, int max_pages,
+__global__ void latent_gather_kernel(const T* __restrict__ pages, int W, const int* __restrict__ table, int max_pages,
                                      const int* __restrict__ cu, int B, T* __restrict__ out, int total, int R, int num_pages,
                                      int* __restrict__ status) {
     kb_dep_trigger();
@@ -96,7 +97,7 @@ __global__ void latent_gather_kernel(const T* __restrict__ pages, const int* __r
         if (page < 0 || page >= num_pages) {
             if (c == 0 && status) atomicMax(status, (int)KB_BAD_INDEX);
         } else {
-            load8(pages + ((long long)page * PAGE + t % PAGE) * R + c, v);
+            load8(pages + (long long)page * PAGE * R + ((c / W) * PAGE + t % PAGE) * W + c % W, v);
         }
         store8(out + (long long)row * R + c, v);
     }
@@ -207,7 +208,8 @@ __global__ void activate_kernel(const T* __restrict__ u, T* __restrict__ out, lo
 #pragma unroll
         for (int j = 0; j < 8; ++j) {
             if (kind == 1) {
-                v[j] = 0.5f * v[j] * (1.0f + erff(v[j] * 0.70710678118654752f));
+                if constexpr (sizeof(T) == 2) v[j] = gelu_bf16(v[j]);
+                else v[j] = 0.5f * v[j] * (1.0f + erff(v[j] * 0.70710678118654752f));
             } else {
                 const float p = fmaxf(v[j], 0.f);
                 v[j] = p * p;
@@ -238,6 +240,7 @@ inline int row_threads(int D) {
 
 }  // namespace
 
+// The latent cache is [pages, R / W, 16, W]: W columns of a page's 16 tokens are contiguous.
 // Types: 0 = bf16, 1 = fp32 activations.  D and R are multiples of 8, bases 16-byte aligned.
 KB_API int kb_embed_pairs(const long long* ids, const int* prev, const void* table, const void* bigram, long long buckets,
                           long long mul_prev, long long mul_cur, float* x, void* h, int N, int D, int V, int type, int* status,
@@ -250,25 +253,25 @@ KB_API int kb_embed_pairs(const long long* ids, const int* prev, const void* tab
     return kb_launch_dep(embed_pairs_kernel<float>, grid, dim3(256), 0, st, ids, prev, (const float*)table, (const float*)bigram,
                          buckets, mul_prev, mul_cur, x, (float*)h, N, D, V, status);
 }
-KB_API int kb_latent_append(const void* rows, long long stride, const float* w, int width, float eps, void* pages,
+KB_API int kb_latent_append(const void* rows, long long stride, const float* w, int width, float eps, void* pages, int W,
                             const long long* slots, void* out, int N, int R, long long num_slots, int type, int* status,
                             cudaStream_t st) {
-    if (R % 8 || stride % 8 || N < 1) return 5;
+    if (R % 8 || stride % 8 || N < 1 || W < 8 || W % 8 || R % W) return 5;
     const dim3 grid((N + 7) / 8);
     if (type == 0)
         return kb_launch_dep(latent_append_kernel<bf16>, grid, dim3(256), 0, st, (const bf16*)rows, stride, w, width, eps,
-                             (bf16*)pages, slots, (bf16*)out, N, R, num_slots, status);
+                             (bf16*)pages, W, slots, (bf16*)out, N, R, num_slots, status);
     return kb_launch_dep(latent_append_kernel<float>, grid, dim3(256), 0, st, (const float*)rows, stride, w, width, eps,
-                         (float*)pages, slots, (float*)out, N, R, num_slots, status);
+                         (float*)pages, W, slots, (float*)out, N, R, num_slots, status);
 }
-KB_API int kb_latent_gather(const void* pages, const int* table, int max_pages, const int* cu, int B, void* out, int total, int R,
+KB_API int kb_latent_gather(const void* pages, int W, const int* table, int max_pages, const int* cu, int B, void* out, int total, int R,
                             int num_pages, int type, int* status, cudaStream_t st) {
-    if (R % 8 || total < 1 || B < 1) return 5;
+    if (R % 8 || total < 1 || B < 1 || W < 8 || W % 8 || R % W) return 5;
     const dim3 grid = flat_grid((long long)total * (R / 8), 256);
     if (type == 0)
-        return kb_launch_dep(latent_gather_kernel<bf16>, grid, dim3(256), 0, st, (const bf16*)pages, table, max_pages, cu, B,
+        return kb_launch_dep(latent_gather_kernel<bf16>, grid, dim3(256), 0, st, (const bf16*)pages, W, table, max_pages, cu, B,
                              (bf16*)out, total, R, num_pages, status);
-    return kb_launch_dep(latent_gather_kernel<float>, grid, dim3(256), 0, st, (const float*)pages, table, max_pages, cu, B,
+    return kb_launch_dep(latent_gather_kernel<float>, grid, dim3(256), 0, st, (const float*)pages, W, table, max_pages, cu, B,
                          (float*)out, total, R, num_pages, status);
 }
 // `at` null: y[N, D] is normalised as it is.  Otherwise y holds `ye_rows` expert output rows (see norm_add_kernel).

@@ -14,6 +14,7 @@
 // All waits are bounded (status word on timeout).
 #include <cuda.h>
 
+#include "act.cuh"
 #include "tc.cuh"
 
 namespace {
@@ -36,18 +37,6 @@ struct GroupedParams {
     int* status;
 };
 
-// erf to 1.5e-7 (Abramowitz & Stegun, Handbook of Mathematical Functions, 7.1.26); the result is rounded to bf16
-__device__ __forceinline__ float gelu_as(float z) {
-    const float x = fabsf(z) * 0.70710678f;
-    const float t = __fdividef(1.0f, fmaf(0.3275911f, x, 1.0f));
-    float p = fmaf(1.061405429f, t, -1.453152027f);
-    p = fmaf(p, t, 1.421413741f);
-    p = fmaf(p, t, -0.284496736f);
-    p = fmaf(p, t, 0.254829592f);
-    const float e = 1.0f - p * t * __expf(-x * x);
-    return 0.5f * z * (1.0f + copysignf(e, z));
-}
-
 template <int BN, int AM>
 __global__ void __launch_bounds__(192, 1)
 gemm_grouped_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ CUtensorMap tmB, const GroupedParams p) {
@@ -66,7 +55,7 @@ gemm_grouped_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_consta
     volatile int* abort_flag = reinterpret_cast<volatile int*>(tmem_slot + 1);
     int* tile_off = reinterpret_cast<int*>(smem + C_::RING + C_::SLACK + 256);   // [G + 1] row tiles before each group
 
-    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const int warp = __shfl_sync(0xffffffffu, threadIdx.x >> 5, 0), lane = threadIdx.x & 31;   // uniform, and known to be
     if (threadIdx.x == 0) {
         for (int s = 0; s < STAGES; ++s) {
             tc::mbar_init(&full[s], 1);
@@ -159,36 +148,32 @@ gemm_grouped_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_consta
             }
         }
     } else if (warp == 1) {
-        if (lane == 0) {
-            const uint32_t idesc = tc::instr_desc_f16(BM, BN, 1, 1, 0, 0);
-            int stage = 0, it = 0;
-            uint32_t phase = 0;
-            bool ok = true;
-            for (int tile = blockIdx.x; tile < num_tiles && ok; tile += gridDim.x, ++it) {
-                const int buf = it & 1;
-                if (!tc::mbar_wait(&acc_empty[buf], ((it >> 1) & 1) ^ 1, abort_flag)) {
-                    atomicMax(p.status, (int)KB_TIMEOUT_MMA);
-                    break;
-                }
+        // the whole warp walks the loop, one elected lane issues: the operands stay in uniform registers
+        const uint32_t idesc = tc::instr_desc_f16(BM, BN, 1, 1, 0, 0);
+        const tc::DescHalves da = tc::smem_desc_halves(smem_u32(sA), 16, 1024), db = tc::smem_desc_halves(smem_u32(sB), 16, 1024);
+        int stage = 0, it = 0;
+        uint32_t phase = 0;
+        bool ok = true;
+        for (int tile = blockIdx.x; tile < num_tiles && ok; tile += gridDim.x, ++it) {
+            const int buf = it & 1;
+            if (!tc::mbar_wait(&acc_empty[buf], ((it >> 1) & 1) ^ 1, abort_flag)) { ok = false; break; }
+            tc::tc_fence_after();
+            for (int kb = 0; kb < kblocks; ++kb) {
+                if (!tc::mbar_wait(&full[stage], phase, abort_flag)) { ok = false; break; }
                 tc::tc_fence_after();
-                for (int kb = 0; kb < kblocks; ++kb) {
-                    if (!tc::mbar_wait(&full[stage], phase, abort_flag)) {
-                        atomicMax(p.status, (int)KB_TIMEOUT_MMA);
-                        ok = false;
-                        break;
-                    }
-                    tc::tc_fence_after();
-                    const uint32_t a_addr = smem_u32(sA + stage * A_STAGE), b_addr = smem_u32(sB + stage * B_STAGE);
+                const uint32_t a_lo = da.lo + stage * (A_STAGE >> 4), b_lo = db.lo + stage * (B_STAGE >> 4);
+                if (tc::elect_one()) {
 #pragma unroll
                     for (int k = 0; k < BK / 16; ++k)
-                        tc::mma_f16(tmem_base + buf * BN, tc::smem_desc_sw128(a_addr + k * 32, 16, 1024),
-                                    tc::smem_desc_sw128(b_addr + k * 32, 16, 1024), idesc, (kb | k) != 0);
+                        tc::mma_f16_h(tmem_base + buf * BN, a_lo + (k * 32 >> 4), da.hi, b_lo + (k * 32 >> 4), db.hi, idesc, (kb | k) != 0);
                     tc::tc_commit(&empty[stage]);
-                    if (++stage == STAGES) { stage = 0; phase ^= 1; }
+                    if (kb + 1 == kblocks) tc::tc_commit(&acc_full[buf]);
                 }
-                if (ok) tc::tc_commit(&acc_full[buf]);
+                __syncwarp();
+                if (++stage == STAGES) { stage = 0; phase ^= 1; }
             }
         }
+        if (!ok && lane == 0) atomicMax(p.status, (int)KB_TIMEOUT_MMA);
     } else {
         const int quarter = warp & 3;
         int it = 0;
@@ -219,7 +204,7 @@ gemm_grouped_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_consta
 #pragma unroll
                             for (int i = 0; i < 8; ++i) {
                                 v[i] = __uint_as_float(acc[j + i]);
-                                if (p.act == 1) v[i] = gelu_as(v[i]);
+                                if (p.act == 1) v[i] = gelu_bf16(v[i]);
                                 else if (p.act == 2) v[i] = fmaxf(v[i], 0.f) * fmaxf(v[i], 0.f);
                             }
                             if (col + j < p.N) st8(dst + col + j, pack8(v));     // N is a multiple of 8

@@ -207,6 +207,10 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_consta
         tc::tmem_alloc(tmem_slot, 512);
         tc::tmem_relinquish();
     }
+    if (!COMM) {
+        kb_dep_trigger();
+        kb_dep_wait();
+    }
     tc::tc_fence_before();
     __syncthreads();
     tc::tc_fence_after();
@@ -562,7 +566,7 @@ static int launch_gemm(const void* A, const void* B, void* C, const void* Cin, i
     } else {
         GemmComm none;
         memset(&none, 0, sizeof(none));
-        gemm_tcgen05_kernel<false><<<grid, 192, SMEM_BYTES, st>>>(tmA, tmB, p, none);
+        return kb_launch_dep(gemm_tcgen05_kernel<false>, dim3(grid), dim3(192), (size_t)SMEM_BYTES, st, tmA, tmB, p, none);
     }
     return kb_launch_status();
 }

@@ -9,7 +9,7 @@ constexpr int PAGE = 16, TILE = 128, MAXE = 8;         // latent sizes up to TIL
 
 template <typename T>
 __global__ void __launch_bounds__(TILE)
-latent_attn_kernel(const T* __restrict__ q, const T* __restrict__ pages, const int* __restrict__ table, int max_pages, int num_pages,
+latent_attn_kernel(const T* __restrict__ q, const T* __restrict__ pages, int W, const int* __restrict__ table, int max_pages, int num_pages,
                    const int* __restrict__ ctx_lens, const int* __restrict__ cu, int B, T* __restrict__ out, int H, int R, float scale,
                    int* __restrict__ status) {
     extern __shared__ float la_smem[];
@@ -42,7 +42,7 @@ latent_attn_kernel(const T* __restrict__ q, const T* __restrict__ pages, const i
         const T* row = nullptr;
         if (k < keys) {
             const int page = table[(long long)b * max_pages + k / PAGE];
-            if (page >= 0 && page < num_pages) row = pages + ((long long)page * PAGE + k % PAGE) * R;
+            if (page >= 0 && page < num_pages) row = pages + (long long)page * PAGE * R + (k % PAGE) * W;
             else if (status) atomicMax(status, (int)KB_BAD_INDEX);
         }
         __syncthreads();                               // qs is there; the previous tile's ps and rowp are done with
@@ -52,7 +52,7 @@ latent_attn_kernel(const T* __restrict__ q, const T* __restrict__ pages, const i
             s = 0.f;
             for (int i = 0; i < R; i += 8) {
                 float c[8];
-                load8(row + i, c);
+                load8(row + (i / W) * PAGE * W + i % W, c);
 #pragma unroll
                 for (int j = 0; j < 8; ++j) s = fmaf(qs[i + j], c[j], s);
             }
@@ -79,9 +79,10 @@ latent_attn_kernel(const T* __restrict__ q, const T* __restrict__ pages, const i
         for (int i = 0; i < MAXE; ++i) {
             const int r = i * TILE + t;
             if (r >= R) break;
+            const int at = (r / W) * PAGE * W + r % W;
             float a = o[i] * f;
             for (int j = 0; j < nk; ++j)
-                if (rowp[j]) a = fmaf(ps[j], to_float(rowp[j][r]), a);
+                if (rowp[j]) a = fmaf(ps[j], to_float(rowp[j][at]), a);
             o[i] = a;
         }
     }
@@ -95,15 +96,15 @@ latent_attn_kernel(const T* __restrict__ q, const T* __restrict__ pages, const i
 
 }  // namespace
 
-// q, out: [N, H, R]; pages: [num_pages, 16, R]; cu null: row n is sequence n.
-KB_API int kb_latent_attn_plain(const void* q, const void* pages, const int* table, int max_pages, int num_pages, const int* ctx_lens,
+// q, out: [N, H, R]; pages: [num_pages, R / W, 16, W]; cu null: row n is sequence n.
+KB_API int kb_latent_attn_plain(const void* q, const void* pages, int W, const int* table, int max_pages, int num_pages, const int* ctx_lens,
                                 const int* cu, int B, void* out, int N, int H, int R, float scale, int type, int* status,
                                 cudaStream_t st) {
-    if (N < 1 || H < 1 || B < 1 || R % 8 || R > TILE * MAXE) return 5;
+    if (N < 1 || H < 1 || B < 1 || R % 8 || R > TILE * MAXE || W < 8 || W % 8 || R % W) return 5;
     const size_t smem = (size_t)(R + TILE) * 4 + TILE * sizeof(void*);
     if (type == 0)
-        return kb_launch_dep(latent_attn_kernel<bf16>, dim3(N, H), dim3(TILE), smem, st, (const bf16*)q, (const bf16*)pages, table,
+        return kb_launch_dep(latent_attn_kernel<bf16>, dim3(N, H), dim3(TILE), smem, st, (const bf16*)q, (const bf16*)pages, W, table,
                              max_pages, num_pages, ctx_lens, cu, B, (bf16*)out, H, R, scale, status);
-    return kb_launch_dep(latent_attn_kernel<float>, dim3(N, H), dim3(TILE), smem, st, (const float*)q, (const float*)pages, table,
+    return kb_launch_dep(latent_attn_kernel<float>, dim3(N, H), dim3(TILE), smem, st, (const float*)q, (const float*)pages, W, table,
                          max_pages, num_pages, ctx_lens, cu, B, (float*)out, H, R, scale, status);
 }

@@ -7,15 +7,21 @@
 //   S^T[128 tokens x HG]   = C[128 x R] . Q^T             A = the latent tile K-major,  B = queries  (both in shared memory)
 //   O^T[R x HG]           += C^T[R x 128] . P[128 x HG]   A = the same tile MN-major,   B = probabilities
 //
-// The tile is fetched by TMA page by page (16 rows x 64 columns each, 128-byte swizzle) into a ring of slots of 128
+// The cache keeps a page as blocks of 64 latent columns, [R / 64][16 tokens][64]: a block is 2 KB of contiguous memory.
+// The tile is fetched by TMA block by block (128-byte swizzle) into a ring of slots of 128
 // tokens x 128 latent columns; it stays there from the first product to the second.  S^T and O^T live in tensor memory.  A
 // thread of the softmax warps owns one token of the tile; a column's maximum is a warp reduction plus an exchange
 // through shared memory, refreshed lazily (O^T is rescaled only when a maximum grows by more than 2^8).
 //
 // Work: a unit is (sequence, group of HG query columns), its tiles are the 128-token tiles of the context that the
-// group sees.  All units' tiles form one line that is cut into equal pieces, one per CTA (persistent, one CTA per SM);
-// a unit whose tiles fall to several CTAs is put together by a merge kernel.  Piece g of unit u writes partial g + u.
-// Roles (192 threads): warp 0 = TMA, warp 1 = MMA issue and TMEM owner, warps 2-5 = softmax and output.
+// group sees; one CTA per SM.  With no more units than SMs every unit is cut into pieces of at most P tiles, P being the
+// smallest number for which there are no more pieces than SMs, and a CTA takes one piece (piece g writes partial g).
+// Otherwise all units' tiles form one line that is cut into equal parts, one per CTA; the part that CTA g has of unit u
+// writes partial g + u.  The pieces of a unit are put together by a merge kernel.
+// Roles (256 threads): warps 0 and 6 = TMA of the latents (one half of a slot each: a lane issues one page, and issuing
+// is what a single warp would be bound by), warp 7 = TMA of the queries, warp 1 = MMA issue and TMEM owner, warps 2-5 = softmax and output.
+// While the softmax of a tile runs, the tensor pipe already works on the scores of the next one, as far as the ring
+// holds it.
 // All waits are bounded (status word on timeout).
 #include <cuda.h>
 
@@ -28,6 +34,7 @@ constexpr int PAGE = 16, TT = 128, MAX_UNITS = 2048;
 constexpr int HALF = TT * 128;                     // 128 tokens x 64 latent columns: 16 KB
 constexpr int SLOT = 2 * HALF;                     // 128 x 128: 32 KB
 constexpr int MAX_SLOTS = 6;
+constexpr int THREADS = 256;
 constexpr float GROW = 8.0f;                       // log2 units
 constexpr float NONE = -1e30f;                     // running maximum of a column that has seen no key
 
@@ -41,7 +48,8 @@ struct LatentParams {
     float scale_log2;
     float* part_o;                 // [slots][HG][R]
     float* part_ml;                // [slots][HG][2]
-    int* unit_off;                 // [units + 1] for the merge kernel
+    int* unit_off;                 // for the merge kernel: [MAX_UNITS + 1] tiles before each unit, [MAX_UNITS + 1] pieces
+                                   // before each unit, P (0: the tiles are cut as one line)
     int slots_ring;
     int* status;
 };
@@ -69,7 +77,7 @@ struct Lay {
 };
 
 template <int HG>
-__global__ void __launch_bounds__(192, 1)
+__global__ void __launch_bounds__(THREADS, 1)
 latent_attn_sm100_kernel(const __grid_constant__ CUtensorMap tmC, const __grid_constant__ CUtensorMap tmQ, const LatentParams p) {
     extern __shared__ uint8_t smem_raw[];
     uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
@@ -94,11 +102,12 @@ latent_attn_sm100_kernel(const __grid_constant__ CUtensorMap tmC, const __grid_c
     uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(xch + 1);
     volatile int* abort_flag = reinterpret_cast<volatile int*>(tmem_slot + 1);
     int* uoff = reinterpret_cast<int*>(reinterpret_cast<uint8_t*>(bars) + 512);   // [units + 1] tiles before each unit
-    __shared__ int wsum[6];
+    __shared__ int wsum[THREADS / 32];
+    __shared__ int best_p;
 
-    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const int warp = __shfl_sync(0xffffffffu, threadIdx.x >> 5, 0), lane = threadIdx.x & 31;   // uniform, and known to be
     if (threadIdx.x == 0) {
-        for (int i = 0; i < MAX_SLOTS; ++i) { tc::mbar_init(full + i, 1); tc::mbar_init(empty + i, 1); }
+        for (int i = 0; i < MAX_SLOTS; ++i) { tc::mbar_init(full + i, 2); tc::mbar_init(empty + i, 1); }
         tc::mbar_init(q_full, 1);
         tc::mbar_init(q_empty, 1);
         tc::mbar_init(s_full, 1);
@@ -118,7 +127,7 @@ latent_attn_sm100_kernel(const __grid_constant__ CUtensorMap tmC, const __grid_c
     kb_dep_trigger();
     // ---- tiles of every unit and their prefix sums
     const int U = p.B * p.cgs;
-    const int per = (U + 191) / 192;
+    const int per = (U + THREADS - 1) / THREADS;
     {
         int mine = 0;
         for (int i = 0; i < per; ++i) {
@@ -148,50 +157,93 @@ latent_attn_sm100_kernel(const __grid_constant__ CUtensorMap tmC, const __grid_c
         }
         if (threadIdx.x == 0) uoff[0] = 0;
     }
+    if (threadIdx.x == 0) best_p = 0x7fffffff;
     tc::tc_fence_before();
     __syncthreads();
     tc::tc_fence_after();
-    if (blockIdx.x == 0)
-        for (int u = threadIdx.x; u <= U; u += 192) p.unit_off[u] = uoff[u];
     const uint32_t tmem = *tmem_slot;
-    const uint32_t tmem_s = tmem, tmem_o = tmem + 32;          // S^T: HG columns; O^T: HG columns per 128-row block
-    const long long T = uoff[U];
-    // pieces: no more than tiles, so that no piece is empty (the merge walks the pieces of a unit)
-    const int g = blockIdx.x, G = (int)(T < (long long)gridDim.x ? T : (long long)gridDim.x);
-    const int t_begin = g < G ? (int)(T * g / G) : 0, t_end = g < G ? (int)(T * (g + 1) / G) : 0;
-    int u0 = 0;
-    if (t_begin < t_end) {
-        int hi = U;
-        while (hi - u0 > 1) {
-            const int m = (u0 + hi) >> 1;
-            if (uoff[m] <= t_begin) u0 = m; else hi = m;
+    const uint32_t tmem_s = tmem, tmem_o = tmem + 64;          // S^T: two buffers of 32 columns; O^T: HG columns per 128-row block
+    const uint32_t T = (uint32_t)uoff[U];
+    const int g = blockIdx.x;
+    int t_begin = 0, t_end = 0, u0 = 0, P = 0;
+    if (U <= (int)gridDim.x) {
+        // smallest P with sum of ceil(tiles / P) <= CTAs: every warp tries another value
+        const int lo = max(1, (int)((T + gridDim.x - 1) / gridDim.x));
+        for (int base = lo;; base += THREADS / 32) {
+            int n = 0;
+            for (int u = lane; u < U; u += 32) n += (uoff[u + 1] - uoff[u] + base + warp - 1) / (base + warp);
+            n = __reduce_add_sync(0xffffffffu, n);
+            if (lane == 0 && n <= (int)gridDim.x) atomicMin(&best_p, base + warp);
+            __syncthreads();
+            if (best_p != 0x7fffffff || base > (int)T) break;  // P = T always does: one piece per unit
+            __syncthreads();
         }
+        P = best_p;
+        // this CTA's piece: walk the units' piece counts (every warp for itself, 32 units at a time)
+        int run = 0;
+        bool found = false;
+        for (int ub = 0; ub < U; ub += 32) {
+            const int u = ub + lane;
+            const int n = u < U ? (uoff[u + 1] - uoff[u] + P - 1) / P : 0;
+            int s = n;
+#pragma unroll
+            for (int o = 1; o < 32; o <<= 1) {
+                const int v = __shfl_up_sync(0xffffffffu, s, o);
+                if (lane >= o) s += v;
+            }
+            const int first = run + s - n;                     // pieces before unit u
+            if (g == 0 && warp == 0 && u < U) p.unit_off[MAX_UNITS + 1 + u] = first;
+            const uint32_t hit = __ballot_sync(0xffffffffu, g >= first && g < first + n);
+            if (hit) {
+                const int src = __ffs(hit) - 1;
+                u0 = ub + src;
+                t_begin = uoff[u0] + (g - __shfl_sync(0xffffffffu, first, src)) * P;
+                t_end = min(t_begin + P, uoff[u0 + 1]);
+                found = true;
+            }
+            run += __shfl_sync(0xffffffffu, s, 31);
+            if (found && g != 0) break;                        // CTA 0 writes all offsets for the merge
+        }
+        if (g == 0 && warp == 0 && lane == 0) p.unit_off[MAX_UNITS + 1 + U] = run;
+    } else {
+        // parts of the line: no more than tiles, so that none is empty (the merge walks the parts of a unit)
+        const int G = (int)(T < gridDim.x ? T : gridDim.x);
+        // (up to 2^24 tiles, in 32 bits: the launcher bounds the context)
+        t_begin = g < G ? (int)(T * g / G) : 0;
+        t_end = g < G ? (int)(T * (g + 1) / G) : 0;
+        if (t_begin < t_end) {
+            int hi = U;
+            while (hi - u0 > 1) {
+                const int m = (u0 + hi) >> 1;
+                if (uoff[m] <= t_begin) u0 = m; else hi = m;
+            }
+        }
+    }
+    if (g == 0) {
+        for (int u = threadIdx.x; u <= U; u += THREADS) p.unit_off[u] = uoff[u];
+        if (threadIdx.x == 0) p.unit_off[2 * (MAX_UNITS + 1)] = P;
     }
     // every role walks the same segments: (unit, tiles [a, e) of the unit)
 #define FOR_SEGMENTS                                                              \
     for (int u = u0, at = t_begin; at < t_end; at = min(t_end, uoff[u + 1]), ++u) \
         if (uoff[u + 1] > at)
 
-    if (warp == 0) {
-        // ------------------------------------------------------------ TMA: lanes 0-15 each bring one page of one half
-        const int pg = (lane >> 1) & 7, hf = lane & 1;
-        uint32_t n_slot = 0, n_q = 0;
+    if (warp == 0 || warp == 6) {
+        // ------------------------------------------------------------ TMA: lanes 0-7 each bring one page of this warp's half
+        const int pg = lane & 7, hf = warp == 6;
+        uint32_t n_slot = 0;
         bool ok = true;
         FOR_SEGMENTS {
             if (!ok) break;
             const int a = at - uoff[u], e = min(t_end, uoff[u + 1]) - uoff[u];
             const int b = u / p.cgs, cg = u % p.cgs;
             const int pages = (unit_len(p, b, cg, HG) + PAGE - 1) / PAGE;
-            if (!tc::mbar_wait(q_empty, (n_q & 1) ^ 1, abort_flag)) { ok = false; break; }
-            if (lane == 0) {
-                const int row = (p.cu ? p.cu[b] : b) * p.H + cg * HG;
-                tc::mbar_expect_tx(q_full, Lay<HG>::q_bytes(R));
-                for (int c = 0; c < R / 64; ++c) tc::tma_load_3d(sQ + c * HG * 128, &tmQ, q_full, c * 64, row, 0);
-            }
-            ++n_q;
+            const int* row = p.table + (long long)b * p.max_pages;
+            // pages behind the context repeat the last one: finite numbers that are masked out
+            int next = row[min(a * (TT / PAGE) + pg, pages - 1)];
             for (int t = a; t < e && ok; ++t) {
-                // pages behind the context repeat the last one: finite numbers that are masked out
-                int page = p.table[(long long)b * p.max_pages + min(t * (TT / PAGE) + pg, pages - 1)];
+                int page = next;
+                if (t + 1 < e) next = row[min((t + 1) * (TT / PAGE) + pg, pages - 1)];
                 if (page < 0 || page >= p.num_pages) {
                     atomicMax(p.status, (int)KB_BAD_INDEX);
                     page = 0;
@@ -199,10 +251,11 @@ latent_attn_sm100_kernel(const __grid_constant__ CUtensorMap tmC, const __grid_c
                 for (int k = 0; k < NB; ++k, ++n_slot) {
                     const int s = n_slot % NS;
                     if (!tc::mbar_wait(empty + s, ((n_slot / NS) & 1) ^ 1, abort_flag)) { ok = false; break; }
-                    if (lane == 0) tc::mbar_expect_tx(full + s, SLOT);
+                    if (lane == 0) tc::mbar_expect_tx(full + s, HALF);
                     __syncwarp();
-                    if (lane < 16)
-                        tc::tma_load_3d(ring + s * SLOT + hf * HALF + pg * PAGE * 128, &tmC, full + s, k * 128 + hf * 64, page * PAGE, 0);
+                    if (lane < 8)
+                        tc::tma_load_3d(ring + s * SLOT + hf * HALF + pg * PAGE * 128, &tmC, full + s, 0,
+                                        (page * (R / 64) + 2 * k + hf) * PAGE, 0);
                 }
             }
         }
@@ -211,48 +264,89 @@ latent_attn_sm100_kernel(const __grid_constant__ CUtensorMap tmC, const __grid_c
             const uint64_t t_0 = global_timer_ns();            // copies in flight land before the block can exit
             while (global_timer_ns() - t_0 < 2000000ull) {}
         }
-    } else if (warp == 1) {
-        // ------------------------------------------------------------ MMA issue (one thread)
+    } else if (warp == 7) {
+        // ------------------------------------------------------------ TMA of the queries
         if (lane == 0) {
-            const uint32_t id_s = tc::instr_desc_f16(128, HG, 1, 1, 0, 0), id_o = tc::instr_desc_f16(128, HG, 1, 1, 1, 0);
-            const uint32_t ring_a = smem_u32(ring), q_a = smem_u32(sQ), p_a = smem_u32(sP);
-            uint32_t n_slot = 0, n_q = 0, n_t = 0;
-            bool ok = true;
+            uint32_t n_q = 0;
             FOR_SEGMENTS {
-                if (!ok) break;
-                const int a = at - uoff[u], e = min(t_end, uoff[u + 1]) - uoff[u];
-                if (!tc::mbar_wait(q_full, n_q & 1, abort_flag)) { ok = false; break; }
+                const int b = u / p.cgs, cg = u % p.cgs;
+                if (!tc::mbar_wait(q_empty, (n_q & 1) ^ 1, abort_flag)) {
+                    atomicMax(p.status, (int)KB_TIMEOUT_TMA);
+                    break;
+                }
+                const int q0 = (p.cu ? p.cu[b] : b) * p.H + cg * HG;
+                tc::mbar_expect_tx(q_full, Lay<HG>::q_bytes(R));
+                for (int c = 0; c < R / 64; ++c) tc::tma_load_3d(sQ + c * HG * 128, &tmQ, q_full, c * 64, q0, 0);
                 ++n_q;
-                for (int t = a; t < e; ++t, ++n_t) {
-                    for (int k = 0; k < NB; ++k) {
-                        const uint32_t n = n_slot + k, s = n % NS;
-                        if (!tc::mbar_wait(full + s, (n / NS) & 1, abort_flag)) { ok = false; break; }
-                        tc::tc_fence_after();
+            }
+        }
+    } else if (warp == 1) {
+        // ------------------------------------------------------------ MMA issue
+        // The whole warp walks the loop and one elected lane issues: the operands of the products then stay in uniform
+        // registers.  (With one thread walking it, moving them there took longer than these small products.)
+        const uint32_t id_s = tc::instr_desc_f16(128, HG, 1, 1, 0, 0), id_o = tc::instr_desc_f16(128, HG, 1, 1, 1, 0);
+        // descriptors are stepped by adding to their low words: rebuilding them would cost more than the products
+        const tc::DescHalves ck = tc::smem_desc_halves(smem_u32(ring), 16, 1024);        // latent tile, K-major
+        const tc::DescHalves cm = tc::smem_desc_halves(smem_u32(ring), HALF, 1024);      // latent tile, MN-major
+        const tc::DescHalves dq = tc::smem_desc_halves(smem_u32(sQ), 16, 1024), dp = tc::smem_desc_halves(smem_u32(sP), 16, 1024);
+        uint32_t n_slot = 0, n_q = 0, n_t = 0;             // n_slot: ring uses before the current tile
+        bool ok = true;
+        // scores of one 128-column block of a latent tile: eight 16-wide steps, two halves of four
+        auto scores = [&](uint32_t s, int k, uint32_t buf) {
+            tc::tc_fence_after();
+            const uint32_t a_lo = ck.lo + s * (SLOT >> 4), b_lo = dq.lo + k * (2 * HG * 128 >> 4);
+            if (tc::elect_one()) {
 #pragma unroll
-                        for (int i = 0; i < 8; ++i) {          // eight 16-wide steps: two halves of four
-                            const uint32_t off = (i & 3) * 32;
-                            tc::mma_f16(tmem_s, tc::smem_desc_sw128(ring_a + s * SLOT + (i >> 2) * HALF + off, 16, 1024),
-                                        tc::smem_desc_sw128(q_a + (2 * k + (i >> 2)) * HG * 128 + off, 16, 1024), id_s, (k | i) != 0);
-                        }
-                    }
-                    if (!ok) break;
+                for (int i = 0; i < 8; ++i)
+                    tc::mma_f16_h(tmem_s + buf * 32, a_lo + (((i >> 2) * HALF + (i & 3) * 32) >> 4), ck.hi,
+                                  b_lo + (((i >> 2) * HG * 128 + (i & 3) * 32) >> 4), dq.hi, id_s, (k | i) != 0);
+            }
+            __syncwarp();
+        };
+        FOR_SEGMENTS {
+            if (!ok) break;
+            const int a = at - uoff[u], e = min(t_end, uoff[u + 1]) - uoff[u];
+            if (!tc::mbar_wait(q_full, n_q & 1, abort_flag)) { ok = false; break; }
+            ++n_q;
+            int early = 0;                                 // blocks of the current tile whose scores were issued before
+            for (int t = a; t < e; ++t, ++n_t) {
+                for (int k = early; k < NB; ++k) {
+                    const uint32_t n = n_slot + k, s = n % NS;
+                    if (!tc::mbar_wait(full + s, (n / NS) & 1, abort_flag)) { ok = false; break; }
+                    scores(s, k, n_t & 1);
+                }
+                if (!ok) break;
+                if (tc::elect_one()) {
                     tc::tc_commit(s_full);
                     if (t + 1 == e) tc::tc_commit(q_empty);
-                    if (!tc::mbar_wait(p_ready, n_t & 1, abort_flag)) { ok = false; break; }
-                    tc::tc_fence_after();
-                    for (int k = 0; k < NB; ++k, ++n_slot) {
-                        const uint32_t s = n_slot % NS;
-#pragma unroll
-                        for (int i = 0; i < 8; ++i)            // eight steps of 16 tokens
-                            tc::mma_f16(tmem_o + k * HG, tc::smem_desc_sw128(ring_a + s * SLOT + i * 2048, HALF, 1024),
-                                        tc::smem_desc_sw128(p_a + (i >> 2) * HG * 128 + (i & 3) * 32, 16, 1024), id_o, t > a || i > 0);
-                        tc::tc_commit(empty + s);
+                }
+                __syncwarp();
+                early = 0;
+                if (t + 1 < e) {
+                    // the next tile's blocks that have arrived in the slots this tile leaves free
+                    for (; early < NB && early < NS - NB; ++early) {
+                        const uint32_t n = n_slot + NB + early, s = n % NS;
+                        if (!__all_sync(0xffffffffu, tc::mbar_try_wait(full + s, (n / NS) & 1))) break;
+                        scores(s, early, (n_t + 1) & 1);
                     }
-                    if (t + 1 == e) tc::tc_commit(o_full);
+                }
+                if (!tc::mbar_wait(p_ready, n_t & 1, abort_flag)) { ok = false; break; }
+                tc::tc_fence_after();
+                for (int k = 0; k < NB; ++k, ++n_slot) {
+                    const uint32_t s = n_slot % NS, a_lo = cm.lo + s * (SLOT >> 4);
+                    if (tc::elect_one()) {
+#pragma unroll
+                        for (int i = 0; i < 8; ++i)        // eight steps of 16 tokens
+                            tc::mma_f16_h(tmem_o + k * HG, a_lo + (i * 2048 >> 4), cm.hi,
+                                          dp.lo + (((i >> 2) * HG * 128 + (i & 3) * 32) >> 4), dp.hi, id_o, (t > a || i > 0) ? 1u : 0u);
+                        tc::tc_commit(empty + s);
+                        if (k + 1 == NB && t + 1 == e) tc::tc_commit(o_full);
+                    }
+                    __syncwarp();
                 }
             }
-            if (!ok) atomicMax(p.status, (int)KB_TIMEOUT_MMA);
         }
+        if (!ok && lane == 0) atomicMax(p.status, (int)KB_TIMEOUT_MMA);
     } else {
         // ------------------------------------------------------------ softmax and output: one token (latent row) per thread
         const int quarter = warp & 3, tk = quarter * 32 + lane;
@@ -286,8 +380,9 @@ latent_attn_sm100_kernel(const __grid_constant__ CUtensorMap tmC, const __grid_c
                 if (!tc::mbar_wait(s_full, n_t & 1, abort_flag)) { ok = false; break; }
                 tc::tc_fence_after();
                 float x[HG];
-                if constexpr (HG == 32) tc::tmem_ld32(tmem_s + lb, reinterpret_cast<uint32_t*>(x));
-                else tc::tmem_ld16(tmem_s + lb, reinterpret_cast<uint32_t*>(x));
+                const uint32_t ts = tmem_s + (n_t & 1) * 32 + lb;
+                if constexpr (HG == 32) tc::tmem_ld32(ts, reinterpret_cast<uint32_t*>(x));
+                else tc::tmem_ld16(ts, reinterpret_cast<uint32_t*>(x));
                 tc::tmem_ld_wait();
                 const int pos = t * TT + tk;
                 float mine = NONE;
@@ -316,6 +411,10 @@ latent_attn_sm100_kernel(const __grid_constant__ CUtensorMap tmC, const __grid_c
                     my_f[lane] = f;
                 }
                 __syncwarp();
+                // read in one go: between the stores below every read would wait for the one before
+                float mv[HG];
+#pragma unroll
+                for (int j = 0; j < HG; j += 4) *reinterpret_cast<float4*>(mv + j) = *reinterpret_cast<const float4*>(my_m + j);
                 // the four warps see the same maxima and take the same branch; S^T of this tile is complete, so the
                 // products into O^T that were issued before it are too
                 if (__any_sync(0xffffffffu, grow)) {
@@ -339,7 +438,7 @@ latent_attn_sm100_kernel(const __grid_constant__ CUtensorMap tmC, const __grid_c
                 const int chunk = (tk & 63) >> 3;
 #pragma unroll
                 for (int j = 0; j < HG; ++j) {
-                    const float e2 = exp2f(x[j] - my_m[j]);
+                    const float e2 = exp2f(x[j] - mv[j]);
                     l[j] += e2;
                     *reinterpret_cast<bf16*>(prow + j * 128 + ((chunk ^ (j & 7)) << 4)) = __float2bfloat16(e2);
                 }
@@ -358,7 +457,7 @@ latent_attn_sm100_kernel(const __grid_constant__ CUtensorMap tmC, const __grid_c
             }
             if (lane < HG) lred[quarter * HG + lane] = lt;
             if (!exchange()) { ok = false; break; }
-            const long long slot = (long long)g + u;
+            const long long slot = P ? (long long)g : (long long)g + u;
             if (quarter == 0 && lane < HG) {
                 float* ml = p.part_ml + (slot * HG + lane) * 2;
                 ml[0] = m_col;
@@ -399,28 +498,37 @@ latent_merge_kernel(const float* __restrict__ part_o, const float* __restrict__ 
     kb_dep_wait();
     const int u = blockIdx.x, j = blockIdx.y, b = u / cgs, col = (u % cgs) * HG + j;
     const int q0 = cu ? cu[b] : b, nq = cu ? cu[b + 1] - q0 : 1;
-    if (col >= nq * H) return;
+    const int P = unit_off[2 * (MAX_UNITS + 1)];
     const long long T = unit_off[units];
-    const int G = (int)(T < (long long)ctas ? T : (long long)ctas);
-    const int lo = unit_off[u], hi = unit_off[u + 1];
+    const int lo = unit_off[u], hi = unit_off[u + 1], first = unit_off[MAX_UNITS + 1 + u];
+    if (col >= nq * H) return;
     bf16* dst = out + ((long long)q0 * H + col) * R;
-    const int g0 = hi > lo ? (int)(((lo + 1ll) * G - 1) / T) : 0, g1 = hi > lo ? (int)(((long long)hi * G - 1) / T) : -1;
-    float M = -INFINITY;
-    for (int g = g0; g <= g1; ++g) M = fmaxf(M, part_ml[((long long)(g + u) * HG + j) * 2]);
-    float den = 0.f;
-    for (int g = g0; g <= g1; ++g) {
-        const float* ml = part_ml + ((long long)(g + u) * HG + j) * 2;
-        den += exp2f(ml[0] - M) * ml[1];
+    int s0, n;                                         // first partial of the unit, how many
+    if (P) {
+        s0 = first;
+        n = (hi - lo + P - 1) / P;
+    } else {
+        const int G = (int)(T < (long long)ctas ? T : (long long)ctas);
+        const int g0 = hi > lo ? (int)(((lo + 1ll) * G - 1) / T) : 0;
+        s0 = g0 + u;
+        n = hi > lo ? (int)(((long long)hi * G - 1) / T) - g0 + 1 : 0;
     }
-    const float inv = den > 0.f ? 1.0f / den : 0.f;
+    const float2* ml = reinterpret_cast<const float2*>(part_ml) + (long long)s0 * HG + j;
+    const float* po = part_o + ((long long)s0 * HG + j) * R;
+    float M = -INFINITY;
+    for (int i = 0; i < n; ++i) M = fmaxf(M, ml[(long long)i * HG].x);
     for (int r = threadIdx.x * 4; r < R; r += 512) {
         float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
-        for (int g = g0; g <= g1; ++g) {
-            const long long s = (long long)(g + u) * HG + j;
-            const float w = exp2f(part_ml[s * 2] - M);
-            const float4 v = *reinterpret_cast<const float4*>(part_o + s * R + r);
+        float den = 0.f;
+#pragma unroll 4
+        for (int i = 0; i < n; ++i) {
+            const float2 x = ml[(long long)i * HG];
+            const float4 v = *reinterpret_cast<const float4*>(po + (long long)i * HG * R + r);
+            const float w = exp2f(x.x - M);
+            den += w * x.y;
             acc.x += w * v.x; acc.y += w * v.y; acc.z += w * v.z; acc.w += w * v.w;
         }
+        const float inv = den > 0.f ? 1.0f / den : 0.f;
         const __nv_bfloat162 o0 = __floats2bfloat162_rn(acc.x * inv, acc.y * inv), o1 = __floats2bfloat162_rn(acc.z * inv, acc.w * inv);
         *reinterpret_cast<uint2*>(dst + r) = make_uint2(*reinterpret_cast<const uint32_t*>(&o0), *reinterpret_cast<const uint32_t*>(&o1));
     }
@@ -469,12 +577,12 @@ int launch(const void* q, const void* pages, const LatentParams& p0, bf16* out, 
         *set = true;
     }
     CUtensorMap tmC, tmQ;
-    int r = make_tmap(&tmC, pages, p.R, (long long)p.num_pages * PAGE, PAGE);
+    int r = make_tmap(&tmC, pages, 64, (long long)p.num_pages * (p.R / 64) * PAGE, PAGE);
     if (r) return r;
     r = make_tmap(&tmQ, q, p.R, p.q_rows, HG);
     if (r) return r;
     const size_t smem = (size_t)p.slots_ring * SLOT + Lay<HG>::fixed(p.R);
-    r = kb_launch_dep(latent_attn_sm100_kernel<HG>, dim3(grid), dim3(192), smem, st, tmC, tmQ, p);
+    r = kb_launch_dep(latent_attn_sm100_kernel<HG>, dim3(grid), dim3(THREADS), smem, st, tmC, tmQ, p);
     if (r) return r;
     return kb_launch_dep(latent_merge_kernel, dim3(p.B * p.cgs, HG), dim3(128), 0, st, (const float*)p.part_o, (const float*)p.part_ml,
                          (const int*)p.unit_off, p.cu, out, p.B * p.cgs, p.cgs, HG, p.H, p.R, grid);
@@ -503,7 +611,7 @@ KB_API int kb_latent_ok(int B, int max_q, int H, int R) {
     if (R < 128 || R % 128 || units > MAX_UNITS) return 0;
     return (hg == 16 ? ring_slots<16>(R) : ring_slots<32>(R)) >= R / 128;
 }
-// q, out: [tokens, H, R] bf16; pages: [num_pages, 16, R] bf16; unit_off: workspace of MAX_UNITS + 1 ints.
+// q, out: [tokens, H, R] bf16; pages: [num_pages, R / 64, 16, 64] bf16; unit_off: workspace of 2 * MAX_UNITS + 3 ints.
 KB_API int kb_latent_attn(const void* q, const void* pages, const int* table, int max_pages, int num_pages, const int* ctx_lens,
                           const int* cu, int B, int max_q, int tokens, int H, int R, float scale, float* part_o, float* part_ml,
                           int* unit_off, void* out, int* status, cudaStream_t st) {
@@ -520,6 +628,7 @@ KB_API int kb_latent_attn(const void* q, const void* pages, const int* table, in
     p.part_o = part_o; p.part_ml = part_ml; p.unit_off = unit_off;
     p.slots_ring = 0;
     p.status = status;
+    if ((long long)B * p.cgs * ((max_pages + 7) / 8) > (1 << 24)) return 12;
     const int grid = sm_count();
     return hg == 16 ? launch<16>(q, pages, p, (bf16*)out, grid, st) : launch<32>(q, pages, p, (bf16*)out, grid, st);
 }

@@ -1,200 +1,239 @@
 // Mixture-of-experts routing: router scores, group-limited top-k, grouping of the (token, choice) pairs by expert
-// and the gather of their rows.  The expert products are in gemm_grouped_sm100.cu (bf16) and gemm_f32.cu, the weighted
-// sum of the experts' outputs is part of the norm kernel in block.cu.  Compiled without fast-math.
+// and the gather of their rows.  Few tokens (decoding): one kernel scores and selects, one groups and gathers, each
+// block finding its places in the grouping from all the choices.  Many tokens: the scores are a matrix product, the
+// selection counts the experts' choices with atomics, the gather turns the counts into places.  The order of an
+// expert's rows does not matter: rows are independent, and a token's outputs are summed in the order of its choices.
+// The expert products are in gemm_grouped_sm100.cu (bf16) and gemm_f32.cu, the weighted sum of the experts' outputs
+// is part of the norm kernel in block.cu.  Compiled without fast-math.
 #include "vec.cuh"
 
 namespace {
 
-// logits[n, e] = h[n, :] . w[e, :], one warp per product; for few tokens (decode)
-template <typename T>
-__global__ void __launch_bounds__(256)
-router_dot_kernel(const T* __restrict__ h, const T* __restrict__ w, float* __restrict__ logits, int E, int D) {
-    kb_dep_trigger();
-    kb_dep_wait();
-    const int e = blockIdx.y * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
-    if (e >= E) return;
-    const T* a = h + (long long)blockIdx.x * D;
-    const T* b = w + (long long)e * D;
-    float acc = 0.f;
-    for (int c = lane * 8; c < D; c += 256) {
-        float x[8], y[8];
-        load8(a + c, x);
-        load8(b + c, y);
-#pragma unroll
-        for (int j = 0; j < 8; ++j) acc += x[j] * y[j];
-    }
-    acc = warp_sum(acc);
-    if (lane == 0) logits[(long long)blockIdx.x * E + e] = acc;
+constexpr int MAX_EXPERTS = 1024;
+
+struct Select {
+    int E, top, groups, keep, gated;
+    float scale;
+    int* ids;                      // [N, top]
+    float* wts;                    // [N, top]
+    float* gate;                   // [N]
+    int* counts;                   // [E] choices per expert, null: not counted
+    int* rank;                     // [N, top] place of the choice among its expert's
+};
+
+// Index of the largest value over the warp (ties: smallest index); every lane brings its best (key 0: none).  Keys are
+// the bits of non-negative floats plus one, which compare like the floats.
+__device__ __forceinline__ int warp_argmax(uint32_t key, int idx) {
+    const uint32_t m = __reduce_max_sync(0xffffffffu, key);
+    return (int)__reduce_min_sync(0xffffffffu, key == m && m != 0u ? (uint32_t)idx : 0x7fffffffu);
 }
 
-// Largest value of v (ties: smallest index) over the warp; returns the index, all lanes agree.
-__device__ __forceinline__ int warp_argmax(float& v, int idx) {
-#pragma unroll
-    for (int o = 16; o > 0; o >>= 1) {
-        const float ov = __shfl_xor_sync(0xffffffffu, v, o);
-        const int oi = __shfl_xor_sync(0xffffffffu, idx, o);
-        if (ov > v || (ov == v && oi < idx)) { v = ov; idx = oi; }
-    }
-    return idx;
-}
-
-constexpr int SEL_WARPS = 4;
-// One warp per token.  Shared memory per warp: E scores and `groups` group scores.
-__global__ void __launch_bounds__(SEL_WARPS * 32)
-moe_select_kernel(const float* __restrict__ logits, int ld, int N, int E, int top, float scale, int groups, int keep, int gated,
-                  int* __restrict__ ids, float* __restrict__ wts, float* __restrict__ gate) {
-    extern __shared__ float sel_smem[];
-    kb_dep_trigger();
-    kb_dep_wait();
-    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
-    const int n = blockIdx.x * SEL_WARPS + warp;
-    if (n >= N) return;
-    float* s = sel_smem + warp * (E + groups);
-    float* gs = s + E;
-    const float* z = logits + (long long)n * ld;
+// One warp selects for token n; z: E logits (and the gate's behind them); s: E + groups floats of shared memory.
+__device__ __forceinline__ void select_experts(const float* z, float* s, const Select& c, int n, int lane) {
+    float* gs = s + c.E;
     float m = -INFINITY;
-    for (int e = lane; e < E; e += 32) m = fmaxf(m, z[e]);
+    for (int e = lane; e < c.E; e += 32) m = fmaxf(m, z[e]);
     m = warp_max(m);
     float sum = 0.f;
-    for (int e = lane; e < E; e += 32) {
+    for (int e = lane; e < c.E; e += 32) {
         const float p = expf(z[e] - m);
         s[e] = p;
         sum += p;
     }
     sum = warp_sum(sum);
     __syncwarp();
-    for (int e = lane; e < E; e += 32) s[e] = s[e] / sum;
-    __syncwarp();
-    if (keep < groups) {
-        const int size = E / groups;
-        for (int g = lane; g < groups; g += 32) {
-            float b = -INFINITY;
+    const int size = c.E / c.groups;
+    const bool limited = c.keep < c.groups;
+    if (limited) {
+        for (int g = lane; g < c.groups; g += 32) {
+            float b = 0.f;
             for (int e = g * size; e < (g + 1) * size; ++e) b = fmaxf(b, s[e]);
             gs[g] = b;
         }
         __syncwarp();
-        for (int k = 0; k < keep; ++k) {               // a kept group's score becomes +inf
-            float b = -INFINITY;
+        for (int k = 0; k < c.keep; ++k) {             // a kept group's score becomes -1
+            uint32_t b = 0u;
             int bi = 0x7fffffff;
-            for (int g = lane; g < groups; g += 32)
-                if (gs[g] != INFINITY && gs[g] > b) { b = gs[g]; bi = g; }
+            for (int g = lane; g < c.groups; g += 32)
+                if (gs[g] >= 0.f && __float_as_uint(gs[g]) + 1u > b) { b = __float_as_uint(gs[g]) + 1u; bi = g; }
             bi = warp_argmax(b, bi);
-            __syncwarp();
-            if (lane == 0 && bi < groups) gs[bi] = INFINITY;
+            if (lane == 0 && bi < c.groups) gs[bi] = -1.f;
             __syncwarp();
         }
-        for (int e = lane; e < E; e += 32)
-            if (gs[e / size] != INFINITY) s[e] = -1.f;
+        for (int e = lane; e < c.E; e += 32)
+            if (gs[e / size] >= 0.f) s[e] = -1.f;
         __syncwarp();
     }
-    for (int k = 0; k < top; ++k) {
-        float b = -INFINITY;
+    for (int k = 0; k < c.top; ++k) {
+        uint32_t b = 0u;
         int bi = 0x7fffffff;
-        for (int e = lane; e < E; e += 32)
-            if (s[e] > b) { b = s[e]; bi = e; }
+        for (int e = lane; e < c.E; e += 32)
+            if (s[e] >= 0.f && __float_as_uint(s[e]) + 1u > b) { b = __float_as_uint(s[e]) + 1u; bi = e; }
         bi = warp_argmax(b, bi);
-        if (bi >= E) bi = 0;                           // only with non-finite scores
+        if (bi >= c.E) bi = 0;                         // only with non-finite scores
         __syncwarp();
         if (lane == 0) {
-            ids[(long long)n * top + k] = bi;
-            wts[(long long)n * top + k] = b * scale;
-            s[bi] = -2.f;
+            const long long i = (long long)n * c.top + k;
+            c.ids[i] = bi;
+            c.wts[i] = s[bi] / sum * c.scale;
+            if (c.counts) c.rank[i] = atomicAdd(&c.counts[bi], 1);
+            s[bi] = -1.f;
         }
         __syncwarp();
     }
-    if (gated && lane == 0) gate[n] = 1.0f / (1.0f + expf(-z[E]));
+    if (c.gated && lane == 0) c.gate[n] = 1.0f / (1.0f + expf(-z[c.E]));
 }
 
-// Groups the A = N * top choices by expert: at[i] = row of choice i, tok[row] = its token, offsets[E + 1].
-// One block; counts and cursors live in shared memory.
-constexpr int IDX_THREADS = 1024, IDX_UNROLL = 8, MAX_EXPERTS = 1024;
-__global__ void __launch_bounds__(IDX_THREADS)
-moe_index_kernel(const int* __restrict__ ids, int A, int top, int E, int* __restrict__ at, int* __restrict__ tok,
-                 int* __restrict__ offsets) {
-    __shared__ int cnt[MAX_EXPERTS], off[MAX_EXPERTS];
+// Few tokens: one block per token, a warp per expert at a time, then the first warp selects.
+template <typename T>
+__global__ void __launch_bounds__(512)
+route_token_kernel(const T* __restrict__ h, const T* __restrict__ w, int rows, int D, const Select c) {
+    extern __shared__ float rt_smem[];
+    float* x = rt_smem;                                // [D]
+    float* z = x + D;                                  // [rows]
     kb_dep_trigger();
     kb_dep_wait();
-    for (int e = threadIdx.x; e < E; e += IDX_THREADS) cnt[e] = 0;
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+    for (int i = threadIdx.x * 8; i < D; i += 512 * 8) load8(h + (long long)blockIdx.x * D + i, x + i);
     __syncthreads();
-    for (int i0 = threadIdx.x; i0 < A; i0 += IDX_THREADS * IDX_UNROLL) {
-        int e[IDX_UNROLL];
+    for (int e = warp; e < rows; e += 16) {
+        const T* b = w + (long long)e * D;
+        float acc = 0.f;
+#pragma unroll 4
+        for (int i = lane * 8; i < D; i += 256) {
+            float y[8];
+            load8(b + i, y);
 #pragma unroll
-        for (int u = 0; u < IDX_UNROLL; ++u) {
-            const int i = i0 + u * IDX_THREADS;
-            e[u] = i < A ? ids[i] : -1;
+            for (int j = 0; j < 8; ++j) acc += x[i + j] * y[j];
         }
-#pragma unroll
-        for (int u = 0; u < IDX_UNROLL; ++u)
-            if (e[u] >= 0) at[i0 + u * IDX_THREADS] = atomicAdd(&cnt[e[u]], 1);
+        acc = warp_sum(acc);
+        if (lane == 0) z[e] = acc;
     }
     __syncthreads();
-    // exclusive prefix sum over the experts (E <= 1024 = block size)
-    if (threadIdx.x < MAX_EXPERTS) off[threadIdx.x] = threadIdx.x < (unsigned)E ? cnt[threadIdx.x] : 0;
+    if (warp == 0) select_experts(z, z + rows, c, blockIdx.x, lane);
+}
+
+// Many tokens: one warp per token on the logits of a matrix product.
+constexpr int SEL_WARPS = 4;
+__global__ void __launch_bounds__(SEL_WARPS * 32)
+moe_select_kernel(const float* __restrict__ logits, int ld, int N, const Select c) {
+    extern __shared__ float sel_smem[];
+    kb_dep_trigger();
+    kb_dep_wait();
+    const int warp = threadIdx.x >> 5, n = blockIdx.x * SEL_WARPS + warp;
+    if (n < N) select_experts(logits + (long long)n * ld, sel_smem + warp * (c.E + c.groups), c, n, threadIdx.x & 31);
+}
+
+// One block per token: the places at[n, k] of its choices in the grouping, offsets[E + 1], and copies of the token's row
+// to these places.  FEW: counts and ranks are found here from all choices (`A` of them); otherwise the selection has left
+// them in `counts` and `at`.
+template <bool FEW>
+__global__ void __launch_bounds__(256)
+moe_gather_kernel(const uint4* __restrict__ h, const int* __restrict__ ids, const int* __restrict__ counts, int* __restrict__ at,
+                  int* __restrict__ offsets, uint4* __restrict__ out, int A, int top, int E, int vecs, int* __restrict__ status) {
+    extern __shared__ int mg_smem[];
+    int* off = mg_smem;                                // [E] counts, then exclusive prefix sums
+    int* place = off + E;                              // [top]
+    __shared__ int wsum[8];
+    kb_dep_trigger();
+    kb_dep_wait();
+    const int n = blockIdx.x, lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+    for (int e = threadIdx.x; e < E; e += 256) off[e] = FEW ? 0 : counts[e];
+    for (int k = threadIdx.x; k < top; k += 256) place[k] = FEW ? 0 : at[(long long)n * top + k];
     __syncthreads();
-    for (int d = 1; d < E; d <<= 1) {
-        const int v = (int)threadIdx.x >= d ? off[threadIdx.x - d] : 0;
-        __syncthreads();
-        off[threadIdx.x] += v;
+    if (FEW) {
+        for (int i = threadIdx.x; i < A; i += 256) {
+            const int e = ids[i];
+            atomicAdd(&off[e], 1);
+            // choices in front of this token's, and its own earlier ones (a token's choices differ)
+            if (i < n * top)
+                for (int k = 0; k < top; ++k)
+                    if (ids[n * top + k] == e) atomicAdd(&place[k], 1);
+        }
         __syncthreads();
     }
-    if (threadIdx.x < (unsigned)E) offsets[threadIdx.x + 1] = off[threadIdx.x];
-    if (threadIdx.x == 0) offsets[0] = 0;
-    for (int i0 = threadIdx.x; i0 < A; i0 += IDX_THREADS * IDX_UNROLL) {
-        int e[IDX_UNROLL], r[IDX_UNROLL];
+    // exclusive prefix sums: a run of experts per thread
+    const int per = (E + 255) / 256;
+    int mine = 0;
+    for (int i = 0; i < per; ++i) {
+        const int e = threadIdx.x * per + i;
+        if (e < E) mine += off[e];
+    }
+    int s = mine;
 #pragma unroll
-        for (int u = 0; u < IDX_UNROLL; ++u) {
-            const int i = i0 + u * IDX_THREADS;
-            e[u] = i < A ? ids[i] : -1;
-            r[u] = i < A ? at[i] : 0;
+    for (int o = 1; o < 32; o <<= 1) {
+        const int v = __shfl_up_sync(0xffffffffu, s, o);
+        if (lane >= o) s += v;
+    }
+    if (lane == 31) wsum[warp] = s;
+    __syncthreads();
+    int run = s - mine;
+    for (int v = 0; v < warp; ++v) run += wsum[v];
+    for (int i = 0; i < per; ++i) {
+        const int e = threadIdx.x * per + i;
+        if (e < E) {
+            const int cnt = off[e];
+            off[e] = run;
+            run += cnt;
+            if (n == 0) offsets[e + 1] = run;
         }
-#pragma unroll
-        for (int u = 0; u < IDX_UNROLL; ++u)
-            if (e[u] >= 0) {
-                const int i = i0 + u * IDX_THREADS;
-                const int row = off[e[u]] - cnt[e[u]] + r[u];
-                at[i] = row;
-                tok[row] = i / top;
-            }
+    }
+    if (n == 0 && threadIdx.x == 0) offsets[0] = 0;
+    __syncthreads();
+    for (int k = threadIdx.x; k < top; k += 256) {
+        int row = off[ids[(long long)n * top + k]] + place[k];
+        if (row < 0 || row >= A) {
+            if (status) atomicMax(status, (int)KB_BAD_INDEX);
+            row = -1;
+        }
+        place[k] = row;
+        at[(long long)n * top + k] = row;
+    }
+    __syncthreads();
+    for (int i = threadIdx.x; i < vecs; i += 256) {
+        const uint4 v = h[(long long)n * vecs + i];
+        for (int k = 0; k < top; ++k)
+            if (place[k] >= 0) out[(long long)place[k] * vecs + i] = v;
     }
 }
 
-// out[r] = h[tok[r]], 16 bytes per thread and step
-__global__ void moe_gather_kernel(const uint4* __restrict__ h, const int* __restrict__ tok, uint4* __restrict__ out, int A, int vecs) {
-    kb_dep_trigger();
-    kb_dep_wait();
-    const long long total = (long long)A * vecs;
-    for (long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x; i < total; i += (long long)gridDim.x * blockDim.x) {
-        const int r = (int)(i / vecs), c = (int)(i % vecs);
-        out[i] = h[(long long)tok[r] * vecs + c];
-    }
+inline bool select_ok(int N, const Select& c) {
+    return N >= 1 && c.E >= 1 && c.E <= MAX_EXPERTS && c.groups >= 1 && c.E % c.groups == 0 && c.keep >= 1 && c.keep <= c.groups &&
+           c.top >= 1 && c.top <= c.keep * (c.E / c.groups);
 }
 
 }  // namespace
 
-KB_API int kb_router_dot(const void* h, const void* w, float* logits, int N, int E, int D, int type, cudaStream_t st) {
-    if (D % 8 || N < 1 || E < 1) return 5;
-    const dim3 grid(N, (E + 7) / 8);
-    if (type == 0) return kb_launch_dep(router_dot_kernel<bf16>, grid, dim3(256), 0, st, (const bf16*)h, (const bf16*)w, logits, E, D);
-    return kb_launch_dep(router_dot_kernel<float>, grid, dim3(256), 0, st, (const float*)h, (const float*)w, logits, E, D);
+// Router and selection for few tokens.  w: [E (+ 1 with `gated`), D]; ids, wts: [N, top]; gate: [N] or null.
+KB_API int kb_moe_route_few(const void* h, const void* w, int N, int E, int D, int top, float scale, int groups, int keep, int gated,
+                            int* ids, float* wts, float* gate, int type, cudaStream_t st) {
+    const Select c{E, top, groups, keep, gated, scale, ids, wts, gate, nullptr, nullptr};
+    const int rows = E + (gated ? 1 : 0);
+    const size_t smem = (size_t)(D + rows + E + groups) * 4;
+    if (D % 8 || !select_ok(N, c) || smem > 48 * 1024) return 5;
+    if (type == 0)
+        return kb_launch_dep(route_token_kernel<bf16>, dim3(N), dim3(512), smem, st, (const bf16*)h, (const bf16*)w, rows, D, c);
+    return kb_launch_dep(route_token_kernel<float>, dim3(N), dim3(512), smem, st, (const float*)h, (const float*)w, rows, D, c);
 }
-// logits[N, ld]: E expert logits per token and, with `gated`, the gate's logit behind them.
+// Selection on logits[N, ld] (E expert logits and, with `gated`, the gate's).  counts[E] (zero) and rank[N, top] receive
+// what kb_moe_group needs.
 KB_API int kb_moe_select(const float* logits, int ld, int N, int E, int top, float scale, int groups, int keep, int gated, int* ids,
-                         float* wts, float* gate, cudaStream_t st) {
-    if (N < 1 || E < 1 || E > MAX_EXPERTS || groups < 1 || E % groups || keep < 1 || keep > groups || top < 1 ||
-        top > keep * (E / groups) || ld < E + (gated ? 1 : 0))
-        return 5;
+                         float* wts, float* gate, int* counts, int* rank, cudaStream_t st) {
+    const Select c{E, top, groups, keep, gated, scale, ids, wts, gate, counts, rank};
+    if (!select_ok(N, c) || ld < E + (gated ? 1 : 0)) return 5;
     return kb_launch_dep(moe_select_kernel, dim3((N + SEL_WARPS - 1) / SEL_WARPS), dim3(SEL_WARPS * 32),
-                         (size_t)SEL_WARPS * (E + groups) * 4, st, logits, ld, N, E, top, scale, groups, keep, gated, ids, wts, gate);
+                         (size_t)SEL_WARPS * (E + groups) * 4, st, logits, ld, N, c);
 }
-// at / tok: [N * top]; offsets: [E + 1]; rows: gathered copies of h's rows, [N * top, row_bytes]
-KB_API int kb_moe_group(const void* h, const int* ids, int N, int top, int E, int row_bytes, int* at, int* tok, int* offsets,
-                        void* rows, cudaStream_t st) {
+// Groups the N * top choices by expert: at[N, top] (with counts: holds the ranks on entry), offsets[E + 1], rows
+// [N * top, row_bytes] = copies of h's rows.  counts null: everything is found from ids (few tokens).
+KB_API int kb_moe_group(const void* h, const int* ids, const int* counts, int N, int top, int E, int row_bytes, int* at, int* offsets,
+                        void* rows, int* status, cudaStream_t st) {
     const long long A = (long long)N * top;
-    if (N < 1 || top < 1 || E < 1 || E > MAX_EXPERTS || row_bytes % 16 || A > 0x7fffffff) return 5;
-    const int r = kb_launch_dep(moe_index_kernel, dim3(1), dim3(IDX_THREADS), 0, st, ids, (int)A, top, E, at, tok, offsets);
-    if (r) return r;
-    long long blocks = (A * (row_bytes / 16) + 255) / 256;
-    if (blocks > 148 * 16) blocks = 148 * 16;
-    return kb_launch_dep(moe_gather_kernel, dim3((unsigned)blocks), dim3(256), 0, st, (const uint4*)h, (const int*)tok, (uint4*)rows,
-                         (int)A, row_bytes / 16);
+    if (N < 1 || top < 1 || E < 1 || E > MAX_EXPERTS || top > E || row_bytes % 16 || A > 0x7fffffff) return 5;
+    const size_t smem = (size_t)(E + top) * 4;
+    if (counts)
+        return kb_launch_dep(moe_gather_kernel<false>, dim3(N), dim3(256), smem, st, (const uint4*)h, ids, counts, at, offsets,
+                             (uint4*)rows, (int)A, top, E, row_bytes / 16, status);
+    return kb_launch_dep(moe_gather_kernel<true>, dim3(N), dim3(256), smem, st, (const uint4*)h, ids, counts, at, offsets, (uint4*)rows,
+                         (int)A, top, E, row_bytes / 16, status);
 }

@@ -686,6 +686,9 @@ class CudaOps(TorchOps):
     def latent_multiple(self, dtype):
         return 128 if dtype == torch.bfloat16 else 8       # 128-row blocks of the tensor-core kernel
 
+    def latent_block(self, dtype, R):
+        return 64 if dtype == torch.bfloat16 else R        # a block of a page is one TMA copy
+
     def embed_pairs(self, ids, prev, table, bigram, consts):
         N, D = ids.numel(), table.shape[1]
         x = torch.empty(N, D, device=table.device, dtype=torch.float32)
@@ -697,14 +700,14 @@ class CudaOps(TorchOps):
     def latent_append(self, rows, w, width, eps, pages, slots):
         N, R = rows.shape
         out = torch.empty(N, R, device=rows.device, dtype=rows.dtype)
-        self._call("kb_latent_append", _p(rows), _LL(rows.stride(0)), _p(w), _I(width), _F(eps), _p(pages), _p(slots), _p(out),
-                   _I(N), _I(R), _LL(pages.shape[0] * pages.shape[1]), _I(_TYPE[rows.dtype]), _p(self.status(rows.device)), _st())
+        self._call("kb_latent_append", _p(rows), _LL(rows.stride(0)), _p(w), _I(width), _F(eps), _p(pages), _I(pages.shape[3]), _p(slots), _p(out),
+                   _I(N), _I(R), _LL(pages.shape[0] * pages.shape[2]), _I(_TYPE[rows.dtype]), _p(self.status(rows.device)), _st())
         return out
 
     def latent_gather(self, pages, page_table, cu_context, total):
-        R = pages.shape[-1]
+        R = pages.shape[1] * pages.shape[3]
         out = torch.empty(total, R, device=pages.device, dtype=pages.dtype)
-        self._call("kb_latent_gather", _p(pages), _p(page_table), _I(page_table.shape[1]), _p(cu_context), _I(page_table.shape[0]),
+        self._call("kb_latent_gather", _p(pages), _I(pages.shape[3]), _p(page_table), _I(page_table.shape[1]), _p(cu_context), _I(page_table.shape[0]),
                    _p(out), _I(total), _I(R), _I(pages.shape[0]), _I(_TYPE[pages.dtype]), _p(self.status(pages.device)), _st())
         return out
 
@@ -717,18 +720,18 @@ class CudaOps(TorchOps):
         out = torch.empty(N, H, R, device=dev, dtype=q.dtype)
         if not q.is_contiguous():
             raise KernelError("latent queries must be dense")
-        if q.dtype == torch.bfloat16 and self.lib.kb_latent_ok(_I(B), _I(max_q), _I(H), _I(R)):
+        if q.dtype == torch.bfloat16 and pages.shape[3] == 64 and self.lib.kb_latent_ok(_I(B), _I(max_q), _I(H), _I(R)):
             cols = self.lib.kb_latent_cols(_I(max_q), _I(H))
             slots = self.lib.kb_latent_partials(_I(B), _I(max_q), _I(H))
             part_o = torch.empty(slots * cols * R, device=dev, dtype=torch.float32)
             part_ml = torch.empty(slots * cols * 2, device=dev, dtype=torch.float32)
-            unit_off = torch.empty(2049, device=dev, dtype=torch.int32)
+            unit_off = torch.empty(2 * 2048 + 3, device=dev, dtype=torch.int32)
             self._call("kb_latent_attn", _p(q), _p(pages), _p(page_table), _I(page_table.shape[1]), _I(pages.shape[0]), _p(ctx_lens),
                        _p(cu_seqlens), _I(B), _I(max_q), _I(N), _I(H), _I(R), _F(scale), _p(part_o), _p(part_ml), _p(unit_off),
                        _p(out), _p(self.status(dev)), _st())
             self.launches += 1
             return out
-        self._call("kb_latent_attn_plain", _p(q), _p(pages), _p(page_table), _I(page_table.shape[1]), _I(pages.shape[0]), _p(ctx_lens),
+        self._call("kb_latent_attn_plain", _p(q), _p(pages), _I(pages.shape[3]), _p(page_table), _I(page_table.shape[1]), _I(pages.shape[0]), _p(ctx_lens),
                    _p(cu_seqlens), _I(B), _p(out), _I(N), _I(H), _I(R), _F(scale), _I(_TYPE[q.dtype]), _p(self.status(dev)), _st())
         return out
 
@@ -780,37 +783,51 @@ class CudaOps(TorchOps):
                    _F(eps), _I(_TYPE[dtype]), _p(self.status(x.device)), _st())
         return out
 
+    moe_few = 256           # tokens up to which routing and grouping are one small kernel each
+
     def moe_route(self, h, router, experts, top, scale, groups, keep):
+        """Returns ``(ids, weights, gate, plan)``; ``plan`` (counts per expert, ranks) is for :meth:`moe_experts`."""
         N, D = h.shape
         E = router.shape[0]
         dev = h.device
-        logits = torch.empty(N, E, device=dev, dtype=torch.float32)
-        if N <= 256:
-            self._call("kb_router_dot", _p(h), _p(router), _p(logits), _I(N), _I(E), _I(D), _I(_TYPE[h.dtype]), _st())
-        else:
-            self.gemm_nt(h, router, out=logits)
         gated = E > experts
         ids = torch.empty(N, top, device=dev, dtype=torch.int32)
         wts = torch.empty(N, top, device=dev, dtype=torch.float32)
         gate = torch.empty(N, device=dev, dtype=torch.float32) if gated else None
-        self._call("kb_moe_select", _p(logits), _I(E), _I(N), _I(experts), _I(top), _F(scale), _I(groups), _I(keep), _I(int(gated)),
-                   _p(ids), _p(wts), _p(gate), _st())
-        return ids, wts, gate
+        if N <= self.moe_few and (D + 2 * E + groups) * 4 <= 48 * 1024:
+            self._call("kb_moe_route_few", _p(h), _p(router), _I(N), _I(experts), _I(D), _I(top), _F(scale), _I(groups), _I(keep),
+                       _I(int(gated)), _p(ids), _p(wts), _p(gate), _I(_TYPE[h.dtype]), _st())
+            return ids, wts, gate, None
+        # one zeroed buffer: the logits (the product adds its K parts up in it) and the experts' counts
+        ld = (E + 3) // 4 * 4
+        buf = torch.zeros(N * ld + experts, device=dev, dtype=torch.float32)
+        logits, counts = buf[: N * ld].view(N, ld)[:, :E], buf[N * ld:].view(torch.int32)
+        if h.dtype == torch.float32:
+            self._gemm(h, router, N, E, D, False, False, out=logits)
+        else:
+            split = max(1, min(4, 148 // ((N + 127) // 128), (D + 63) // 128))
+            self._call("kb_gemm", _p(h), _p(router), _p(logits), _p(None), _I(N), _I(E), _I(D), _I(1), _LL(h.stride(0)),
+                       _LL(router.stride(0)), _LL(ld), _LL(0), _LL(0), _LL(0), _LL(0), _LL(0), _I(0), _I(0), _I(1), _I(1), _I(2),
+                       _F(1.0), _F(0.0), _p(self.status(dev)), _I(0), _I(split), _st())
+        rank = torch.empty(N, top, device=dev, dtype=torch.int32)
+        self._call("kb_moe_select", _p(logits), _I(ld), _I(N), _I(experts), _I(top), _F(scale), _I(groups), _I(keep), _I(int(gated)),
+                   _p(ids), _p(wts), _p(gate), _p(counts), _p(rank), _st())
+        return ids, wts, gate, (counts, rank)
 
-    def moe_experts(self, h, ids, up, down, kind):
+    def moe_experts(self, h, ids, up, down, kind, plan=None):
+        rows, offsets, at = self._moe_group(h, ids, up.shape[0], plan)
+        return self._grouped(self._grouped(rows, up, offsets, kind), down, offsets, None), at
+
+    def _moe_group(self, h, ids, E, plan):
         N, top = ids.shape
-        E, ff, D = up.shape
-        A = N * top
+        D = h.shape[1]
         dev = h.device
-        at = torch.empty(N, top, device=dev, dtype=torch.int32)
-        tok = torch.empty(A, device=dev, dtype=torch.int32)
+        counts, at = plan if plan is not None else (None, torch.empty(N, top, device=dev, dtype=torch.int32))
         offsets = torch.empty(E + 1, device=dev, dtype=torch.int32)
-        rows = torch.empty(A, D, device=dev, dtype=h.dtype)
-        self._call("kb_moe_group", _p(h), _p(ids), _I(N), _I(top), _I(E), _I(D * h.element_size()), _p(at), _p(tok), _p(offsets),
-                   _p(rows), _st())
-        self.launches += 1
-        u = self._grouped(rows, up, offsets, kind)
-        return self._grouped(u, down, offsets, None), at
+        rows = torch.empty(N * top, D, device=dev, dtype=h.dtype)
+        self._call("kb_moe_group", _p(h), _p(ids), _p(counts), _I(N), _I(top), _I(E), _I(D * h.element_size()), _p(at), _p(offsets),
+                   _p(rows), _p(self.status(dev)), _st())
+        return rows, offsets, at
 
     def _grouped(self, rows, w, offsets, kind):
         A, K = rows.shape

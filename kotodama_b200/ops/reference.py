@@ -657,6 +657,16 @@ class TorchOps:
         """What the cached latent's size is padded to."""
         return 8
 
+    def latent_block(self, dtype: torch.dtype, R: int) -> int:
+        """Columns of the latent that the cache keeps together: pages are ``[R / W, 16 tokens, W]``."""
+        return R
+
+    @staticmethod
+    def latent_rows(pages, page_ids, n):
+        """The first ``n`` cached latents of the given pages, ``[n, R]``."""
+        t = pages[page_ids.long()]                                      # [p, R / W, 16, W]
+        return t.transpose(1, 2).reshape(t.shape[0] * 16, -1)[:n]
+
     def embed_pairs(self, ids, prev, table, bigram, consts):
         """``x = table[id] (+ bigram[row])`` with ``row = (prev * mul_prev + id * mul_cur) mod buckets``, or row
         ``buckets`` where ``prev < 0``; ``consts = (buckets, mul_prev, mul_cur)``.  Returns ``x`` fp32 and its rounding to the table's dtype."""
@@ -668,18 +678,18 @@ class TorchOps:
         return x, x.to(table.dtype, copy=True)
 
     def latent_append(self, rows, w, width, eps, pages, slots):
-        """RMS norm of ``rows[N, R]`` (mean over ``width``), written to cache slots ``slots`` of ``pages[P, 16, R]``
+        """RMS norm of ``rows[N, R]`` (mean over ``width``), written to cache slots ``slots`` of ``pages[P, R / W, 16, W]``
         (negative: nowhere) and returned."""
         r = _f(rows)
         c = (r * torch.rsqrt(r.pow(2).sum(-1, keepdim=True) / width + eps) * w).to(pages.dtype)
         ok = slots >= 0
-        pages[slots[ok] // 16, slots[ok] % 16] = c[ok]
+        pages[slots[ok] // 16, :, slots[ok] % 16] = c[ok].view(-1, pages.shape[1], pages.shape[3])
         return c
 
     def latent_gather(self, pages, page_table, cu_context, total):
         """The cached latents of every sequence, packed: ``[total, R]``."""
         cu = cu_context.tolist()
-        return torch.cat([pages[page_table[b, : (n + 15) // 16].long()].flatten(0, 1)[:n]
+        return torch.cat([self.latent_rows(pages, page_table[b, : (n + 15) // 16], n)
                           for b, n in enumerate(j - i for i, j in zip(cu, cu[1:]))])
 
     def latent_attention(self, q, pages, page_table, ctx_lens, cu_seqlens, max_q, max_ctx, scale):
@@ -690,7 +700,7 @@ class TorchOps:
         cu = cu_seqlens.tolist() if cu_seqlens is not None else list(range(N + 1))
         for b, n in enumerate(ctx_lens.tolist()):
             lo, hi = cu[b], cu[b + 1]
-            c = _f(pages[page_table[b, : (n + 15) // 16].long()].flatten(0, 1)[:n])
+            c = _f(self.latent_rows(pages, page_table[b, : (n + 15) // 16], n))
             s = torch.einsum("nhr,tr->nht", _f(q[lo:hi]), c) * scale
             seen = torch.arange(n, device=q.device)[None, :] <= torch.arange(n - (hi - lo), n, device=q.device)[:, None]
             p = torch.softmax(s.masked_fill(~seen[:, None, :], float("-inf")), -1)
@@ -732,7 +742,8 @@ class TorchOps:
 
     def moe_route(self, h, router, experts, top, scale, groups, keep):
         """Softmax router with group-limited top-k.  ``router[E (+ 1), D]``: an extra row is the shared expert's gate.
-        Returns expert ids ``[N, top]`` int32, weights ``[N, top]`` fp32 (score * scale) and the gate's sigmoid ``[N]`` or None."""
+        Returns expert ids ``[N, top]`` int32, weights ``[N, top]`` fp32 (score * scale), the gate's sigmoid ``[N]`` or None, and what the
+        back end wants handed on to :meth:`moe_experts`."""
         z = _f(h) @ _f(router).t()
         s = torch.softmax(z[:, :experts], -1)
         elig = s
@@ -741,9 +752,9 @@ class TorchOps:
             ok = torch.zeros(s.shape[0], groups, dtype=torch.bool, device=s.device).scatter_(1, best, True)
             elig = s.masked_fill(~ok.repeat_interleave(experts // groups, 1), -1.0)
         w, ids = elig.topk(top, -1)
-        return ids.to(torch.int32), w * scale, torch.sigmoid(z[:, experts]) if router.shape[0] > experts else None
+        return ids.to(torch.int32), w * scale, torch.sigmoid(z[:, experts]) if router.shape[0] > experts else None, None
 
-    def moe_experts(self, h, ids, up, down, kind):
+    def moe_experts(self, h, ids, up, down, kind, plan=None):
         """Every token through its chosen experts (``up[E, ff, D]``, ``down[E, D, ff]``).  Returns the outputs as rows
         grouped by expert, and ``at[N, top]``: the row of each (token, choice)."""
         flat = ids.flatten().long()

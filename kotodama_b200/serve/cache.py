@@ -45,9 +45,9 @@ class PagedKVCache(PagePool):
 
 
 class PagedLatentCache(PagePool):
-    """One latent row per token and layer (``[pages, 16, width]``; the layers' widths may differ): the attention
-    reads the same row as key and as value."""
+    """One latent row per token and layer (the layers' widths may differ): the attention reads the same row as key and as
+    value.  A page is ``[width / block, 16, block]``: ``block`` columns of its 16 tokens are contiguous."""
 
-    def __init__(self, widths: Sequence[int], num_pages: int, device: torch.device, dtype: torch.dtype) -> None:
+    def __init__(self, widths: Sequence[int], blocks: Sequence[int], num_pages: int, device: torch.device, dtype: torch.dtype) -> None:
         super().__init__(num_pages)
-        self.c = [torch.zeros(num_pages, PAGE, w, device=device, dtype=dtype) for w in widths]
+        self.c = [torch.zeros(num_pages, w // k, PAGE, k, device=device, dtype=dtype) for w, k in zip(widths, blocks)]

@@ -215,7 +215,8 @@ class LatentRunner:
         return out
 
     def make_cache(self, pages: int) -> PagedLatentCache:
-        self.cache = PagedLatentCache([lw["R"] for lw in self.layers], pages, self.device, self.dtype)
+        widths = [lw["R"] for lw in self.layers]
+        self.cache = PagedLatentCache(widths, [self.ops.latent_block(self.dtype, w) for w in widths], pages, self.device, self.dtype)
         return self.cache
 
     def _attention(self, h: torch.Tensor, lw: dict, pages: torch.Tensor, b: Batch) -> torch.Tensor:
@@ -238,8 +239,8 @@ class LatentRunner:
 
     def _experts(self, x: torch.Tensor, h: torch.Tensor, lw: dict) -> torch.Tensor:
         ops, f = self.ops, lw["mlp"]
-        ids, wts, gate = ops.moe_route(h, lw["router"], f.experts, f.top, f.scale, f.groups, f.keep)
-        ye, at = ops.moe_experts(h, ids, lw["eup"], lw["edown"], "gelu")
+        ids, wts, gate, plan = ops.moe_route(h, lw["router"], f.experts, f.top, f.scale, f.groups, f.keep)
+        ye, at = ops.moe_experts(h, ids, lw["eup"], lw["edown"], "gelu", plan)
         ys = None
         if f.shared_ff:
             ys = ops.gemm_nt(ops.activate(ops.gemm_nt(h, lw["sup"]), "gelu"), lw["sdown"])

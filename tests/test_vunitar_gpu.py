@@ -69,7 +69,7 @@ def test_latent_attention_against_fp32(H, R, lens, news):
     g = torch.Generator().manual_seed(H)
     mp = max((c + 15) // 16 for c in lens) + 1
     P = len(lens) * mp + 3
-    pages = torch.randn(P, 16, R, generator=g).bfloat16().cuda()
+    pages = torch.randn(P, R // 64, 16, 64, generator=g).bfloat16().cuda()
     table = torch.randperm(P, generator=g)[: len(lens) * mp].int().view(len(lens), mp).contiguous().cuda()
     cu = torch.tensor([0] + list(torch.tensor(news).cumsum(0)), dtype=torch.int32).cuda()
     q = torch.randn(sum(news), H, R, generator=g).bfloat16().cuda()

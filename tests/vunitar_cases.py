@@ -200,12 +200,12 @@ def check_generation(name, device, dtype):
 
 
 # ---------------------------------------------------------------------------------- mechanisms alone
-def pages_for(rows, page_ids):
+def pages_for(rows, page_ids, block):
     """Cache pages holding ``rows`` in the given page order."""
     n, R = rows.shape
-    pages = torch.zeros(max(page_ids) + 1, 16, R, dtype=rows.dtype, device=rows.device)
+    pages = torch.zeros(max(page_ids) + 1, R // block, 16, block, dtype=rows.dtype, device=rows.device)
     for i in range(n):
-        pages[page_ids[i // 16], i % 16] = rows[i]
+        pages[page_ids[i // 16], :, i % 16] = rows[i].view(R // block, block)
     return pages
 
 
@@ -216,7 +216,8 @@ def check_far_keys(ops, device, dtype, R=128, H=3, ctx=700):
     c = torch.randn(ctx, R, generator=g)
     c = c / c.norm(dim=-1, keepdim=True)
     ids = torch.randperm((ctx + 15) // 16 + 3, generator=g).tolist()[: (ctx + 15) // 16]
-    pages = pages_for(c.to(dtype), ids).to(device)
+    pages = pages_for(c.to(dtype), ids, 64 if device == "cuda" and dtype == torch.bfloat16 else R).to(device)
+    crows = c.to(dtype).float()
     table = torch.tensor([ids], dtype=torch.int32, device=device)
     tol = 0.02 if dtype == torch.bfloat16 else 1e-5
     spots = [0, 1, 14, 15, 16, 17, 126, 127, 128, 129, 255, 256, 383, 384, 511, 512, 640, ctx - 2, ctx - 1]
@@ -229,8 +230,8 @@ def check_far_keys(ops, device, dtype, R=128, H=3, ctx=700):
                                        n, ctx, 1.0).float().cpu()
             for i in range(n):
                 last = ctx - n + i
-                s = (q[i].float().cpu() @ pages_rows(pages, ids, ctx).float().cpu().t())[:, : last + 1]
-                want = torch.softmax(s, -1) @ pages_rows(pages, ids, ctx).float().cpu()[: last + 1]
+                s = (q[i].float().cpu() @ crows.t())[:, : last + 1]
+                want = torch.softmax(s, -1) @ crows[: last + 1]
                 assert float((out[i] - want).abs().max()) < tol, (n, i, mark)
                 for h, m in enumerate(mark):
                     seen = float(out[i, h] @ c[m]) > 0.9
@@ -248,10 +249,6 @@ def check_far_keys(ops, device, dtype, R=128, H=3, ctx=700):
             last = torch.arange(ctx - n, ctx)
             dot = torch.einsum("nhd,hd->nh", out, kd[m].float().cpu())
             assert ((dot > 0.9) == (m <= last)[:, None]).all(), (n, m)
-
-
-def pages_rows(pages, ids, n):
-    return pages[torch.tensor(ids, device=pages.device)].flatten(0, 1)[:n]
 
 
 def check_ops(ops, device, dtype):
@@ -278,7 +275,7 @@ def check_ops(ops, device, dtype):
     ids = [3, 0]
     slots = torch.tensor([ids[i // 16] * 16 + i % 16 for i in range(n)])
     slots[5] = -1
-    pages = torch.zeros(5, 16, Rp, dtype=dtype, device=device)
+    pages = torch.zeros(5, Rp // 8, 16, 8, dtype=dtype, device=device)
     got = ops.latent_append(dev(pad(raw.to(dtype), Rp)), dev(pad(w, Rp)), R, 1e-3, pages, dev(slots))
     want = oracle.rms(raw.to(dtype).double(), w.double(), 1e-3)
     assert close(got[:, :R], want)
@@ -320,14 +317,14 @@ def check_experts(ops, device, dtype, N=37):
         router = rnd(E + int(shared), D).to(dtype)
         r = dict(top=top, scale=1.3, groups=dict(count=groups[0], keep=groups[1]))
         up, down = (rnd(E, ff, D) * D ** -0.5).to(dtype), (rnd(E, D, ff) * ff ** -0.5).to(dtype)
-        ids, wts, gate = ops.moe_route(h.to(device), router.to(device), E, top, 1.3, *groups)
+        ids, wts, gate, plan = ops.moe_route(h.to(device), router.to(device), E, top, 1.3, *groups)
         picks = oracle.route(h.double(), router[:E].double(), r)
         for i, p in enumerate(picks):
             assert ids[i].tolist() == [e for e, _ in p], (E, i)
             assert torch.allclose(wts[i].double().cpu(), torch.stack([s for _, s in p]), rtol=2e-5)
         if shared:
             assert torch.allclose(gate.double().cpu(), torch.sigmoid(h.double() @ router[E].double()), rtol=1e-4, atol=1e-6)
-        ye, at = ops.moe_experts(h.to(device), ids, up.to(device), down.to(device), "gelu")
+        ye, at = ops.moe_experts(h.to(device), ids, up.to(device), down.to(device), "gelu", plan)
         ys = rnd(N, D).to(dtype) if shared else None
         x0, gn = rnd(N, D), rnd(D)
         x = x0.clone().to(device)
