@@ -64,12 +64,14 @@ def llama_config(z: dict) -> ModelConfig:
 
 
 def timed(calls: list, reps: int = 5) -> float:
-    """Mean device time of one call in ms: the calls (over different buffers) captured in one graph, replayed."""
+    """Mean device time of one call in ms: the calls (over different buffers) captured in one graph, replayed.  The
+    decode kernels of both models are launched as in serving, as programmatic dependents of one another."""
     for c in calls[:2]:
         c()
     torch.cuda.synchronize()
     g = torch.cuda.CUDAGraph()
-    with torch.cuda.graph(g):
+    from kotodama_b200.ops import get_ops
+    with torch.cuda.graph(g), get_ops("cuda").dependent_launch(True):
         keep = [c() for c in calls]
     for _ in range(2):
         g.replay()

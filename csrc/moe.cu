@@ -1,7 +1,7 @@
 // Mixture-of-experts routing: router scores, group-limited top-k, grouping of the (token, choice) pairs by expert
-// and the gather of their rows.  Few tokens (decoding): one kernel scores and selects, one groups and gathers, each
-// block finding its places in the grouping from all the choices.  Many tokens: the scores are a matrix product, the
-// selection counts the experts' choices with atomics, the gather turns the counts into places.  The order of an
+// and the gather of their rows.  Few tokens (decoding): the scores are dot products, and each block of the gather finds
+// its places in the grouping from all the choices.  Many tokens: the scores are a matrix product, the selection
+// counts the experts' choices with atomics, the gather turns the counts into places.  The order of an
 // expert's rows does not matter: rows are independent, and a token's outputs are summed in the order of its choices.
 // The expert products are in gemm_grouped_sm100.cu (bf16) and gemm_f32.cu, the weighted sum of the experts' outputs
 // is part of the norm kernel in block.cu.  Compiled without fast-math.
@@ -10,6 +10,7 @@
 namespace {
 
 constexpr int MAX_EXPERTS = 1024;
+constexpr int COUNT_STRIDE = 32;   // ints between the experts' counters: one cache line each, or the atomics queue up
 
 struct Select {
     int E, top, groups, keep, gated;
@@ -17,7 +18,7 @@ struct Select {
     int* ids;                      // [N, top]
     float* wts;                    // [N, top]
     float* gate;                   // [N]
-    int* counts;                   // [E] choices per expert, null: not counted
+    int* counts;                   // [E * COUNT_STRIDE] choices per expert, null: not counted
     int* rank;                     // [N, top] place of the choice among its expert's
 };
 
@@ -64,56 +65,76 @@ __device__ __forceinline__ void select_experts(const float* z, float* s, const S
             if (gs[e / size] >= 0.f) s[e] = -1.f;
         __syncwarp();
     }
-    for (int k = 0; k < c.top; ++k) {
-        uint32_t b = 0u;
-        int bi = 0x7fffffff;
-        for (int e = lane; e < c.E; e += 32)
-            if (s[e] >= 0.f && __float_as_uint(s[e]) + 1u > b) { b = __float_as_uint(s[e]) + 1u; bi = e; }
-        bi = warp_argmax(b, bi);
-        if (bi >= c.E) bi = 0;                         // only with non-finite scores
-        __syncwarp();
-        if (lane == 0) {
-            const long long i = (long long)n * c.top + k;
-            c.ids[i] = bi;
-            c.wts[i] = s[bi] / sum * c.scale;
-            if (c.counts) c.rank[i] = atomicAdd(&c.counts[bi], 1);
-            s[bi] = -1.f;
+    const float norm = c.scale / sum;
+    for (int k0 = 0; k0 < c.top; k0 += 32) {           // lane k keeps choice k: stores and atomics of 32 choices go together
+        const int n_k = min(32, c.top - k0);
+        int mine = 0;
+        float score = 0.f;
+        for (int k = 0; k < n_k; ++k) {
+            uint32_t b = 0u;
+            int bi = 0x7fffffff;
+            for (int e = lane; e < c.E; e += 32)
+                if (s[e] >= 0.f && __float_as_uint(s[e]) + 1u > b) { b = __float_as_uint(s[e]) + 1u; bi = e; }
+            bi = warp_argmax(b, bi);
+            if (bi >= c.E) bi = 0;                     // only with non-finite scores
+            if (lane == k) {
+                mine = bi;
+                score = s[bi];
+            }
+            __syncwarp();
+            if (lane == 0) s[bi] = -1.f;
+            __syncwarp();
         }
-        __syncwarp();
+        if (lane < n_k) {
+            const long long i = (long long)n * c.top + k0 + lane;
+            c.ids[i] = mine;
+            c.wts[i] = score * norm;
+            if (c.counts) c.rank[i] = atomicAdd(&c.counts[mine * COUNT_STRIDE], 1);
+        }
     }
     if (c.gated && lane == 0) c.gate[n] = 1.0f / (1.0f + expf(-z[c.E]));
 }
 
-// Few tokens: one block per token, a warp per expert at a time, then the first warp selects.
+// Few tokens: logits[n, e] = h[n, :] . w[e, :].  A block takes eight tokens (their rows in shared memory) and eight
+// experts, one per warp, so that a row of w is read once for eight tokens.
+constexpr int DOT_TOKENS = 8;
 template <typename T>
-__global__ void __launch_bounds__(512)
-route_token_kernel(const T* __restrict__ h, const T* __restrict__ w, int rows, int D, const Select c) {
-    extern __shared__ float rt_smem[];
-    float* x = rt_smem;                                // [D]
-    float* z = x + D;                                  // [rows]
+__global__ void __launch_bounds__(256)
+router_dot_kernel(const T* __restrict__ h, const T* __restrict__ w, float* __restrict__ logits, int N, int E, int D) {
+    extern __shared__ __align__(16) uint8_t rd_smem[];
+    T* x = reinterpret_cast<T*>(rd_smem);              // [DOT_TOKENS][D]
     kb_dep_trigger();
+    const int n0 = blockIdx.x * DOT_TOKENS, e = blockIdx.y * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
     kb_dep_wait();
-    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
-    for (int i = threadIdx.x * 8; i < D; i += 512 * 8) load8(h + (long long)blockIdx.x * D + i, x + i);
-    __syncthreads();
-    for (int e = warp; e < rows; e += 16) {
-        const T* b = w + (long long)e * D;
-        float acc = 0.f;
-#pragma unroll 4
-        for (int i = lane * 8; i < D; i += 256) {
-            float y[8];
-            load8(b + i, y);
-#pragma unroll
-            for (int j = 0; j < 8; ++j) acc += x[i + j] * y[j];
-        }
-        acc = warp_sum(acc);
-        if (lane == 0) z[e] = acc;
+    constexpr int V = 16 / sizeof(T);
+    for (int i = threadIdx.x; i < DOT_TOKENS * D / V; i += 256) {
+        const int t = min(n0 + i / (D / V), N - 1);
+        reinterpret_cast<uint4*>(x)[i] = reinterpret_cast<const uint4*>(h + (long long)t * D)[i % (D / V)];
     }
     __syncthreads();
-    if (warp == 0) select_experts(z, z + rows, c, blockIdx.x, lane);
+    if (e >= E) return;
+    const T* b = w + (long long)e * D;
+    float acc[DOT_TOKENS] = {};
+#pragma unroll 4
+    for (int i = lane * 8; i < D; i += 256) {
+        float y[8];
+        load8(b + i, y);
+#pragma unroll
+        for (int t = 0; t < DOT_TOKENS; ++t) {
+            float v[8];
+            load8(x + t * D + i, v);
+#pragma unroll
+            for (int j = 0; j < 8; ++j) acc[t] += v[j] * y[j];
+        }
+    }
+#pragma unroll
+    for (int t = 0; t < DOT_TOKENS; ++t) {
+        acc[t] = warp_sum(acc[t]);
+        if (lane == t && n0 + t < N) logits[(long long)(n0 + t) * E + e] = acc[t];
+    }
 }
 
-// Many tokens: one warp per token on the logits of a matrix product.
+// One warp per token.
 constexpr int SEL_WARPS = 4;
 __global__ void __launch_bounds__(SEL_WARPS * 32)
 moe_select_kernel(const float* __restrict__ logits, int ld, int N, const Select c) {
@@ -138,7 +159,7 @@ moe_gather_kernel(const uint4* __restrict__ h, const int* __restrict__ ids, cons
     kb_dep_trigger();
     kb_dep_wait();
     const int n = blockIdx.x, lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
-    for (int e = threadIdx.x; e < E; e += 256) off[e] = FEW ? 0 : counts[e];
+    for (int e = threadIdx.x; e < E; e += 256) off[e] = FEW ? 0 : counts[e * COUNT_STRIDE];
     for (int k = threadIdx.x; k < top; k += 256) place[k] = FEW ? 0 : at[(long long)n * top + k];
     __syncthreads();
     if (FEW) {
@@ -204,19 +225,26 @@ inline bool select_ok(int N, const Select& c) {
 
 }  // namespace
 
-// Router and selection for few tokens.  w: [E (+ 1 with `gated`), D]; ids, wts: [N, top]; gate: [N] or null.
-KB_API int kb_moe_route_few(const void* h, const void* w, int N, int E, int D, int top, float scale, int groups, int keep, int gated,
-                            int* ids, float* wts, float* gate, int type, cudaStream_t st) {
-    const Select c{E, top, groups, keep, gated, scale, ids, wts, gate, nullptr, nullptr};
-    const int rows = E + (gated ? 1 : 0);
-    const size_t smem = (size_t)(D + rows + E + groups) * 4;
-    if (D % 8 || !select_ok(N, c) || smem > 48 * 1024) return 5;
-    if (type == 0)
-        return kb_launch_dep(route_token_kernel<bf16>, dim3(N), dim3(512), smem, st, (const bf16*)h, (const bf16*)w, rows, D, c);
-    return kb_launch_dep(route_token_kernel<float>, dim3(N), dim3(512), smem, st, (const float*)h, (const float*)w, rows, D, c);
+// logits[N, E] for few tokens (their rows are staged in shared memory, eight at a time).
+KB_API int kb_router_dot(const void* h, const void* w, float* logits, int N, int E, int D, int type, cudaStream_t st) {
+    const size_t smem = (size_t)DOT_TOKENS * D * (type == 0 ? 2 : 4);
+    if (D % 8 || N < 1 || E < 1 || smem > 200 * 1024) return 5;
+    static bool flags[2][64] = {};
+    bool* set = kb_device_flag(flags[type == 0 ? 0 : 1]);
+    if (!set) return 7;
+    if (!*set) {
+        if ((type == 0 ? cudaFuncSetAttribute(router_dot_kernel<bf16>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024)
+                       : cudaFuncSetAttribute(router_dot_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024)) !=
+            cudaSuccess)
+            return 7;
+        *set = true;
+    }
+    const dim3 grid((N + DOT_TOKENS - 1) / DOT_TOKENS, (E + 7) / 8);
+    if (type == 0) return kb_launch_dep(router_dot_kernel<bf16>, grid, dim3(256), smem, st, (const bf16*)h, (const bf16*)w, logits, N, E, D);
+    return kb_launch_dep(router_dot_kernel<float>, grid, dim3(256), smem, st, (const float*)h, (const float*)w, logits, N, E, D);
 }
-// Selection on logits[N, ld] (E expert logits and, with `gated`, the gate's).  counts[E] (zero) and rank[N, top] receive
-// what kb_moe_group needs.
+// Selection on logits[N, ld] (E expert logits and, with `gated`, the gate's).  ids, wts: [N, top]; gate: [N] or null.
+// counts[32 E] (every 32nd used, zero on entry) and rank[N, top] receive what kb_moe_group needs; null: not wanted.
 KB_API int kb_moe_select(const float* logits, int ld, int N, int E, int top, float scale, int groups, int keep, int gated, int* ids,
                          float* wts, float* gate, int* counts, int* rank, cudaStream_t st) {
     const Select c{E, top, groups, keep, gated, scale, ids, wts, gate, counts, rank};

@@ -783,7 +783,7 @@ class CudaOps(TorchOps):
                    _F(eps), _I(_TYPE[dtype]), _p(self.status(x.device)), _st())
         return out
 
-    moe_few = 256           # tokens up to which routing and grouping are one small kernel each
+    moe_few = 256           # tokens up to which the router is dot products and the grouping is found from the choices alone
 
     def moe_route(self, h, router, experts, top, scale, groups, keep):
         """Returns ``(ids, weights, gate, plan)``; ``plan`` (counts per expert, ranks) is for :meth:`moe_experts`."""
@@ -794,25 +794,20 @@ class CudaOps(TorchOps):
         ids = torch.empty(N, top, device=dev, dtype=torch.int32)
         wts = torch.empty(N, top, device=dev, dtype=torch.float32)
         gate = torch.empty(N, device=dev, dtype=torch.float32) if gated else None
-        if N <= self.moe_few and (D + 2 * E + groups) * 4 <= 48 * 1024:
-            self._call("kb_moe_route_few", _p(h), _p(router), _I(N), _I(experts), _I(D), _I(top), _F(scale), _I(groups), _I(keep),
-                       _I(int(gated)), _p(ids), _p(wts), _p(gate), _I(_TYPE[h.dtype]), _st())
-            return ids, wts, gate, None
-        # one zeroed buffer: the logits (the product adds its K parts up in it) and the experts' counts
-        ld = (E + 3) // 4 * 4
-        buf = torch.zeros(N * ld + experts, device=dev, dtype=torch.float32)
-        logits, counts = buf[: N * ld].view(N, ld)[:, :E], buf[N * ld:].view(torch.int32)
-        if h.dtype == torch.float32:
-            self._gemm(h, router, N, E, D, False, False, out=logits)
+        counts = rank = None
+        if N <= self.moe_few and 8 * D * h.element_size() <= 200 * 1024:
+            ld = E
+            logits = torch.empty(N, E, device=dev, dtype=torch.float32)
+            self._call("kb_router_dot", _p(h), _p(router), _p(logits), _I(N), _I(E), _I(D), _I(_TYPE[h.dtype]), _st())
         else:
-            split = max(1, min(4, 148 // ((N + 127) // 128), (D + 63) // 128))
-            self._call("kb_gemm", _p(h), _p(router), _p(logits), _p(None), _I(N), _I(E), _I(D), _I(1), _LL(h.stride(0)),
-                       _LL(router.stride(0)), _LL(ld), _LL(0), _LL(0), _LL(0), _LL(0), _LL(0), _I(0), _I(0), _I(1), _I(1), _I(2),
-                       _F(1.0), _F(0.0), _p(self.status(dev)), _I(0), _I(split), _st())
-        rank = torch.empty(N, top, device=dev, dtype=torch.int32)
+            ld = (E + 3) // 4 * 4            # rows the epilogue can store four numbers at a time
+            logits = torch.empty(N, ld, device=dev, dtype=torch.float32)
+            self._gemm(h, router, N, E, D, False, False, out=logits[:, :E])
+            counts = torch.zeros(experts * 32, device=dev, dtype=torch.int32)
+            rank = torch.empty(N, top, device=dev, dtype=torch.int32)
         self._call("kb_moe_select", _p(logits), _I(ld), _I(N), _I(experts), _I(top), _F(scale), _I(groups), _I(keep), _I(int(gated)),
                    _p(ids), _p(wts), _p(gate), _p(counts), _p(rank), _st())
-        return ids, wts, gate, (counts, rank)
+        return ids, wts, gate, None if counts is None else (counts, rank)
 
     def moe_experts(self, h, ids, up, down, kind, plan=None):
         rows, offsets, at = self._moe_group(h, ids, up.shape[0], plan)

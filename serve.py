@@ -2,7 +2,11 @@
 """Inference server entry point.
 
     python serve.py --checkpoint checkpoints/run/step_00045775.pt [--device cuda] [--host 0.0.0.0] [--port 2222]
+    python serve.py --model_dir models/some-model [--dtype bfloat16|float32] [--prefill_portion 512]
     torchrun --nproc-per-node 8 --master-addr 127.0.0.1 serve.py --model_size 3b ...    # tensor-parallel
+
+``--model_dir`` names a folder with ``config.json`` and ``model.safetensors``; the family is chosen by the configuration's
+``architecture`` (``kotodama_b200/models/registry.py``).
 
 Under ``torchrun`` the model is sharded over the ranks (tensor parallelism: heads, KV cache and MLP
 columns); rank 0 hosts the HTTP app and drives the other ranks in lock-step.
@@ -26,6 +30,7 @@ sys.path.insert(0, os.path.dirname(os.path.abspath(__file__)))
 from kotodama_b200.ckpt.manager import clean_state_dict, load_checkpoint_file  # noqa: E402
 from kotodama_b200.config import MODEL_PRESETS, ModelConfig  # noqa: E402
 from kotodama_b200.models.llama import KotodamaModel  # noqa: E402
+from kotodama_b200.models.registry import load_model as load_model_dir, read_config  # noqa: E402
 from kotodama_b200.serve.app import create_app, load_tokenizer  # noqa: E402
 from kotodama_b200.serve.engine import ServingEngine  # noqa: E402
 
@@ -72,6 +77,12 @@ def main() -> None:
     ap.add_argument("--max_ctx", type=int, default=None)
     ap.add_argument("--tokenizer", default=TOKENIZER_NAME)
     ap.add_argument("--random_init", action="store_true", help="serve random weights (smoke tests)")
+    ap.add_argument("--model_dir", default=None,
+                    help="folder with config.json and model.safetensors (with --random_init: config.json alone); replaces --checkpoint / --model_size")
+    ap.add_argument("--dtype", default=None, choices=["bfloat16", "float32"],
+                    help="default: bfloat16 on CUDA, float32 on CPU; float32 on CUDA for families with 32-bit kernels")
+    ap.add_argument("--prefill_portion", type=int, default=0,
+                    help="most prompt tokens of one request per step (0: whole prompts); families that continue a cached context")
     args = ap.parse_args()
     logging.basicConfig(level=logging.INFO, format="%(asctime)s %(levelname)s %(name)s: %(message)s")
     device = "cuda" if args.device == "cuda" and torch.cuda.is_available() else "cpu"
@@ -88,11 +99,20 @@ def main() -> None:
         else:
             dist.init_process_group("gloo")
         tp = ServeTP()
-    model = load_model(args.checkpoint, args.model_size, args.attn_res_boundaries, args.attn_res_n_blocks,
-                       not args.no_attn_res, args.random_init)
-    engine = ServingEngine(model, device=device, dtype=torch.bfloat16 if device.startswith("cuda") else torch.float32,
-                           max_batch=args.max_batch, max_ctx=args.max_ctx, tp=tp,
-                           prefill_batch_tokens=args.prefill_batch_tokens)
+    if args.model_dir is not None:
+        if args.random_init:
+            family, cfg = read_config(args.model_dir)
+            model = family.random(cfg, 0)
+        else:
+            model = load_model_dir(args.model_dir)
+        name = os.path.basename(os.path.normpath(args.model_dir))
+    else:
+        model = load_model(args.checkpoint, args.model_size, args.attn_res_boundaries, args.attn_res_n_blocks,
+                           not args.no_attn_res, args.random_init)
+        name = f"kotodama-{args.model_size}"
+    dtype = getattr(torch, args.dtype) if args.dtype else torch.bfloat16 if device.startswith("cuda") else torch.float32
+    engine = ServingEngine(model, device=device, dtype=dtype, max_batch=args.max_batch, max_ctx=args.max_ctx, tp=tp,
+                           prefill_batch_tokens=args.prefill_batch_tokens, prefill_portion=args.prefill_portion)
     if tp is not None and rank > 0:
         run_follower(engine, tp)
         return
@@ -102,7 +122,7 @@ def main() -> None:
     logger.info("Device %s, tokenizer %s, paged KV cache with %d pages", device, type(tok).__name__,
                 engine.cache.num_pages)
     import uvicorn
-    uvicorn.run(create_app(engine, tok, model_name=f"kotodama-{args.model_size}", checkpoint=args.checkpoint or ""), host=args.host, port=args.port)
+    uvicorn.run(create_app(engine, tok, model_name=name, checkpoint=args.model_dir or args.checkpoint or ""), host=args.host, port=args.port)
 
 
 if __name__ == "__main__":
