@@ -142,7 +142,20 @@ def kernels(name: str, z: dict, batch: int = 64, ctx: int = 1280, tokens: int = 
     ws = [ops.decode_weight(bf(nq, D)) for _ in range(max(2, int(400e6 // (nq * D * 2)) + 1))]
     ms = timed([lambda w=w: ops.gemm_nt(a, w) for w in ws])
     add("llama: q | k | v projection (decode)", "decode product", ms, nq * D * 2 + B * (D + nq) * 2, 2.0 * B * nq * D)
+    # what small decode launches cost in the Llama family: a product of about the bytes of a per-head product, row kernels
+    ws = [ops.decode_weight(bf(512, D)) for _ in range(64)]
+    ms = timed([lambda w=w: ops.gemm_nt(a, w) for w in ws])
+    add("llama: k or v projection alone (decode)", "decode product", ms, 512 * D * 2 + B * (D + 512) * 2, 2.0 * B * 512 * D)
     del ws
+    xs, one = [bf(B, D) for _ in range(8)], torch.ones(D, device=dev, dtype=torch.bfloat16)
+    ms = timed([lambda x=x: ops.route_norm_fwd([x], None, None, one, 1e-5) for x in xs])
+    add("llama: RMS norm (decode)", "row kernel", ms, B * D * 4)
+    gus = [bf(B, 2 * F) for _ in range(8)]
+    ms = timed([lambda x=x: ops.swiglu_fwd(x) for x in gus])
+    add("llama: SwiGLU (decode)", "row kernel", ms, B * 3 * F * 2)
+    xf, ones = [torch.randn(B, D, device=dev) for _ in range(8)], torch.ones(D, device=dev)
+    ms = timed([lambda x=x: ops.norm_add(x, a, ones, D, 1e-5) for x in xf])
+    add("norm + layer scale + residual (decode)", "row kernel", ms, B * D * 12)
     if z["experts"]:
         E, top, ff = z["experts"], z["top"], z["ff"]
         for n, tag, like in ((B, "decode", "decode product"), (tokens, "prefill", "product")):

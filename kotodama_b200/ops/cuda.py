@@ -801,9 +801,17 @@ class CudaOps(TorchOps):
             self._call("kb_router_dot", _p(h), _p(router), _p(logits), _I(N), _I(E), _I(D), _I(_TYPE[h.dtype]), _st())
         else:
             ld = (E + 3) // 4 * 4            # rows the epilogue can store four numbers at a time
-            logits = torch.empty(N, ld, device=dev, dtype=torch.float32)
-            self._gemm(h, router, N, E, D, False, False, out=logits[:, :E])
-            counts = torch.zeros(experts * 32, device=dev, dtype=torch.int32)
+            # one zeroed buffer: the logits (the product adds the parts of its K range up in it) and the experts' counters
+            buf = torch.zeros(N * ld + experts * 32, device=dev, dtype=torch.float32)
+            logits, counts = buf[: N * ld].view(N, ld), buf[N * ld:].view(torch.int32)
+            if h.dtype == torch.float32:
+                self._gemm(h, router, N, E, D, False, False, out=logits[:, :E])
+            else:
+                # a product this narrow has one tile per 128 tokens: K is cut so that all SMs stream rows
+                split = max(1, min(4, 148 // ((N + 127) // 128), (D + 63) // 64 // 4))
+                self._call("kb_gemm", _p(h), _p(router), _p(logits), _p(None), _I(N), _I(E), _I(D), _I(1), _LL(h.stride(0)),
+                           _LL(router.stride(0)), _LL(ld), _LL(0), _LL(0), _LL(0), _LL(0), _LL(0), _I(0), _I(0), _I(1), _I(1), _I(2),
+                           _F(1.0), _F(0.0), _p(self.status(dev)), _I(0), _I(split), _st())
             rank = torch.empty(N, top, device=dev, dtype=torch.int32)
         self._call("kb_moe_select", _p(logits), _I(ld), _I(N), _I(experts), _I(top), _F(scale), _I(groups), _I(keep), _I(int(gated)),
                    _p(ids), _p(wts), _p(gate), _p(counts), _p(rank), _st())

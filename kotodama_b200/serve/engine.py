@@ -100,6 +100,7 @@ class ServingEngine:
         self.tp = tp                                  # tensor-parallel helper (``serve.tp``) or None
         self.runner = make_runner(self)
         self.arena = getattr(self.runner, "arena", None)
+        self.H, self.KV = getattr(self.runner, "H", None), getattr(self.runner, "KV", None)     # local heads, where one number describes all layers
         cfg = self.cfg
         self.max_ctx = max_ctx or cfg.max_position_embeddings
         self.max_batch = max_batch

@@ -120,3 +120,23 @@ def test_decode_graphs_and_plain_launches_agree():
         s = eng.open()
         outs.append(cases.feed(eng, s, cases.tokens(cfg, 60, 2), [20, 1]))
     assert float((outs[0] - outs[1]).abs().max()) < 1e-4
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+def test_kernels_write_inside_their_tensors(dtype):
+    """Canary bands around every allocation: prompts, portions, decoding and generation at ragged sizes."""
+    from kotodama_b200.utils.guard import GuardRegions
+    with GuardRegions() as g:
+        for name in ("odd", "wide"):
+            cfg = cases.CONFIGS[name]
+            eng = cases.engine(cases.weights(cfg, 4), "cuda", dtype, max_ctx=400)
+            eng.use_cuda_graphs = False
+            s, t = eng.open(), eng.open()
+            toks = cases.tokens(cfg, 340, 3)
+            eng.feed([(s, toks[:301], [0, 300]), (t, toks[:7], [6])])
+            eng.feed([(s, toks[301:304], [2]), (t, toks[7:27], [])])
+            for i in range(5):
+                eng.feed([(s, [toks[304 + i]], [0]), (t, [toks[27 + i]], [0])])
+        torch.cuda.synchronize()
+        g.assert_clean()
+    get_ops("cuda").check_status()
