@@ -207,7 +207,7 @@ def run_serve(args, rank, world, local):
     with a device synchronize around every scheduler step: the host scheduling is part of serving."""
     sys.path.insert(0, os.path.join(ROOT, "benchmarks"))
     import serve_bench
-    a = argparse.Namespace(model=args.model, requests=64, min_prompt=128, max_prompt=2048, new_tokens=256, seed=0,
+    a = argparse.Namespace(model=args.model, requests=64, min_prompt=128, max_prompt=2048, new_tokens=256, seed=0, graph_times=False,
                            device="cuda", passes=2, profile_decode_step=-1, op_times="", prefill_batch_tokens=8192,
                            attn_res_blocks=args.attn_res_blocks)
     return serve_bench.run(a, rank, world, local)
