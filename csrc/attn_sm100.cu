@@ -25,6 +25,8 @@
 // through a two-stage ring.  The running maximum is refreshed lazily: O and the running sum are
 // rescaled only when a row's maximum grows by more than 2^8.
 // Every wait is bounded (status word on timeout).
+// Optional (template CAP): scores pass cap * tanh(score / cap) before the softmax, in fp32 on the accumulator.  Optional (runtime):
+// head outputs times the sigmoid of a gate per token and head, and output rows narrower than the head.
 #include "attn_common.cuh"
 
 namespace {
@@ -42,6 +44,26 @@ constexpr float RESCALE_THRESHOLD = 8.0f;          // in log2 units
 constexpr int EMU = 2;                             // of every 4 pairs of exponentials, this many run on the FMA pipe
 constexpr int FWD_THREADS = 320;                   // 8 softmax warps, MMA warp, TMA warp
 
+enum Cap { CAP_NONE = 0, CAP_SMALL = 1, CAP_ANY = 2 };
+constexpr float CAP_SMALL_BOUND = 0.6f;            // largest |score / cap| of CAP_SMALL
+
+// tanh of a pair.  CAP_SMALL: odd polynomial (Chebyshev interpolation of tanh(x) / x in x^2 on |x| <= 0.6, error 4e-8) on the FMA
+// pipe.  CAP_ANY: 1 - 2 / (1 + e^2x), error 1e-7 over the whole range.
+template <int CAP>
+__device__ __forceinline__ float2 tanh_pair(float2 x) {
+    if constexpr (CAP == CAP_SMALL) {
+        const float2 z = __fmul2_rn(x, x);
+        float2 p = __ffma2_rn(z, make_float2(0.015468751f, 0.015468751f), make_float2(-0.052096654f, -0.052096654f));
+        p = __ffma2_rn(p, z, make_float2(0.13310064f, 0.13310064f));
+        p = __ffma2_rn(p, z, make_float2(-0.33332303f, -0.33332303f));
+        p = __ffma2_rn(p, z, make_float2(0.99999994f, 0.99999994f));
+        return __fmul2_rn(p, x);
+    } else {
+        const float2 e = make_float2(exp2f(x.x * (2.0f * LOG2E)), exp2f(x.y * (2.0f * LOG2E)));
+        return make_float2(1.0f - __fdividef(2.0f, 1.0f + fminf(e.x, 1e30f)), 1.0f - __fdividef(2.0f, 1.0f + fminf(e.y, 1e30f)));
+    }
+}
+
 struct FlashParams {
     int B, T, H, KV;
     const int* cu_seqlens;                         // [B + 1] token offsets, or null: sequence b = rows [b*T, (b+1)*T)
@@ -57,6 +79,10 @@ struct FlashParams {
     long long q_stride, q_rows;
     int n_tiles;                                   // query tiles per sequence (grid decode)
     int* status;
+    float cap_in;                                  // CAP: scores enter tanh as score * cap_in; scale_log2 is then cap * log2(e)
+    const __nv_bfloat16* gate;                     // [rows, H] gates in rows gate_stride apart, or null
+    long long gate_stride;
+    int out_cols;                                  // leading columns per head that are written (a multiple of 8)
 };
 
 #ifdef KB_ATTN_PROFILE
@@ -77,7 +103,7 @@ constexpr int fwd_smem_bytes() {
     return (KST + VST) * Tile<HD>::BYTES + 1024 + 256 + 6 * BT * 4;
 }
 
-template <int HD>
+template <int HD, int CAP>
 __global__ void __launch_bounds__(FWD_THREADS, 1)
 flash_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK,
                  const __grid_constant__ CUtensorMap tmV, const FlashParams p) {
@@ -261,6 +287,14 @@ flash_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant_
             tc::tmem_ld32(tmem_s + hf * 64 + 32, reinterpret_cast<uint32_t*>(s + 32));
             tc::tmem_ld_wait();
             KB_TICK(2, tk)                                              // tensor-memory load
+            if constexpr (CAP != CAP_NONE) {
+#pragma unroll
+                for (int c = 0; c < 64; c += 2) {
+                    const float2 th = tanh_pair<CAP>(make_float2(s[c] * p.cap_in, s[c + 1] * p.cap_in));
+                    s[c] = th.x;
+                    s[c + 1] = th.y;
+                }
+            }
             if (j * BT + BT - 1 > qpos) {                           // tile on the diagonal: causal mask
                 const int cmax = qpos - j * BT + r - hf * 64;
 #pragma unroll
@@ -360,12 +394,14 @@ flash_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant_
         if (ok) {
             if (tc::mbar_wait(o_done, (n - 1) & 1, abort_flag)) {
                 tc::tc_fence_after();
-                const float inv = TRUNC_BIAS / l;
+                float inv = TRUNC_BIAS / l;
                 // Rows past the end of the sequence (zero-filled by TMA, or the first rows of the next
                 // sequence) are computed but never stored; for the valid rows the causal mask already
                 // excludes every key at or beyond the end.
                 const bool valid = qt * BT + r < Tb;
-                __nv_bfloat16* dst = p.out + (size_t)(seq_row0 + qt * BT + r) * p.out_stride + head * HD + hf * (HD / 2);
+                __nv_bfloat16* dst = p.out + (size_t)(seq_row0 + qt * BT + r) * p.out_stride + head * p.out_cols + hf * (HD / 2);
+                if (p.gate && valid)
+                    inv /= 1.0f + __expf(-__bfloat162float(p.gate[(size_t)(seq_row0 + qt * BT + r) * p.gate_stride + head]));
 #pragma unroll 1
                 for (int c = 0; c < HD / 2; c += 32) {
                     uint32_t o[32];
@@ -377,7 +413,7 @@ flash_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant_
                             float f8[8];
 #pragma unroll
                             for (int e = 0; e < 8; ++e) f8[e] = __uint_as_float(o[i + e]) * inv;
-                            st8(dst + c + i, pack8(f8));
+                            if (hf * (HD / 2) + c + i < p.out_cols) st8(dst + c + i, pack8(f8));
                         }
                     }
                 }
@@ -411,14 +447,14 @@ int ensure_smem(K kernel, int bytes, bool* done_for_device) {
     return 0;
 }
 
-template <int HD>
+template <int HD, int CAP>
 int launch_fwd(const CUtensorMap& tmQ, const CUtensorMap& tmK, const CUtensorMap& tmV, const FlashParams& p,
                int max_T, cudaStream_t st) {
     static bool attr[64] = {};
-    int r = ensure_smem(flash_fwd_kernel<HD>, fwd_smem_bytes<HD>(), attr);
+    int r = ensure_smem(flash_fwd_kernel<HD, CAP>, fwd_smem_bytes<HD>(), attr);
     if (r) return r;
     const int grid = p.n_tiles * p.H * p.B;
-    flash_fwd_kernel<HD><<<grid, FWD_THREADS, fwd_smem_bytes<HD>(), st>>>(tmQ, tmK, tmV, p);
+    flash_fwd_kernel<HD, CAP><<<grid, FWD_THREADS, fwd_smem_bytes<HD>(), st>>>(tmQ, tmK, tmV, p);
     return cudaGetLastError() == cudaSuccess ? 0 : 8;
 }
 
@@ -433,7 +469,9 @@ KB_API int kb_attn_dbg_read(long long* host16) {
 static int flash_fwd_impl(const void* q, long long q_stride, int q_cols, int q_col0, const void* k, long long k_stride,
                           int k_cols, int k_col0, const void* v, long long v_stride, int v_cols, int v_col0, void* out,
                           long long out_stride, float* lse, const int* cu_seqlens, long long total, const int* cu_keys,
-                          long long total_keys, int B, int max_T, int H, int KV, int hd, float scale, int* status, cudaStream_t st) {
+                          long long total_keys, int B, int max_T, int H, int KV, int hd, float scale, int* status, cudaStream_t st,
+                          float softcap = 0.f, float bound = 0.f, const void* gate = nullptr, long long gate_stride = 0, int out_cols = 0) {
+    if (out_cols < 0 || out_cols > hd || out_cols % 8) return 5;
     if ((hd != 128 && hd != 64) || max_T < 1 || B < 1 || KV < 1 || H % KV != 0) return 5;
     if (!operand_ok(q, q_stride, q_col0) || !operand_ok(k, k_stride, k_col0) || !operand_ok(v, v_stride, v_col0)) return 6;
     if (((uintptr_t)out & 15) || (out_stride & 7)) return 6;
@@ -463,7 +501,18 @@ static int flash_fwd_impl(const void* q, long long q_stride, int q_cols, int q_c
     p.q_rows = rows;
     p.n_tiles = (max_T + BT - 1) / BT;
     p.status = status;
-    return hd == 128 ? launch_fwd<128>(tmQ, tmK, tmV, p, max_T, st) : launch_fwd<64>(tmQ, tmK, tmV, p, max_T, st);
+    p.cap_in = 0.f;
+    p.gate = (const __nv_bfloat16*)gate;
+    p.gate_stride = gate_stride;
+    p.out_cols = out_cols ? out_cols : hd;
+    if (softcap > 0.f) {
+        p.cap_in = scale / softcap;
+        p.scale_log2 = softcap * LOG2E;
+        if (bound > 0.f && bound <= CAP_SMALL_BOUND * softcap)
+            return hd == 128 ? launch_fwd<128, CAP_SMALL>(tmQ, tmK, tmV, p, max_T, st) : launch_fwd<64, CAP_SMALL>(tmQ, tmK, tmV, p, max_T, st);
+        return hd == 128 ? launch_fwd<128, CAP_ANY>(tmQ, tmK, tmV, p, max_T, st) : launch_fwd<64, CAP_ANY>(tmQ, tmK, tmV, p, max_T, st);
+    }
+    return hd == 128 ? launch_fwd<128, CAP_NONE>(tmQ, tmK, tmV, p, max_T, st) : launch_fwd<64, CAP_NONE>(tmQ, tmK, tmV, p, max_T, st);
 }
 
 // q/k/v: token-major matrices [total tokens, *] whose rows hold the heads side by side (row strides
@@ -480,11 +529,14 @@ KB_API int kb_flash_fwd(const void* q, long long q_stride, int q_cols, int q_col
 
 // Packed queries against packed contexts: the queries of sequence b (rows cu_seqlens[b] .. cu_seqlens[b + 1] of q) are
 // the last of its key positions (rows cu_keys[b] .. cu_keys[b + 1] of k and v); max_T bounds the queries of a sequence.
+// softcap > 0: soft-capped scores; `bound` > 0: a bound on |score| (before the cap) that the caller vouches for.  gate: see FlashParams.
+// out_cols: leading columns per head that are written, heads out_cols apart (0: all).
 KB_API int kb_flash_fwd_context(const void* q, long long q_stride, int q_cols, const void* k, long long k_stride, int k_cols,
                                 const void* v, long long v_stride, int v_cols, void* out, long long out_stride,
                                 const int* cu_seqlens, long long total, const int* cu_keys, long long total_keys, int B, int max_T,
-                                int H, int KV, int hd, float scale, int* status, cudaStream_t st) {
+                                int H, int KV, int hd, float scale, float softcap, float bound, const void* gate, long long gate_stride,
+                                int out_cols, int* status, cudaStream_t st) {
     if (!cu_seqlens || !cu_keys) return 5;
     return flash_fwd_impl(q, q_stride, q_cols, 0, k, k_stride, k_cols, 0, v, v_stride, v_cols, 0, out, out_stride, nullptr, cu_seqlens,
-                          total, cu_keys, total_keys, B, max_T, H, KV, hd, scale, status, st);
+                          total, cu_keys, total_keys, B, max_T, H, KV, hd, scale, status, st, softcap, bound, gate, gate_stride, out_cols);
 }

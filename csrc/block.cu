@@ -1,5 +1,5 @@
-// Per-token steps of decoders with output norms and latent attention: pair embedding, latent norm + cache
-// append, cache gather, output norm + layer scale + residual, final norm, activations, logit soft-cap.
+// Per-token steps of decoders: pair embedding, latent norm + cache append, cache gather, output norm + layer
+// scale + residual, residual + pre-norm, final norm, activations, logit soft-cap.
 // The residual stream is fp32; T (bf16 or fp32) is the activation type.  Rows may be padded with zeros on the
 // right up to a multiple of 8 elements: `width` is the true size that means are taken over.
 // Compiled without fast-math: the fp32 mode is meant to be exact to fp32 rounding.
@@ -13,7 +13,8 @@ constexpr int PAGE = 16;
 template <typename T>
 __global__ void embed_pairs_kernel(const long long* __restrict__ ids, const int* __restrict__ prev, const T* __restrict__ table,
                                    const T* __restrict__ bigram, long long buckets, long long mul_prev, long long mul_cur,
-                                   float* __restrict__ x, T* __restrict__ h, int N, int D, int V, int* __restrict__ status) {
+                                   float scale, float* __restrict__ x, T* __restrict__ h, int N, int D, int V,
+                                   int* __restrict__ status) {
     kb_dep_trigger();
     kb_dep_wait();
     const int dc = D >> 3;
@@ -34,9 +35,11 @@ __global__ void embed_pairs_kernel(const long long* __restrict__ ids, const int*
 #pragma unroll
                 for (int j = 0; j < 8; ++j) v[j] += w[j];
             }
+#pragma unroll
+            for (int j = 0; j < 8; ++j) v[j] *= scale;
         }
         store8(x + (long long)row * D + c, v);
-        if ((const void*)h != (const void*)x) store8(h + (long long)row * D + c, v);
+        if (h && (const void*)h != (const void*)x) store8(h + (long long)row * D + c, v);
     }
 }
 
@@ -167,6 +170,61 @@ __global__ void norm_add_kernel(float* __restrict__ x, const T* __restrict__ y, 
     }
 }
 
+// x += y (+ step, one vector for all rows); h = rms(x) * w.  One block per row, eight elements per thread and step.  With
+// `rows`, output row i is made from row rows[i] and x is left as it is.
+template <typename T>
+__global__ void __launch_bounds__(1024)
+add_norm_kernel(float* __restrict__ x, const T* __restrict__ y, const float* __restrict__ step, const long long* __restrict__ rows,
+                const float* __restrict__ w, T* __restrict__ h, int N, int D, int width, float eps, int* __restrict__ status) {
+    __shared__ float scratch[32];
+    kb_dep_trigger();
+    kb_dep_wait();
+    long long row = blockIdx.x;
+    if (rows) {
+        row = rows[row];
+        if (row < 0 || row >= N) {                     // uniform over the block
+            if (threadIdx.x == 0 && status) atomicMax(status, (int)KB_BAD_INDEX);
+            return;
+        }
+    }
+    float v[MAXC][8];
+    float ss[1] = {0.f};
+#pragma unroll
+    for (int i = 0; i < MAXC; ++i) {
+        const int c = (i * blockDim.x + threadIdx.x) * 8;
+        if (c >= D) break;
+        float* a = v[i];
+        load8(x + row * D + c, a);
+        if (y) {
+            float e[8];
+            load8(y + row * D + c, e);
+#pragma unroll
+            for (int j = 0; j < 8; ++j) a[j] += e[j];
+        }
+        if (step) {
+            float e[8];
+            load8(step + c, e);
+#pragma unroll
+            for (int j = 0; j < 8; ++j) a[j] += e[j];
+        }
+        if (!rows && (y || step)) store8(x + row * D + c, a);
+#pragma unroll
+        for (int j = 0; j < 8; ++j) ss[0] += a[j] * a[j];
+    }
+    block_sum<1>(ss, scratch);
+    const float r = 1.0f / sqrtf(ss[0] / (float)width + eps);
+#pragma unroll
+    for (int i = 0; i < MAXC; ++i) {
+        const int c = (i * blockDim.x + threadIdx.x) * 8;
+        if (c >= D) break;
+        float g[8];
+        load8(w + c, g);
+#pragma unroll
+        for (int j = 0; j < 8; ++j) v[i][j] = v[i][j] * r * g[j];
+        store8(h + (long long)blockIdx.x * D + c, v[i]);
+    }
+}
+
 template <typename T>
 __global__ void norm_rows_kernel(const float* __restrict__ x, const long long* __restrict__ rows, const float* __restrict__ w,
                                  T* __restrict__ out, int N, int D, int width, float eps, int* __restrict__ status) {
@@ -219,6 +277,17 @@ __global__ void activate_kernel(const T* __restrict__ u, T* __restrict__ out, lo
     }
 }
 
+// act = silu(gate) * up from rows of gate | up, fp32 (the bf16 form is kb_swiglu_fwd)
+__global__ void swiglu_f32_kernel(const float* __restrict__ gu, float* __restrict__ act, long long N, int F) {
+    kb_dep_trigger();
+    kb_dep_wait();
+    for (long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x; i < N * F; i += (long long)gridDim.x * blockDim.x) {
+        const long long row = i / F, c = i % F;
+        const float g = gu[row * 2 * F + c];
+        act[i] = g / (1.0f + expf(-g)) * gu[row * 2 * F + F + c];
+    }
+}
+
 __global__ void softcap_kernel(float* __restrict__ x, long long n, float cap) {
     kb_dep_trigger();
     kb_dep_wait();
@@ -243,15 +312,15 @@ inline int row_threads(int D) {
 // The latent cache is [pages, R / W, 16, W]: W columns of a page's 16 tokens are contiguous.
 // Types: 0 = bf16, 1 = fp32 activations.  D and R are multiples of 8, bases 16-byte aligned.
 KB_API int kb_embed_pairs(const long long* ids, const int* prev, const void* table, const void* bigram, long long buckets,
-                          long long mul_prev, long long mul_cur, float* x, void* h, int N, int D, int V, int type, int* status,
-                          cudaStream_t st) {
+                          long long mul_prev, long long mul_cur, float scale, float* x, void* h, int N, int D, int V, int type,
+                          int* status, cudaStream_t st) {
     if (D % 8 || N < 1 || V < 1 || (bigram && (buckets < 1 || !prev || mul_prev < 0 || mul_cur < 0))) return 5;
     const dim3 grid = flat_grid((long long)N * (D / 8), 256);
     if (type == 0)
         return kb_launch_dep(embed_pairs_kernel<bf16>, grid, dim3(256), 0, st, ids, prev, (const bf16*)table, (const bf16*)bigram,
-                             buckets, mul_prev, mul_cur, x, (bf16*)h, N, D, V, status);
+                             buckets, mul_prev, mul_cur, scale, x, (bf16*)h, N, D, V, status);
     return kb_launch_dep(embed_pairs_kernel<float>, grid, dim3(256), 0, st, ids, prev, (const float*)table, (const float*)bigram,
-                         buckets, mul_prev, mul_cur, x, (float*)h, N, D, V, status);
+                         buckets, mul_prev, mul_cur, scale, x, (float*)h, N, D, V, status);
 }
 KB_API int kb_latent_append(const void* rows, long long stride, const float* w, int width, float eps, void* pages, int W,
                             const long long* slots, void* out, int N, int R, long long num_slots, int type, int* status,
@@ -302,6 +371,20 @@ KB_API int kb_norm_rows(const float* x, const long long* rows, const float* w, v
                              eps, status);
     return kb_launch_dep(norm_rows_kernel<float>, dim3(n_rows), dim3(row_threads(D)), 0, st, x, rows, w, (float*)out, N, D, width,
                          eps, status);
+}
+KB_API int kb_add_norm(float* x, const void* y, const float* step, const long long* rows, const float* w, void* h, int n_rows, int N, int D,
+                       int width, float eps, int type, int* status, cudaStream_t st) {
+    if (D % 8 || D > 1024 * 8 * MAXC || n_rows < 1) return 5;
+    const dim3 grid(n_rows), block(row_threads(D));
+    if (type == 0)
+        return kb_launch_dep(add_norm_kernel<bf16>, grid, block, 0, st, x, (const bf16*)y, step, rows, w, (bf16*)h, N, D, width, eps,
+                             status);
+    return kb_launch_dep(add_norm_kernel<float>, grid, block, 0, st, x, (const float*)y, step, rows, w, (float*)h, N, D, width, eps,
+                         status);
+}
+KB_API int kb_swiglu_f32(const float* gu, float* act, long long N, int F, cudaStream_t st) {
+    if (N < 1 || F < 1) return 5;
+    return kb_launch_dep(swiglu_f32_kernel, flat_grid(N * F, 256), dim3(256), 0, st, gu, act, N, F);
 }
 KB_API int kb_activate(const void* u, void* out, long long n, int kind, int type, cudaStream_t st) {
     if (n % 8 || (kind != 1 && kind != 2)) return 5;

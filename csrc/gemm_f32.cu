@@ -10,9 +10,9 @@ constexpr int TM = 64, TN = 64, TK = 16;
 struct F32Params {
     const float *A, *B;
     float* C;
-    const float* Cin;              // added, may be null, laid out like C
+    const float* Cin;              // added, may be null; rows ldcin apart (0: one row for all), batches like C
     int M, N, K;
-    long long lda, ldb, ldc, a_bs, b_bs, c_bs;
+    long long lda, ldb, ldc, ldcin, a_bs, b_bs, c_bs;
     int b_mn;                      // B is [K, N]
     const int* offsets;            // grouped: blockIdx.z is the group, M is ignored
 };
@@ -75,7 +75,7 @@ __global__ void __launch_bounds__(256) gemm_f32_kernel(const F32Params p) {
 #pragma unroll
         for (int j = 0; j < 4; ++j) {
             const int n = col0 + tx * 4 + j;
-            if (n < p.N) C[(long long)m * p.ldc + n] = acc[i][j] + (Cin ? Cin[(long long)m * p.ldc + n] : 0.f);
+            if (n < p.N) C[(long long)m * p.ldc + n] = acc[i][j] + (Cin ? Cin[(long long)m * p.ldcin + n] : 0.f);
         }
     }
 }
@@ -84,9 +84,9 @@ __global__ void __launch_bounds__(256) gemm_f32_kernel(const F32Params p) {
 
 // Grouped (offsets not null): `M` is the total number of rows, `batch` the number of groups.
 KB_API int kb_gemm_f32(const float* A, const float* B, float* C, const float* Cin, int M, int N, int K, int batch, long long lda,
-                       long long ldb, long long ldc, long long a_bs, long long b_bs, long long c_bs, int b_mn, const int* offsets,
+                       long long ldb, long long ldc, long long ldcin, long long a_bs, long long b_bs, long long c_bs, int b_mn, const int* offsets,
                        cudaStream_t st) {
     if (M < 1 || N < 1 || K < 1 || batch < 1 || batch > 65535 || (M + TM - 1) / TM > 65535) return 5;
-    F32Params p{A, B, C, Cin, M, N, K, lda, ldb, ldc, a_bs, b_bs, c_bs, b_mn, offsets};
+    F32Params p{A, B, C, Cin, M, N, K, lda, ldb, ldc, ldcin, a_bs, b_bs, c_bs, b_mn, offsets};
     return kb_launch_dep(gemm_f32_kernel, dim3((N + TN - 1) / TN, (M + TM - 1) / TM, batch), dim3(256), 0, st, p);
 }

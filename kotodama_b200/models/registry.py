@@ -15,6 +15,7 @@ import torch
 
 from ..ckpt.safetensors import load_safetensors
 from ..config import ModelConfig
+from .lisunex import LisunexConfig, LisunexModel
 from .llama import KotodamaModel
 from .vunitar import VunitarConfig, VunitarModel
 
@@ -51,6 +52,9 @@ FAMILIES: dict[str, Family] = {
     "Vunitar": Family(VunitarConfig.from_dict, VunitarModel, VunitarModel.random_init, VunitarModel, "LatentRunner",
                       ("elementwise", "serve", "sampler", "attn_sm100", "gemm_sm100", "gemm2_sm100", "gemm_skinny_sm100",
                        "latent_attn", "latent_attn_sm100", "moe", "gemm_grouped_sm100", "gemm_f32", "block")),
+    "Lisunex": Family(LisunexConfig.from_dict, LisunexModel, LisunexModel.random_init, LisunexModel, "HybridRunner",
+                      ("elementwise", "serve", "sampler", "attn_sm100", "gemm_sm100", "gemm2_sm100", "gemm_skinny_sm100",
+                       "gemm_f32", "block", "paged_attn", "delta")),
 }
 
 

@@ -148,7 +148,7 @@ class CudaOps(TorchOps):
         tiles = ((M + 127) // 128) * ((N + 255) // 256)
         kblocks = (K + 63) // 64
         if (batch == 1 and M <= 128 and tiles <= 74 and kblocks >= 8 and out.dtype == torch.bfloat16
-                and out.is_contiguous() and (cin is None or cin.is_contiguous()) and self.split_k_small_m):
+                and out.is_contiguous() and (cin is None or cin.stride(-1) == 1) and self.split_k_small_m):
             # skinny (decode-size) products: too few output tiles to fill the GPU.  bf16 K-major operands: the K
             # range is split over the CTAs of a thread-block cluster and the partial tiles are summed through
             # distributed shared memory (one launch); otherwise split-K with fp32 atomics and a finishing kernel
@@ -164,6 +164,7 @@ class CudaOps(TorchOps):
                 if rc != 9:                          # 9: the runtime could not place the cluster - use the atomics path
                     self._rc(rc, "kb_gemm_skinny")
                 self.skinny_cluster = False
+            cin = cin.contiguous() if cin is not None else None
             split = max(2, min(148 // tiles, kblocks // 2, 16))
             # one fp32 workspace per output size, zeroed once: the finishing kernel clears it again
             key = (M * N, a.device.index)
@@ -217,11 +218,12 @@ class CudaOps(TorchOps):
         if out is None:
             out = torch.empty(*((batch,) if batch > 1 else ()), M, N, device=a.device, dtype=torch.float32)
         if a.stride(-1) != 1 or b.stride(-1) != 1 or out.stride(-1) != 1 or out.dtype != torch.float32 or (
-                cin is not None and cin.stride() != out.stride()):
-            raise KernelError("fp32 products take row-major operands; the addend is laid out like the output")
+                cin is not None and (cin.stride(-1) != 1 or (batch > 1 and cin.stride() != out.stride()))):
+            raise KernelError("fp32 products take row-major operands; the addend of a batch is laid out like the output")
         bs = lambda t: t.stride(0) if batch > 1 else 0
         self._call("kb_gemm_f32", _p(a), _p(b), _p(out), _p(cin), _I(M), _I(N), _I(K), _I(batch), _LL(a.stride(-2)),
-                   _LL(b.stride(-2)), _LL(out.stride(-2)), _LL(bs(a)), _LL(bs(b)), _LL(bs(out)), _I(int(b_mn)), _p(None), _st())
+                   _LL(b.stride(-2)), _LL(out.stride(-2)), _LL(cin.stride(-2) if cin is not None else 0), _LL(bs(a)), _LL(bs(b)), _LL(bs(out)),
+                   _I(int(b_mn)), _p(None), _st())
         return out
 
     # ------------------------------------------------------------------ block-scaled fp8
@@ -538,6 +540,9 @@ class CudaOps(TorchOps):
     def swiglu_fwd(self, gu):
         N, F2 = gu.shape
         act = torch.empty(N, F2 // 2, device=gu.device, dtype=gu.dtype)
+        if gu.dtype == torch.float32:
+            self._call("kb_swiglu_f32", _p(gu), _p(act), _LL(N), _I(F2 // 2), _st())
+            return act
         self._rc(self.lib.kb_swiglu_fwd(_p(gu), _p(act), _LL(N), _I(F2 // 2), _st()), "kb_swiglu_fwd")
         return act
 
@@ -689,12 +694,12 @@ class CudaOps(TorchOps):
     def latent_block(self, dtype, R):
         return 64 if dtype == torch.bfloat16 else R        # a block of a page is one TMA copy
 
-    def embed_pairs(self, ids, prev, table, bigram, consts):
+    def embed_pairs(self, ids, prev, table, bigram, consts, scale=1.0):
         N, D = ids.numel(), table.shape[1]
         x = torch.empty(N, D, device=table.device, dtype=torch.float32)
         h = x if table.dtype == torch.float32 else torch.empty(N, D, device=table.device, dtype=table.dtype)
         self._call("kb_embed_pairs", _p(ids), _p(prev), _p(table), _p(bigram), _LL(consts[0]), _LL(consts[1]), _LL(consts[2]),
-                   _p(x), _p(h), _I(N), _I(D), _I(table.shape[0]), _I(_TYPE[table.dtype]), _p(self.status(table.device)), _st())
+                   _F(scale), _p(x), _p(h), _I(N), _I(D), _I(table.shape[0]), _I(_TYPE[table.dtype]), _p(self.status(table.device)), _st())
         return x, h
 
     def latent_append(self, rows, w, width, eps, pages, slots):
@@ -735,7 +740,7 @@ class CudaOps(TorchOps):
                    _p(cu_seqlens), _I(B), _p(out), _I(N), _I(H), _I(R), _F(scale), _I(_TYPE[q.dtype]), _p(self.status(dev)), _st())
         return out
 
-    def attention_context(self, q, k, v, cu_seqlens, cu_context, max_q, scale):
+    def attention_context(self, q, k, v, cu_seqlens, cu_context, max_q, scale, softcap=0.0, gate=None, cols=0, bound=0.0):
         Nq, H, hd = q.shape
         Nk, KV = k.shape[0], k.shape[1]
         if q.dtype != torch.bfloat16 or hd not in (64, 128) or v.shape[2] != hd:
@@ -743,10 +748,14 @@ class CudaOps(TorchOps):
         for t in (q, k, v):
             if t.stride(2) != 1 or t.stride(1) != hd:
                 raise KernelError("attention operands are token-major rows with the heads side by side")
-        out = torch.empty(Nq, H, hd, device=q.device, dtype=q.dtype)
+        if gate is not None and gate.stride(1) != 1:
+            raise KernelError("attention gates are rows of one number per head")
+        cols = cols or hd
+        out = torch.empty(Nq, H, cols, device=q.device, dtype=q.dtype)
         self._call("kb_flash_fwd_context", _p(q), _LL(q.stride(0)), _I(H * hd), _p(k), _LL(k.stride(0)), _I(KV * hd), _p(v),
-                   _LL(v.stride(0)), _I(KV * hd), _p(out), _LL(H * hd), _p(cu_seqlens), _LL(Nq), _p(cu_context), _LL(Nk),
-                   _I(cu_seqlens.numel() - 1), _I(max_q), _I(H), _I(KV), _I(hd), _F(scale), _p(self.status(q.device)), _st())
+                   _LL(v.stride(0)), _I(KV * hd), _p(out), _LL(H * cols), _p(cu_seqlens), _LL(Nq), _p(cu_context), _LL(Nk),
+                   _I(cu_seqlens.numel() - 1), _I(max_q), _I(H), _I(KV), _I(hd), _F(scale), _F(softcap), _F(bound), _p(gate),
+                   _LL(gate.stride(0) if gate is not None else 0), _I(cols), _p(self.status(q.device)), _st())
         return out
 
     def head_gemm(self, a, w, transposed=False):
@@ -838,10 +847,67 @@ class CudaOps(TorchOps):
         out = torch.empty(A, M, device=rows.device, dtype=rows.dtype)
         if rows.dtype == torch.float32:
             self._call("kb_gemm_f32", _p(rows), _p(w), _p(out), _p(None), _I(A), _I(M), _I(K), _I(E), _LL(K), _LL(K), _LL(M), _LL(0),
-                       _LL(M * K), _LL(0), _I(0), _p(offsets), _st())
+                       _LL(0), _LL(M * K), _LL(0), _I(0), _p(offsets), _st())
             return self.activate(out, kind) if kind else out
         self._call("kb_gemm_grouped", _p(rows), _p(w), _p(out), _p(offsets), _I(A), _I(E), _I(M), _I(K), _LL(M),
                    _I({None: 0, "gelu": 1, "relu2": 2}[kind]), _I(int(A <= 24 * E)), _p(self.status(rows.device)), _st())
+        return out
+
+    # ------------------------------------------------------------------ pre-norm decoders with grouped attention and delta rule
+    def add_norm(self, x, y, step, w, width, eps, dtype, rows=None):
+        n = x.shape[0] if rows is None else rows.numel()
+        h = torch.empty(n, x.shape[1], device=x.device, dtype=dtype)
+        self._call("kb_add_norm", _p(x), _p(y), _p(step), _p(rows), _p(w), _p(h), _I(n), _I(x.shape[0]), _I(x.shape[1]), _I(width), _F(eps),
+                   _I(_TYPE[dtype]), _p(self.status(x.device)), _st())
+        return h
+
+    def flash_heads(self, dtype, dim, vdim):
+        return super().flash_heads(dtype, dim, vdim) if dtype == torch.bfloat16 else 0
+
+    def head_rotary_norm(self, rows, H, G, dim, vdim, cos, sin, positions, eps, k_pages, v_pages, slots, keep):
+        N = rows.shape[0]
+        kd, vd = k_pages.shape[3], v_pages.shape[3]
+        up8 = lambda n: (n + 7) // 8 * 8
+        col_k = up8(H * dim)
+        q = torch.empty(N, H, kd, device=rows.device, dtype=rows.dtype)
+        k = torch.empty(N, G, kd, device=rows.device, dtype=rows.dtype) if keep else None
+        v = torch.empty(N, G, vd, device=rows.device, dtype=rows.dtype) if keep else None
+        self._call("kb_head_rotary", _p(rows), _LL(rows.stride(0)), _I(H), _I(G), _I(dim), _I(vdim), _I(kd), _I(vd), _I(cos.shape[1]), _I(col_k),
+                   _I(col_k + up8(G * dim)), _p(cos), _p(sin), _I(cos.shape[0]), _p(positions), _F(eps), _p(q), _p(k), _p(v), _p(k_pages),
+                   _p(v_pages), _p(slots), _LL(k_pages.shape[0] * k_pages.shape[2]), _I(N), _I(_TYPE[rows.dtype]), _p(self.status(rows.device)),
+                   _st())
+        return q, k, v
+
+    def kv_gather(self, k_pages, v_pages, page_table, seg_seq, seg_first, cu, total):
+        G, kd, vd = k_pages.shape[1], k_pages.shape[3], v_pages.shape[3]
+        k = torch.empty(total, G, kd, device=k_pages.device, dtype=k_pages.dtype)
+        v = torch.empty(total, G, vd, device=k_pages.device, dtype=k_pages.dtype)
+        self._call("kb_kv_gather", _p(k_pages), _p(v_pages), _I(G), _I(kd), _I(vd), _p(page_table), _I(page_table.shape[0]), _I(page_table.shape[1]),
+                   _I(k_pages.shape[0]), _p(seg_seq), _p(seg_first), _p(cu), _I(seg_seq.numel()), _p(k), _p(v), _I(total),
+                   _I(_TYPE[k_pages.dtype]), _p(self.status(k_pages.device)), _st())
+        return k, v
+
+    def paged_attention(self, q, k_pages, v_pages, page_table, ctx_lens, cu_seqlens, max_ctx, scale, softcap, chunk, gate, vdim, cols):
+        N, H, kd = q.shape
+        out = torch.empty(N, H * cols, device=q.device, dtype=q.dtype)
+        self._call("kb_paged_attn_plain", _p(q), _p(k_pages), _p(v_pages), _I(k_pages.shape[1]), _I(kd), _I(v_pages.shape[3]), _p(page_table),
+                   _I(page_table.shape[1]), _I(k_pages.shape[0]), _p(ctx_lens), _p(cu_seqlens), _I(page_table.shape[0]), _p(gate),
+                   _LL(gate.stride(0) if gate is not None else 0), _p(out), _I(N), _I(H), _I(vdim), _I(cols), _F(scale), _F(softcap), _I(chunk),
+                   _I(_TYPE[q.dtype]), _p(self.status(q.device)), _st())
+        return out
+
+    def delta_rule(self, rows, H, G, d, dv, conv, a_log, dt_bias, norm, eps, state, ring, slots, cu_seqlens, ctx_lens, max_q):
+        N = rows.shape[0]
+        up8 = lambda n: (n + 7) // 8 * 8
+        cols = [0]
+        for n in (G * d, G * d, H * dv, H * dv, H):
+            cols.append(cols[-1] + up8(n))
+        width = up8(H * dv)
+        out = (torch.empty if width == H * dv else torch.zeros)(N, width, device=rows.device, dtype=rows.dtype)
+        self._call("kb_delta_step", _p(rows), _LL(rows.stride(0)), *map(_I, cols), _p(conv), _p(a_log), _p(dt_bias), _p(norm),
+                   _I(conv.shape[1]), _I(H), _I(G), _I(d), _I(dv), _I(state.shape[3]), _F(eps), _p(state), _p(ring), _I(ring.shape[2]),
+                   _I(state.shape[0]), _p(slots), _p(cu_seqlens), _p(ctx_lens), _I(slots.numel()), _p(out), _LL(width), _I(_TYPE[rows.dtype]),
+                   _p(self.status(rows.device)), _st())
         return out
 
     def softcap_(self, logits, cap):

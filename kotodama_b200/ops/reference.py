@@ -667,14 +667,15 @@ class TorchOps:
         t = pages[page_ids.long()]                                      # [p, R / W, 16, W]
         return t.transpose(1, 2).reshape(t.shape[0] * 16, -1)[:n]
 
-    def embed_pairs(self, ids, prev, table, bigram, consts):
-        """``x = table[id] (+ bigram[row])`` with ``row = (prev * mul_prev + id * mul_cur) mod buckets``, or row
+    def embed_pairs(self, ids, prev, table, bigram, consts, scale=1.0):
+        """``x = (table[id] (+ bigram[row])) * scale`` with ``row = (prev * mul_prev + id * mul_cur) mod buckets``, or row
         ``buckets`` where ``prev < 0``; ``consts = (buckets, mul_prev, mul_cur)``.  Returns ``x`` fp32 and its rounding to the table's dtype."""
         x = _f(table[ids]).clone()
         if bigram is not None:
             n, a, c = consts
             row = torch.where(prev < 0, torch.full_like(ids, n), (prev.long() * a + ids * c) % n)
             x = x + _f(bigram[row])
+        x = x * scale
         return x, x.to(table.dtype, copy=True)
 
     def latent_append(self, rows, w, width, eps, pages, slots):
@@ -707,18 +708,29 @@ class TorchOps:
             out[lo:hi] = torch.einsum("nht,tr->nhr", p, c).to(q.dtype)
         return out
 
-    def attention_context(self, q, k, v, cu_seqlens, cu_context, max_q, scale):
-        """Causal attention of packed query rows ``q[Nq, H, d]`` against packed contexts ``k, v[Nk, H, d]``: the queries
-        of sequence ``b`` are the last of its ``cu_context[b+1] - cu_context[b]`` positions."""
-        out = torch.empty(q.shape[0], q.shape[1], v.shape[2], device=q.device, dtype=q.dtype)
+    def attention_context(self, q, k, v, cu_seqlens, cu_context, max_q, scale, softcap=0.0, gate=None, cols=0, bound=0.0):
+        """Causal attention of packed query rows ``q[Nq, H, d]`` against packed contexts ``k, v[Nk, G, d]`` (``G`` divides
+        ``H``): the queries of sequence ``b`` are the last of its ``cu_context[b+1] - cu_context[b]`` positions.  ``softcap``:
+        scores pass ``softcap * tanh(score / softcap)``; ``gate[Nq, H]``: head outputs are multiplied by its sigmoid; ``cols``: leading
+        output columns per head that are wanted (0: all); ``bound`` > 0: no score (before the soft-cap) is larger."""
+        cols = cols or v.shape[2]
+        out = torch.empty(q.shape[0], q.shape[1], cols, device=q.device, dtype=q.dtype)
         cq, ck = cu_seqlens.tolist(), cu_context.tolist()
+        rep = q.shape[1] // k.shape[1]
         for b in range(len(cq) - 1):
             qb, kb, vb = _f(q[cq[b]:cq[b + 1]]), _f(k[ck[b]:ck[b + 1]]), _f(v[ck[b]:ck[b + 1]])
+            if rep > 1:
+                kb, vb = kb.repeat_interleave(rep, 1), vb.repeat_interleave(rep, 1)
             n, t = qb.shape[0], kb.shape[0]
             s = torch.einsum("nhd,thd->hnt", qb, kb) * scale
+            if softcap:
+                s = softcap * torch.tanh(s / softcap)
             seen = torch.arange(t, device=q.device)[None, :] <= torch.arange(t - n, t, device=q.device)[:, None]
             p = torch.softmax(s.masked_fill(~seen, float("-inf")), -1)
-            out[cq[b]:cq[b + 1]] = torch.einsum("hnt,thd->nhd", p, vb).to(q.dtype)
+            o = torch.einsum("hnt,thd->nhd", p, vb)[..., :cols]
+            if gate is not None:
+                o = o * torch.sigmoid(_f(gate[cq[b]:cq[b + 1]]))[..., None]
+            out[cq[b]:cq[b + 1]] = o.to(q.dtype)
         return out
 
     def head_gemm(self, a, w, transposed: bool = False):
@@ -776,6 +788,138 @@ class TorchOps:
         if ys is not None:
             y = y + gate.unsqueeze(-1) * _f(ys)
         return self.norm_add(x, y, g, width, eps).to(dtype)
+
+    # ------------------------------------------------------------- pre-norm decoders with grouped attention and delta rule
+    def add_norm(self, x, y, step, w, width, eps, dtype, rows=None):
+        """``x += y`` (rows; None: nothing) and ``x += step`` (one vector for all rows; None: nothing) in place; returns
+        ``rms(x) * w`` in ``dtype``.  With ``rows``: the result for these rows only, and ``x`` stays as it is."""
+        if rows is not None:
+            x, y = x[rows], y[rows] if y is not None else None
+        if y is not None:
+            x += _f(y)
+        if step is not None:
+            x += step
+        return (x * torch.rsqrt(x.pow(2).sum(-1, keepdim=True) / width + eps) * w).to(dtype)
+
+    def flash_heads(self, dtype: torch.dtype, dim: int, vdim: int) -> int:
+        """Size that keys and values of such heads are padded to for :meth:`attention_context` (0: it does not take them)."""
+        n = max(dim, vdim)
+        return 0 if n > 128 else 64 if n <= 64 else 128
+
+    def head_rotary_norm(self, rows, H, G, dim, vdim, cos, sin, positions, eps, k_pages, v_pages, slots, keep):
+        """``rows[N, *]`` hold ``q [H, dim] | k [G, dim] | v [G, vdim]``, each part starting at a multiple of eight columns.  Rotary
+        positions on the first ``2 * cos.shape[1]`` elements of the query and key heads (element ``i`` with ``i + half``),
+        then every head is divided by its root mean square.  Keys and values go to cache slots ``slots`` (negative: nowhere) of
+        ``pages[P, G, 16, size >= dim, vdim]``.  Returns ``q[N, H, size]`` and, when ``keep``, ``k, v[N, G, size]``, padded
+        with zeros like the cache."""
+        N, half = rows.shape[0], cos.shape[1]
+        up8 = lambda n: (n + 7) // 8 * 8
+        kd, vd = k_pages.shape[3], v_pages.shape[3]
+        at = up8(H * dim), up8(H * dim) + up8(G * dim)
+        c, s = cos[positions.long()][:, None], sin[positions.long()][:, None]
+
+        def turn(z):
+            z = _f(z)
+            u, v = z[..., :half], z[..., half:2 * half]
+            z = torch.cat([u * c - v * s, v * c + u * s, z[..., 2 * half:]], -1)
+            z = z * torch.rsqrt(z.pow(2).mean(-1, keepdim=True) + eps)
+            return F.pad(z, (0, kd - dim)).to(rows.dtype)
+
+        q = turn(rows[:, : H * dim].reshape(N, H, dim))
+        k = turn(rows[:, at[0]: at[0] + G * dim].reshape(N, G, dim))
+        v = F.pad(rows[:, at[1]: at[1] + G * vdim].reshape(N, G, vdim), (0, vd - vdim))
+        ok = slots >= 0
+        k_pages[slots[ok] // 16, :, slots[ok] % 16] = k[ok]
+        v_pages[slots[ok] // 16, :, slots[ok] % 16] = v[ok]
+        return (q, k, v) if keep else (q, None, None)
+
+    def kv_gather(self, k_pages, v_pages, page_table, seg_seq, seg_first, cu, total):
+        """Packed copies ``k, v[total, G, size]`` of cached rows: segment ``s`` holds positions ``seg_first[s] ..`` of sequence
+        ``seg_seq[s]`` in rows ``cu[s] .. cu[s + 1]``."""
+        ks, vs = [], []
+        cul = cu.tolist()
+        for i, (b, f) in enumerate(zip(seg_seq.tolist(), seg_first.tolist())):
+            t = torch.arange(f, f + cul[i + 1] - cul[i], device=k_pages.device)
+            page = page_table[b, t // 16].long()
+            ks.append(k_pages[page, :, t % 16])
+            vs.append(v_pages[page, :, t % 16])
+        return torch.cat(ks), torch.cat(vs)
+
+    def paged_attention(self, q, k_pages, v_pages, page_table, ctx_lens, cu_seqlens, max_ctx, scale, softcap, chunk, gate, vdim, cols):
+        """``q[N, H, size]`` against the paged cache; sequence ``b`` owns rows ``cu_seqlens[b:b+2]`` (None: row ``b``), the last of
+        its ``ctx_lens[b]`` tokens.  A query sees the keys up to its own position, with ``chunk`` > 0 only those of its chunk of the
+        sequence.  ``softcap``, ``gate`` as in :meth:`attention_context`.  Returns ``[N, H * cols]`` (columns past ``vdim`` are zero)."""
+        N, H = q.shape[:2]
+        out = torch.zeros(N, H, cols, device=q.device, dtype=q.dtype)
+        cu = cu_seqlens.tolist() if cu_seqlens is not None else list(range(N + 1))
+        rep = H // k_pages.shape[1]
+        for b, n in enumerate(ctx_lens.tolist()):
+            lo, hi = cu[b], cu[b + 1]
+            t = torch.arange(n, device=q.device)
+            page = page_table[b, t // 16].long()
+            k = _f(k_pages[page, :, t % 16]).repeat_interleave(rep, 1)
+            v = _f(v_pages[page, :, t % 16]).repeat_interleave(rep, 1)[..., :vdim]
+            s = torch.einsum("nhd,thd->hnt", _f(q[lo:hi]), k) * scale
+            if softcap:
+                s = softcap * torch.tanh(s / softcap)
+            p = torch.arange(n - (hi - lo), n, device=q.device)[:, None]
+            seen = t[None, :] <= p
+            if chunk:
+                seen = seen & (torch.div(t[None, :], chunk, rounding_mode="floor") == torch.div(p, chunk, rounding_mode="floor"))
+            w = torch.softmax(s.masked_fill(~seen, float("-inf")), -1)
+            o = torch.einsum("hnt,thd->nhd", w, v)
+            if gate is not None:
+                o = o * torch.sigmoid(_f(gate[lo:hi]))[..., None]
+            out[lo:hi, :, :vdim] = o.to(q.dtype)
+        return out.view(N, H * cols)
+
+    def delta_rule(self, rows, H, G, d, dv, conv, a_log, dt_bias, norm, eps, state, ring, slots, cu_seqlens, ctx_lens, max_q):
+        """Gated delta rule over packed tokens.  ``rows[N, *]`` hold ``q [G, d] | k [G, d] | v [H, dv] | gate [H, dv] | b [H] |
+        a [H]``, each part starting at a multiple of eight columns; ``conv[2 G d + H dv, taps]`` are the short convolutions of q, k and v.  Sequence
+        ``i`` owns rows ``cu_seqlens[i:i+2]`` (None: row ``i``), the last of its ``ctx_lens[i]`` tokens, and continues from
+        ``state[slots[i]]`` (``[H, d, dv'>=dv]`` fp32) and ``ring[slots[i]]`` (``[H, taps - 1, 2 d + dv]``, the convolutions' last inputs);
+        both are replaced.  A sequence that starts here starts from zero; a negative slot keeps nothing.  Per head
+
+            S = g S;  u = beta (v - S^T k);  S = S + k u^T;  o = S^T q
+
+        with ``g = exp(-exp(a_log) softplus(a + dt_bias))``, ``beta = sigmoid(b)`` and unit vectors ``k``, ``q sqrt(d)``.  Returns
+        ``rms(o) * norm * silu(gate)``, ``[N, H * dv]`` with rows padded to a multiple of eight."""
+        N, taps = rows.shape[0], conv.shape[1]
+        up8 = lambda n: (n + 7) // 8 * 8
+        rep = H // G
+        starts = [0]
+        for n in (G * d, G * d, H * dv, H * dv, H, H):
+            starts.append(starts[-1] + up8(n))
+        part = lambda i, n: _f(rows[:, starts[i]: starts[i] + n])
+        heads = lambda z: z.reshape(-1, G, d).repeat_interleave(rep, 1)
+        raw = torch.cat([heads(part(0, G * d)), heads(part(1, G * d)), part(2, H * dv).reshape(N, H, dv)], -1)      # [N, H, 2 d + dv]
+        w = torch.cat([conv[: G * d].view(G, d, taps).repeat_interleave(rep, 0), conv[G * d: 2 * G * d].view(G, d, taps).repeat_interleave(rep, 0),
+                       conv[2 * G * d:].view(H, dv, taps)], 1)                                                      # [H, 2 d + dv, taps]
+        gate, beta = part(3, H * dv).reshape(N, H, dv), torch.sigmoid(part(4, H))
+        g = torch.exp(-torch.exp(a_log) * F.softplus(part(5, H) + dt_bias))
+        out = torch.zeros(N, up8(H * dv), device=rows.device, dtype=rows.dtype)
+        cu = cu_seqlens.tolist() if cu_seqlens is not None else list(range(N + 1))
+        for i, (slot, ctx) in enumerate(zip(slots.tolist(), ctx_lens.tolist())):
+            lo, hi = cu[i], cu[i + 1]
+            fresh = slot < 0 or ctx == hi - lo
+            past = torch.zeros(taps - 1, H, 2 * d + dv) if fresh else _f(ring[slot, :, : taps - 1]).transpose(0, 1)
+            S = torch.zeros(H, d, dv) if fresh else state[slot, :, :, :dv].clone()
+            z = torch.cat([past, raw[lo:hi]])
+            c = F.silu(sum(z[j: j + hi - lo] * w[:, :, j] for j in range(taps)))
+            unit = lambda t: t * torch.rsqrt(t.pow(2).sum(-1, keepdim=True) + 1e-6)
+            q, k, v = unit(c[..., :d]) * d ** -0.5, unit(c[..., d: 2 * d]), c[..., 2 * d:]
+            for t in range(hi - lo):
+                S = g[lo + t][:, None, None] * S
+                u = beta[lo + t][:, None] * (v[t] - torch.einsum("hdv,hd->hv", S, k[t]))
+                S = S + k[t][:, :, None] * u[:, None, :]
+                o = torch.einsum("hdv,hd->hv", S, q[t])
+                o = o * torch.rsqrt(o.pow(2).mean(-1, keepdim=True) + eps) * norm * F.silu(gate[lo + t])
+                out[lo + t, : H * dv] = o.reshape(-1).to(rows.dtype)
+            if slot >= 0:
+                state[slot, :, :, :dv] = S
+                if taps > 1:
+                    ring[slot, :, : taps - 1] = z[z.shape[0] - taps + 1:].transpose(0, 1).to(ring.dtype)
+        return out
 
     def softcap_(self, logits, cap: float):
         """``cap * tanh(logits / cap)`` in place."""

@@ -58,6 +58,8 @@ class Request:
     finish_reason: str = ""
     slot: int = -1                       # row of the engine's seen-token bitmap (repetition penalty)
     prev: int = -1                       # the last token that is in the cache (-1: none): part of the sequence's state
+    state: int = -1                      # slot of the recurrent layers' states (families that have them)
+    freed: int = 0                       # leading pages that were given back because no later token sees them
 
 
 def request_seed(r: Request) -> int:
@@ -98,12 +100,12 @@ class ServingEngine:
         self.cfg = model.config
         self.ops = ops or get_ops(self.device)
         self.tp = tp                                  # tensor-parallel helper (``serve.tp``) or None
+        self.max_batch = max_batch
+        self.max_ctx = max_ctx or self.cfg.max_position_embeddings
         self.runner = make_runner(self)
         self.arena = getattr(self.runner, "arena", None)
         self.H, self.KV = getattr(self.runner, "H", None), getattr(self.runner, "KV", None)     # local heads, where one number describes all layers
         cfg = self.cfg
-        self.max_ctx = max_ctx or cfg.max_position_embeddings
-        self.max_batch = max_batch
         if prefill_portion and not self.runner.continues:
             raise ValueError(f"{type(self.runner).__name__} prefills whole prompts only")
         self.prefill_portion = prefill_portion        # most tokens of one prompt per prefill pass; 0: the whole prompt
@@ -199,10 +201,14 @@ class ServingEngine:
             batch.cu_context = torch.tensor([0] + np.cumsum(ctx).tolist(), dtype=torch.int32).to(dev)
             batch.total_context = sum(ctx)
             batch.max_ctx = max(ctx)
+            batch.spans = [(r.ctx_len, n) for (r, _), n in zip(parts, ns)]
+        if self.cache.num_states:
+            batch.states = torch.tensor([r.state for r, _ in parts], dtype=torch.int32).to(dev)
         logits = self.runner.forward(batch)
         for (r, toks), n in zip(parts, ns):
             r.ctx_len += n
             r.prev = int(toks[-1])
+            self._trim(r)
         self.stats["prefill_tokens"] += total
         self.stats["prefill_passes"] += 1
         return logits
@@ -232,12 +238,13 @@ class ServingEngine:
         while self.waiting and len(self.running) < self.max_batch:
             r = self.waiting[0]
             need = self.cache.pages_for(min(len(r.prompt) + r.params.max_new_tokens, self.max_ctx))
-            if not self.cache.can_allocate(need):
+            if not self.cache.can_allocate(need) or not self.cache.can_take_state():
                 break
             # pages are handed out in admission order, which is also the order of the decode batch:
             # neighbouring requests of a decode step then read neighbouring pages
             r.pages = self.cache.allocate(need)
             r.slot = self._free_slots.pop()
+            r.state = self.cache.take_state()
             if r.params.repetition_penalty != 1.0:
                 self._init_seen(r)
             self.waiting.pop(0)
@@ -267,10 +274,21 @@ class ServingEngine:
             np.bitwise_or.at(words, ids >> 5, (np.uint32(1) << (ids & 31).astype(np.uint32)))
         self.seen[r.slot].copy_(torch.from_numpy(words.view(np.int32)), non_blocking=True)
 
+    def _trim(self, r: Request) -> None:
+        """Gives back the pages in front of everything that later tokens of the sequence can see (their numbers stay in
+        the page table, where nothing reads them)."""
+        first = self.runner.first_visible(r.ctx_len) // PAGE if self.runner.continues else 0
+        if first > r.freed:
+            self.cache.release(r.pages[r.freed:first])
+            r.freed = first
+
     def _release(self, r: Request) -> None:
         if r.pages:
-            self.cache.release(r.pages)
-            r.pages = []
+            self.cache.release(r.pages[r.freed:])
+            r.pages, r.freed = [], 0
+        if r.state >= 0:
+            self.cache.give_state(r.state)
+            r.state = -1
         if r.slot >= 0:
             self._free_slots.append(r.slot)
             r.slot = -1
@@ -295,10 +313,12 @@ class ServingEngine:
         st = self._dec_states.get(B)
         if st is None:
             # ids | slots (int64), pos | ctx (int32) and, for families whose embedding looks at it, the token before
-            # (int32) live in ONE device buffer with a pinned host twin: a decode step costs one host -> device copy
-            # of 24 (28) bytes per request
+            # (int32) and, for families with recurrent layers, the state slot (int32) live in ONE device buffer with a
+            # pinned host twin: a decode step costs one host -> device copy of 24 (28, 32) bytes per request
             dev = self.device
-            width = 28 if self.runner.needs_prev else 24
+            at_prev = 24 if self.runner.needs_prev else None
+            at_state = (28 if self.runner.needs_prev else 24) if self.cache.num_states else None
+            width = 24 + 4 * (at_prev is not None) + 4 * (at_state is not None)
             packed = torch.zeros(width * B, dtype=torch.uint8, device=dev)
             host = torch.zeros(width * B, dtype=torch.uint8, pin_memory=dev.type == "cuda")
             cut = lambda t, lo, hi, dt: t[lo * B: hi * B].view(dt)
@@ -307,8 +327,10 @@ class ServingEngine:
                   "pos": cut(packed, 16, 20, torch.int32), "ctx": cut(packed, 20, 24, torch.int32),
                   "h_ids": cut(host, 0, 8, torch.long).numpy(), "h_slots": cut(host, 8, 16, torch.long).numpy(),
                   "h_pos": cut(host, 16, 20, torch.int32).numpy(), "h_ctx": cut(host, 20, 24, torch.int32).numpy(),
-                  "prev": cut(packed, 24, 28, torch.int32) if width == 28 else None,
-                  "h_prev": cut(host, 24, 28, torch.int32).numpy() if width == 28 else None,
+                  "prev": cut(packed, at_prev, at_prev + 4, torch.int32) if at_prev else None,
+                  "h_prev": cut(host, at_prev, at_prev + 4, torch.int32).numpy() if at_prev else None,
+                  "states": cut(packed, at_state, at_state + 4, torch.int32) if at_state else None,
+                  "h_states": cut(host, at_state, at_state + 4, torch.int32).numpy() if at_state else None,
                   "table": torch.zeros(B, self.max_pages_per_req, dtype=torch.int32, device=dev),
                   "rows": torch.arange(B, device=dev), "idx": np.arange(B), "graphs": {}}
             self._dec_states[B] = st
@@ -326,6 +348,8 @@ class ServingEngine:
         st["h_ctx"][:] = lens + 1
         if st["h_prev"] is not None:
             st["h_prev"][:] = np.fromiter((r.prev for r in reqs), dtype=np.int32, count=B)
+        if st["h_states"] is not None:
+            st["h_states"][:] = np.fromiter((r.state for r in reqs), dtype=np.int32, count=B)
         st["packed"].copy_(st["host"], non_blocking=True)
         return st
 
@@ -339,14 +363,18 @@ class ServingEngine:
         # grid of the split-KV kernel, where the family's attention kernel is launched for a context size
         bucket = min(self.max_ctx, ((max_ctx + 511) // 512) * 512) if self.runner.context_buckets else self.max_ctx
         batch = Batch(ids=st["ids"], positions=st["pos"], slots=st["slots"], rows=st["rows"], prev=st["prev"],
-                      page_table=st["table"], ctx_lens=st["ctx"], max_ctx=bucket, decode=True)
+                      states=st["states"], page_table=st["table"], ctx_lens=st["ctx"], max_ctx=bucket, decode=True)
         toks = None
         if self.device.type == "cuda" and self.use_cuda_graphs:
             g = st["graphs"].get(bucket)
             if g is None:
-                # one eager pass first: lazy initialisation must not happen under capture
+                # one eager pass first: lazy initialisation must not happen under capture.  It must not advance the
+                # recurrent states either: they are detached (slot -1) until the replay
+                if st["states"] is not None:
+                    st["states"].fill_(-1)
                 self.runner.forward(batch)
                 torch.cuda.synchronize()
+                st["packed"].copy_(st["host"])
                 graph = torch.cuda.CUDAGraph()
                 # the captured launches are programmatic dependents of one another (the graph keeps the edges)
                 with torch.cuda.graph(graph), self.ops.dependent_launch(self.dependent_launch):
@@ -367,6 +395,7 @@ class ServingEngine:
         for r, t in zip(reqs, tokens):
             r.ctx_len += 1
             r.prev = int(t)
+            self._trim(r)
         self.stats["decode_tokens"] += len(reqs)
         return logits, toks
 
@@ -411,6 +440,8 @@ class ServingEngine:
             more = self.cache.pages_for(n) - len(r.pages)
             if more > 0:
                 r.pages = r.pages + self.cache.allocate(more)
+            if r.state < 0:
+                r.state = self.cache.take_state()
         out: list[Any] = [None] * len(entries)
         single = [i for i, (r, toks, _) in enumerate(entries) if len(toks) == 1 and r.ctx_len > 0]
         packed = [i for i in range(len(entries)) if i not in set(single)]

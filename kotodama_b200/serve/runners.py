@@ -3,7 +3,8 @@ serving engine.
 
 A runner has ``make_cache(pages)``, ``forward(batch) -> logits[rows]`` and three traits: ``continues`` (a pass may
 start from a cached context), ``needs_prev`` (the embedding looks at the token before) and ``context_buckets`` (the decode
-attention is launched for a context size, so decode graphs are captured per size).
+attention is launched for a context size, so decode graphs are captured per size).  A runner that continues also has
+``first_visible(n)``: the first position that tokens from position ``n`` on can still see.
 """
 from __future__ import annotations
 
@@ -13,9 +14,10 @@ from typing import Any, Optional
 import torch
 
 from ..engine import ParamArena
+from ..models.lisunex import AttentionMixer, DeltaMixer, LisunexModel
 from ..models.registry import family_of
 from ..models.vunitar import DenseMLP, MoEMLP, VunitarModel
-from .cache import PagedKVCache, PagedLatentCache
+from .cache import HybridCache, PagedKVCache, PagedLatentCache
 
 
 @dataclass
@@ -35,6 +37,8 @@ class Batch:
     max_ctx: int = 0
     cu_context: Optional[torch.Tensor] = None      # [B + 1] prefix sums of ctx_lens
     total_context: int = 0
+    states: Optional[torch.Tensor] = None          # [B] int32 state slot of every sequence (-1: its state is not kept)
+    spans: Optional[list[tuple[int, int]]] = None  # per sequence (tokens in the cache before, new tokens); not for decode
 
 
 def make_runner(engine: Any) -> Any:
@@ -214,6 +218,9 @@ class LatentRunner:
         out[tuple(slice(0, n) for n in t.shape)] = t
         return out
 
+    def first_visible(self, n: int) -> int:
+        return 0
+
     def make_cache(self, pages: int) -> PagedLatentCache:
         widths = [lw["R"] for lw in self.layers]
         self.cache = PagedLatentCache(widths, [self.ops.latent_block(self.dtype, w) for w in widths], pages, self.device, self.dtype)
@@ -265,3 +272,150 @@ class LatentRunner:
         n = ops.norm_rows(x, b.rows, self.final, self.D, eps, h.dtype)
         logits = ops.gemm_nt(n, self.head, out=torch.empty(n.shape[0], cfg.vocab_size, device=n.device, dtype=torch.float32))
         return ops.softcap_(logits, cfg.logit_softcap) if cfg.logit_softcap else logits
+
+
+class HybridRunner:
+    """Pre-norm decoder whose layers mix tokens by grouped attention (optionally inside chunks of the sequence) or by a
+    gated delta rule, some of them run several times (``models/lisunex.py``).
+
+    The residual stream is fp32; a sub-layer's output is added by the norm in front of the next one.  Attention layers keep keys
+    and values in pages, delta layers a matrix state and the last convolution inputs per sequence; every run of a looped layer has
+    its own.  Attention takes one of two forms:
+
+    * decoding and short portions read the paged cache where it lies;
+    * in long portions every chunk of a sequence is a packed sequence of its own for the flash kernel, its queries the last of the
+      chunk's positions so far; keys of the chunk that an earlier pass left are gathered in front of the new ones.
+    """
+
+    continues = True
+    needs_prev = False
+
+    def __init__(self, eng: Any) -> None:
+        if eng.tp is not None:
+            raise ValueError("hybrid models are served on one GPU")
+        self.ops, self.device, self.dtype = eng.ops, eng.device, eng.dtype
+        self.max_ctx, self.max_states = eng.max_ctx, eng.max_batch
+        model: LisunexModel = eng.model
+        cfg = self.cfg = model.config
+        self.D, self.short_portion = cfg.hidden_size, 16
+        Dp = self.Dp = _up(self.D, 8)
+        pad = LatentRunner._pad
+        w = model.weights
+        f32 = lambda t: t.to(self.device, torch.float32).contiguous()
+        put = lambda t: t.to(self.device, self.dtype)
+        vec = lambda t: pad(f32(t), Dp)
+        dw = self.ops.decode_weight
+        # one product for everything that reads the layer's input: the parts start at multiples of eight rows
+        fuse = lambda parts: torch.cat([pad(put(t), _up(t.shape[0], 8), Dp) for t in parts])
+        self.embed = pad(put(w["embed"]), cfg.vocab_size, Dp)
+        self.steps = [vec(t) for t in w["loop.step"]] if cfg.loop else []
+        tables: dict[Any, tuple[torch.Tensor, torch.Tensor]] = {}
+        self.layers: list[dict[str, Any]] = []
+        for i, layer in enumerate(cfg.layers):
+            p, m = f"l{i}.", layer.mixer
+            x = lambda n: w[p + "mix." + n]
+            lw: dict[str, Any] = dict(m=m, norm1=vec(w[p + "norm1"]), delta=isinstance(m, DeltaMixer))
+            if isinstance(m, AttentionMixer):
+                lw["hd"] = hd = self.ops.flash_heads(self.dtype, m.dim, m.vdim)
+                lw.update(kd=hd or _up(m.dim, 8), vd=hd or _up(m.vdim, 8), cols=_up(m.vdim, 8))
+                if m.rot not in tables:
+                    tables[m.rot] = tuple(t.to(self.device).contiguous() for t in m.rot.table(self.max_ctx))
+                lw["win"] = dw(fuse([x("q"), x("k"), x("v"), x("g")]))
+                lw["bias"] = torch.cat([pad(put(b), _up(b.shape[0], 8)) for b in (x("q.b"), x("k.b"), x("v.b"), torch.zeros(m.heads))])
+                lw["cs"] = tables[m.rot]
+                lw["gate"] = _up(m.heads * m.dim, 8) + _up(m.kv_heads * m.dim, 8) + _up(m.kv_heads * m.vdim, 8)
+                o = pad(put(x("o")).view(self.D, m.heads, m.vdim), Dp, m.heads, lw["cols"])
+                lw["wo"] = dw(o.reshape(Dp, m.heads * lw["cols"]))
+            else:
+                lw["win"] = dw(fuse([x("q"), x("k"), x("v"), x("g"), x("b"), x("a")]))
+                lw["conv"] = torch.cat([f32(x(n + ".conv")) for n in "qkv"])
+                lw.update(a_log=f32(x("A_log")), dt=f32(x("dt_bias")), norm=f32(x("norm")))
+                lw["wo"] = dw(pad(put(x("o")), Dp, _up(m.heads * m.vdim, 8)))
+            if layer.mlp is not None:
+                fp = _up(layer.mlp.ff, 8)
+                lw.update(norm2=vec(w[p + "norm2"]), wgu=dw(fuse([w[p + "mlp.gate"], w[p + "mlp.up"]])),
+                          wd=dw(pad(put(w[p + "mlp.down"]), Dp, fp)))
+            self.layers.append(lw)
+        self.final = vec(w["final.norm"])
+        self.head = pad(put(w["head"]), cfg.vocab_size, Dp)
+        self.runs = cfg.runs()
+        self.chunks = {lw["m"].chunk for lw in self.layers if not lw["delta"]}
+        self.context_buckets = 0 in self.chunks
+        self.cache: Any = None
+        self.layer_trace: Optional[list] = None      # when a list: the residual stream after every layer run is appended
+
+    def first_visible(self, n: int) -> int:
+        return min((n // c * c if c else 0 for c in self.chunks), default=n)
+
+    def make_cache(self, pages: int) -> HybridCache:
+        kv, rec = [], []
+        for i, _ in self.runs:
+            lw, m = self.layers[i], self.layers[i]["m"]
+            kv.append(None if lw["delta"] else (m.kv_heads, lw["kd"], lw["vd"]))
+            rec.append((m.heads, m.dim, m.vdim, m.taps) if lw["delta"] else None)
+        self.cache = HybridCache(kv, rec, pages, self.max_states, self.device, self.dtype)
+        return self.cache
+
+    def _segments(self, b: Batch, chunk: int) -> dict[str, Any]:
+        """The chunks (0: whole contexts) that the batch's queries lie in, as packed sequences."""
+        cq, ck, seq, first = [0], [0], [], []
+        cached = False
+        for i, (start, n) in enumerate(b.spans):
+            at = start
+            while at < start + n:
+                lo = at // chunk * chunk if chunk else 0
+                end = min(start + n, lo + chunk) if chunk else start + n
+                cached |= lo < start
+                seq.append(i)
+                first.append(lo)
+                cq.append(cq[-1] + end - at)
+                ck.append(ck[-1] + end - lo)
+                at = end
+        t = lambda v: torch.tensor(v, dtype=torch.int32).to(self.device)
+        return dict(cq=t(cq), ck=t(ck), seq=t(seq), first=t(first), total=ck[-1], cached=cached, max_q=max(y - x for x, y in zip(cq, cq[1:])))
+
+    def _attention(self, h: torch.Tensor, lw: dict, run: int, b: Batch, segments: dict) -> torch.Tensor:
+        ops, m, N = self.ops, lw["m"], h.shape[0]
+        rows = ops.gemm_nt(h, lw["win"], residual=lw["bias"].expand(N, -1))
+        kp, vp = self.cache.k[run], self.cache.v[run]
+        packed = lw["hd"] > 0 and not b.decode and b.max_seqlen > self.short_portion
+        if packed and m.chunk not in segments:
+            segments[m.chunk] = self._segments(b, m.chunk)
+        s = segments.get(m.chunk)
+        q, k, v = ops.head_rotary_norm(rows, m.heads, m.kv_heads, m.dim, m.vdim, *lw["cs"], b.positions, self.cfg.norm_eps, kp, vp, b.slots,
+                                       packed and not s["cached"])
+        gate = rows[:, lw["gate"]: lw["gate"] + m.heads]
+        if not packed:
+            return ops.paged_attention(q, kp, vp, b.page_table, b.ctx_lens, b.cu_seqlens, b.max_ctx, m.scale, m.softcap, m.chunk, gate,
+                                       m.vdim, lw["cols"])
+        if s["cached"]:
+            k, v = ops.kv_gather(kp, vp, b.page_table, s["seq"], s["first"], s["ck"], s["total"])
+        # unit-RMS queries and keys: |q . k| <= dim (rounding of the two included)
+        bound = 1.02 * m.dim * abs(m.scale)
+        return ops.attention_context(q, k, v, s["cq"], s["ck"], s["max_q"], m.scale, m.softcap, gate, lw["cols"], bound).view(N, -1)
+
+    def _delta(self, h: torch.Tensor, lw: dict, run: int, b: Batch) -> torch.Tensor:
+        m = lw["m"]
+        return self.ops.delta_rule(self.ops.gemm_nt(h, lw["win"]), m.heads, m.kv_heads, m.dim, m.vdim, lw["conv"], lw["a_log"], lw["dt"],
+                                   lw["norm"], self.cfg.norm_eps, self.cache.state[run], self.cache.ring[run], b.states, b.cu_seqlens,
+                                   b.ctx_lens, b.max_seqlen)
+
+    @torch.no_grad()
+    def forward(self, b: Batch) -> torch.Tensor:
+        ops, cfg = self.ops, self.cfg
+        eps, D = cfg.norm_eps, self.D
+        x, _ = ops.embed_pairs(b.ids, None, self.embed, None, (0, 0, 0), cfg.embedding_scale)
+        y = None
+        segments: dict[int, dict] = {}
+        for run, (i, t) in enumerate(self.runs):
+            lw = self.layers[i]
+            h = ops.add_norm(x, y, None if t is None else self.steps[t], lw["norm1"], D, eps, self.dtype)
+            o = self._delta(h, lw, run, b) if lw["delta"] else self._attention(h, lw, run, b, segments)
+            y = ops.gemm_nt(o, lw["wo"])
+            if "wd" in lw:
+                h = ops.add_norm(x, y, None, lw["norm2"], D, eps, self.dtype)
+                y = ops.gemm_nt(ops.swiglu_fwd(ops.gemm_nt(h, lw["wgu"])), lw["wd"])
+            if self.layer_trace is not None:
+                self.layer_trace.append((x + y.float())[:, :D].cpu())
+        n = ops.add_norm(x, y, None, self.final, D, eps, self.dtype, rows=b.rows)
+        return ops.gemm_nt(n, self.head, out=torch.empty(n.shape[0], cfg.vocab_size, device=n.device, dtype=torch.float32))

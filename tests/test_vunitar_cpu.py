@@ -121,7 +121,7 @@ def test_model_folders_load_by_architecture(tmp_path):
     assert torch.equal(load_model(lf).embed_tokens.weight, lm.embed_tokens.weight)
     with pytest.raises(ValueError):
         read_config(write_model(tmp_path / "x", {"architecture": "other"}, {"a": torch.zeros(1)}))
-    assert set(FAMILIES) == {"Kotodama", "Vunitar"}
+    assert {"Kotodama", "Vunitar"} <= set(FAMILIES)
 
 
 def test_wrong_weights_and_configurations_are_refused(tmp_path):
