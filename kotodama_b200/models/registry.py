@@ -54,7 +54,7 @@ FAMILIES: dict[str, Family] = {
                        "latent_attn", "latent_attn_sm100", "moe", "gemm_grouped_sm100", "gemm_f32", "block")),
     "Lisunex": Family(LisunexConfig.from_dict, LisunexModel, LisunexModel.random_init, LisunexModel, "HybridRunner",
                       ("elementwise", "serve", "sampler", "attn_sm100", "gemm_sm100", "gemm2_sm100", "gemm_skinny_sm100",
-                       "gemm_f32", "block", "paged_attn", "delta")),
+                       "gemm_f32", "block", "paged_attn", "delta", "delta_sm100")),
 }
 
 

@@ -22,7 +22,7 @@ OBJ_DIR = ROOT / "build" / "obj"
 NVCC_FLAGS = ["-gencode", "arch=compute_100a,code=sm_100a", "-lineinfo", "-O3", "-std=c++17",
               "-Xcompiler", "-fPIC", "-Xcompiler", "-fvisibility=hidden"]
 # sources of the 32-bit mode (and of fp32 statistics) keep IEEE division, square roots and full-precision functions
-PRECISE = {"block", "moe", "gemm_f32", "latent_attn", "paged_attn", "delta"}
+PRECISE = {"block", "moe", "gemm_f32", "latent_attn", "paged_attn", "delta", "delta_sm100"}
 
 _lib = None
 

@@ -72,6 +72,9 @@ class CudaOps(TorchOps):
                      "kb_route_blocked_grid"):
             if hasattr(self.lib, name):          # a library of the serving kernels alone does not have the training ones
                 getattr(self.lib, name).restype = _I
+        for name in ("kb_delta_chunk_tt_bytes", "kb_delta_chunk_scalars"):
+            if hasattr(self.lib, name):
+                getattr(self.lib, name).restype = _LL
 
     # ------------------------------------------------------------------ utils
     def _rc(self, rc: int, what: str) -> None:
@@ -896,16 +899,31 @@ class CudaOps(TorchOps):
                    _I(_TYPE[q.dtype]), _p(self.status(q.device)), _st())
         return out
 
+    delta_short = 16        # most tokens of a sequence in one pass for which the recurrence is walked token by token
+
     def delta_rule(self, rows, H, G, d, dv, conv, a_log, dt_bias, norm, eps, state, ring, slots, cu_seqlens, ctx_lens, max_q):
         N = rows.shape[0]
         up8 = lambda n: (n + 7) // 8 * 8
         cols = [0]
         for n in (G * d, G * d, H * dv, H * dv, H):
             cols.append(cols[-1] + up8(n))
-        width = up8(H * dv)
-        out = (torch.empty if width == H * dv else torch.zeros)(N, width, device=rows.device, dtype=rows.dtype)
+        width, taps, B, dev = up8(H * dv), conv.shape[1], slots.numel(), rows.device
+        out = (torch.empty if width == H * dv else torch.zeros)(N, width, device=dev, dtype=rows.dtype)
+        if (rows.dtype == torch.bfloat16 and cu_seqlens is not None and max_q > self.delta_short
+                and self.lib.kb_delta_chunk_ok(_I(H), _I(G), _I(d), _I(dv), _I(taps))):
+            D, dvt = 64 if d <= 64 else 128, (dv + 63) // 64 * 64
+            buf = lambda n, exact: (torch.empty if exact else torch.zeros)(N, n, device=dev, dtype=rows.dtype)
+            q, k, v, o = buf(G * D, d == D), buf(G * D, d == D), buf(H * dvt, dv == dvt), buf(H * dvt, True)
+            tt = torch.empty(self.lib.kb_delta_chunk_tt_bytes(_I(N), _I(B), _I(H)), device=dev, dtype=torch.uint8)
+            scal = torch.empty(self.lib.kb_delta_chunk_scalars(_I(N), _I(B), _I(H)), device=dev, dtype=torch.float32)
+            self._call("kb_delta_chunks", _p(rows), _LL(rows.stride(0)), *map(_I, cols), _p(conv), _p(a_log), _p(dt_bias), _p(norm), _I(taps),
+                       _I(N), _I(B), _I(H), _I(G), _I(d), _I(dv), _I(D), _I(dvt), _I(state.shape[3]), _F(eps), _p(state), _p(ring),
+                       _I(ring.shape[2]), _I(state.shape[0]), _p(slots), _p(cu_seqlens), _p(ctx_lens), _p(q), _p(k), _p(v), _p(o), _p(tt),
+                       _p(scal), _p(out), _LL(width), _p(self.status(dev)), _st())
+            self.launches += 4 - (taps == 1)
+            return out
         self._call("kb_delta_step", _p(rows), _LL(rows.stride(0)), *map(_I, cols), _p(conv), _p(a_log), _p(dt_bias), _p(norm),
-                   _I(conv.shape[1]), _I(H), _I(G), _I(d), _I(dv), _I(state.shape[3]), _F(eps), _p(state), _p(ring), _I(ring.shape[2]),
+                   _I(taps), _I(H), _I(G), _I(d), _I(dv), _I(state.shape[3]), _F(eps), _p(state), _p(ring), _I(ring.shape[2]),
                    _I(state.shape[0]), _p(slots), _p(cu_seqlens), _p(ctx_lens), _I(slots.numel()), _p(out), _LL(width), _I(_TYPE[rows.dtype]),
                    _p(self.status(rows.device)), _st())
         return out
