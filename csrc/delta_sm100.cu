@@ -30,7 +30,7 @@ constexpr int CH = 64;                             // tokens per chunk
 constexpr int BLK = CH * 128;                      // a 64-row block of 128-byte rows: 8 KB
 constexpr int TT_BYTES = 4 * BLK;                  // [T; A T] upper halves, then lower halves
 constexpr int SCALARS = 3 * CH + 8;                // per (chunk, head): e^G r_k | e^G r_q | e^(G_64 - G) r_k | e^G_64
-constexpr int LP = 68;                             // pitch (floats) of the fp32 matrices
+constexpr int LP = 36, TB = 32 * LP;               // pitch and size (floats) of a 32 x 32 fp32 block
 
 struct ChunkParams {
     int N, B, H, G, d, dv, dvt, dvp;               // dvt: columns per head of v and o (a multiple of 64), dvp: of the state
@@ -51,12 +51,14 @@ struct ChunkParams {
 // Chunk c of sequence b has slot cu[b] / 64 + b + c: slots of different sequences never meet, and N / 64 + B of them suffice.
 __device__ __forceinline__ int slot_base(const int* cu, int b) { return cu[b] / CH + b; }
 
-__device__ __forceinline__ float silu(float z) { return z / (1.0f + expf(-z)); }
+// results are rounded to bf16 where this is used
+__device__ __forceinline__ float silu(float z) { return __fdividef(z, 1.0f + __expf(-z)); }
 
-// 64 numbers of a row as two bf16 numbers each, to row `row` of two 128-byte-swizzled tiles
-__device__ __forceinline__ void store_row_split(uint8_t* hi, uint8_t* lo, int row, const float* x) {
+// 8 * CHUNKS numbers of a row as two bf16 numbers each, from 16-byte chunk `c0` on, to row `row` of two 128-byte-swizzled tiles
+template <int CHUNKS>
+__device__ __forceinline__ void store_row_split(uint8_t* hi, uint8_t* lo, int row, int c0, const float* x) {
 #pragma unroll
-    for (int c = 0; c < 8; ++c) {
+    for (int c = 0; c < CHUNKS; ++c) {
         uint32_t h[4], l[4];
 #pragma unroll
         for (int j = 0; j < 4; ++j) {
@@ -66,7 +68,7 @@ __device__ __forceinline__ void store_row_split(uint8_t* hi, uint8_t* lo, int ro
             h[j] = *reinterpret_cast<const uint32_t*>(&u);
             l[j] = attn::pack_bf16(a - f.x, b - f.y);
         }
-        const int at = row * 128 + ((c ^ (row & 7)) << 4);
+        const int at = row * 128 + (((c0 + c) ^ (row & 7)) << 4);
         *reinterpret_cast<uint4*>(hi + at) = make_uint4(h[0], h[1], h[2], h[3]);
         *reinterpret_cast<uint4*>(lo + at) = make_uint4(l[0], l[1], l[2], l[3]);
     }
@@ -75,6 +77,16 @@ __device__ __forceinline__ void tmem_row64(uint32_t taddr, float* x) {
     tc::tmem_ld32(taddr, reinterpret_cast<uint32_t*>(x));
     tc::tmem_ld32(taddr + 32, reinterpret_cast<uint32_t*>(x + 32));
     tc::tmem_ld_wait();
+}
+__device__ __forceinline__ void tmem_row32(uint32_t taddr, float* x) {
+    tc::tmem_ld32(taddr, reinterpret_cast<uint32_t*>(x));
+    tc::tmem_ld_wait();
+}
+// 2^x by the special-function unit (relative error 2^-22)
+__device__ __forceinline__ float ex2(float x) {
+    float y;
+    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+    return y;
 }
 __device__ __forceinline__ void bulk_load(void* dst, const void* src, uint32_t bytes, uint64_t* bar) {
     asm volatile("cp.async.bulk.shared::cta.global.mbarrier::complete_tx::bytes [%0], [%1], %2, [%3];" ::"r"(smem_u32(dst)),
@@ -104,73 +116,97 @@ __device__ __forceinline__ void mma_steps(uint32_t d, uint32_t a_addr, uint32_t 
 }
 
 // ------------------------------------------------------------------------------------------------ prepare
-constexpr int PREP_SMEM = 4 * BLK + 2 * BLK + CH * LP * 4 + 1024;
+// A (16 KB); [K; Q] (32 KB), which gives way to the fp32 blocks of L and X and then to T
+constexpr int PREP_SMEM = 6 * BLK + 1024;
+
+// acc[0 .. 4 Q) = a row of a product of two blocks: sum over m < M of A[m] B[m][0 .. 4 Q)
+template <int M, int Q>
+__device__ __forceinline__ void block_row(const float* A, const float* B, float* acc) {
+#pragma unroll
+    for (int j = 0; j < 4 * Q; ++j) acc[j] = 0.f;
+#pragma unroll
+    for (int m = 0; m < M; m += 4) {
+        const float4 a4 = *reinterpret_cast<const float4*>(A + m);
+        const float a[4] = {a4.x, a4.y, a4.z, a4.w};
+#pragma unroll
+        for (int e = 0; e < 4; ++e)
+#pragma unroll
+            for (int q = 0; q < Q; ++q) {
+                const float4 b = *reinterpret_cast<const float4*>(B + (m + e) * LP + 4 * q);
+                acc[4 * q] = fmaf(a[e], b.x, acc[4 * q]);
+                acc[4 * q + 1] = fmaf(a[e], b.y, acc[4 * q + 1]);
+                acc[4 * q + 2] = fmaf(a[e], b.z, acc[4 * q + 2]);
+                acc[4 * q + 3] = fmaf(a[e], b.w, acc[4 * q + 3]);
+            }
+    }
+}
 
 template <int D>
-__global__ void __launch_bounds__(128)
+__global__ void __launch_bounds__(128, 4)
 delta_prepare_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constant__ CUtensorMap tmQ, const ChunkParams p) {
     extern __shared__ uint8_t smem_raw[];
     uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
-    uint8_t* sA = smem + 4 * BLK;                      // A, upper and lower half; behind [K; Q], which becomes L and then T
-    float* Xs = reinterpret_cast<float*>(sA + 2 * BLK);
-    float* Ls = reinterpret_cast<float*>(smem);
-    float* M1 = Ls + CH * LP;                          // [32][36]
-    uint8_t* sT = smem;
+    uint8_t *sA = smem, *sKQ = smem + 2 * BLK, *sT = sKQ;                  // A and T: upper and lower half
+    // blocks (0, 0), (1, 0), (1, 1) of L, a product, and the same blocks of X = (I + L)^-1; T lies over L
+    float *Lb = reinterpret_cast<float*>(sKQ), *M1 = Lb + 3 * TB, *Xb = M1 + TB;
     __shared__ uint64_t bars[2];
     __shared__ uint32_t tmem_slot;
     __shared__ int abort_flag;
-    __shared__ float gsum[CH], beta[CH], unit[2 * CH];
-    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+    __shared__ __align__(16) float gsum[CH], beta[CH], unit[2 * CH]; // sums of log2 of the decays; step sizes; scalars of the unit norms
+    const int tid = threadIdx.x, warp = __shfl_sync(0xffffffffu, tid >> 5, 0), lane = tid & 31;    // the warp's number is uniform, and known to be
     const int slot = blockIdx.x, head = blockIdx.y, kvh = head / (p.H / p.G);
-    int lo = 0, hi = p.B;
-    while (hi - lo > 1) {
-        const int m = (lo + hi) >> 1;
-        if (slot_base(p.cu, m) <= slot) lo = m; else hi = m;
+    int b = 0;                                         // the last sequence whose slots begin at or in front of this one
+    for (int b0 = 0; b0 < p.B; b0 += 32) {
+        const unsigned in = __ballot_sync(0xffffffffu, b0 + lane < p.B && slot_base(p.cu, b0 + lane) <= slot);
+        if (in) b = b0 + 31 - __clz(in);
+        if (in != 0xffffffffu) break;
     }
-    const int first = p.cu[lo] + (slot - slot_base(p.cu, lo)) * CH;
-    const int valid = min(CH, p.cu[lo + 1] - first);
+    const int first = p.cu[b] + (slot - slot_base(p.cu, b)) * CH;
+    const int valid = min(CH, p.cu[b + 1] - first);
     if (valid <= 0) return;                            // uniform: a slot that no chunk has
     if (tid == 0) {
         tc::mbar_init(&bars[0], 1);
         tc::mbar_init(&bars[1], 1);
         abort_flag = 0;
         tc::fence_barrier_init();
+        load_kq<D>(sKQ, &tmK, &tmQ, &bars[0], kvh, first);
     }
+    __syncwarp();
     if (warp == 0) {
         tc::tmem_alloc(&tmem_slot, 128);
         tc::tmem_relinquish();
     }
-    tc::tc_fence_before();
-    __syncthreads();
-    tc::tc_fence_after();
-    const uint32_t tmem = tmem_slot;
-    bool ok = true;
-    if (tid == 0) {
-        load_kq<D>(smem, &tmK, &tmQ, &bars[0], kvh, first);
-        if (tc::mbar_wait(&bars[0], 0, &abort_flag)) {
-            const uint32_t a = smem_u32(smem);
-            mma_steps<D / 16, 32, 32, true, true>(tmem, a, 16, a, tc::instr_desc_f16(128, CH, 1, 1, 0, 0), false);
-            tc::tc_commit(&bars[1]);
-        }
-    }
-    __syncwarp();
-    if (tid < CH) {                                    // decay logarithms (running sum) and step sizes
+    if (tid >= 64) {                                   // decays (running sum) and step sizes of the tokens
+        const int t = tid - 64;
         float lg = 0.f, be = 0.f;
-        if (tid < valid) {
-            const bf16* row = p.rows + (long long)(first + tid) * p.stride;
+        if (t < valid) {
+            const bf16* row = p.rows + (long long)(first + t) * p.stride;
             const float z = to_float(row[p.col_a + head]) + p.dt_bias[head];
-            lg = -expf(p.a_log[head]) * (z > 20.f ? z : log1pf(expf(z)));
+            lg = -expf(p.a_log[head]) * (z > 20.f ? z : log1pf(expf(z))) * attn::LOG2E;
             be = 1.0f / (1.0f + expf(-to_float(row[p.col_b + head])));
         }
 #pragma unroll
         for (int o = 1; o < 32; o <<= 1) {
-            const float t = __shfl_up_sync(0xffffffffu, lg, o);
-            if (lane >= o) lg += t;
+            const float u = __shfl_up_sync(0xffffffffu, lg, o);
+            if (lane >= o) lg += u;
         }
-        gsum[tid] = lg;
-        beta[tid] = be;
+        gsum[t] = lg;
+        beta[t] = be;
     }
-    ok = tc::mbar_wait(&bars[0], 0, &abort_flag);
+    tc::tc_fence_before();
+    __syncthreads();
+    tc::tc_fence_after();
+    const uint32_t tmem = __shfl_sync(0xffffffffu, tmem_slot, 0), lane_base = (uint32_t)(warp * 32) << 16;
+    bool ok = tc::mbar_wait(&bars[0], 0, &abort_flag);
+    // Products are issued by one elected lane of a whole warp: their operands then stay in uniform registers.
+    if (warp == 0 && __all_sync(0xffffffffu, ok)) {
+        const uint32_t a = smem_u32(sKQ);
+        if (tc::elect_one()) {
+            mma_steps<D / 16, 32, 32, true, true>(tmem, a, 16, a, tc::instr_desc_f16(128, CH, 1, 1, 0, 0), false);
+            tc::tc_commit(&bars[1]);
+        }
+        __syncwarp();
+    }
     {
         float ss = 0.f;                                // row tid of [K; Q]
 #pragma unroll
@@ -178,7 +214,7 @@ delta_prepare_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_const
 #pragma unroll
             for (int c = 0; c < 8; ++c) {
                 float x[8];
-                load8(reinterpret_cast<const bf16*>(smem + h * 2 * BLK + tid * 128 + ((c ^ (tid & 7)) << 4)), x);
+                load8(reinterpret_cast<const bf16*>(sKQ + h * 2 * BLK + tid * 128 + ((c ^ (tid & 7)) << 4)), x);
 #pragma unroll
                 for (int j = 0; j < 8; ++j) ss += x[j] * x[j];
             }
@@ -186,98 +222,117 @@ delta_prepare_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_const
         unit[tid] = (tid & 63) < valid ? (tid < CH ? r : r / sqrtf((float)p.d)) : 0.f;
     }
     ok = tc::mbar_wait(&bars[1], 0, &abort_flag) && ok;
+    if (tid >= 32 && tid < CH) gsum[tid] += gsum[31];
     if (__syncthreads_or(!ok)) {
         if (tid == 0) atomicMax(p.status, (int)KB_TIMEOUT_TMA);
     } else {
-        if (tid >= 32 && tid < CH) gsum[tid] += gsum[31];
-        __syncthreads();
         tc::tc_fence_after();
         const int i = tid & 63;
-        const uint32_t lane_base = (uint32_t)(warp * 32) << 16;
         {
             float x[64];
             tmem_row64(tmem + lane_base, x);
             const float gi = gsum[i], s = tid < CH ? unit[i] * beta[i] : unit[tid];
             const int last = tid < CH ? i - 1 : i;     // columns up to here
 #pragma unroll
-            for (int j = 0; j < 64; ++j) x[j] = j <= last ? x[j] * s * unit[j] * expf(gi - gsum[j]) : 0.f;
+            for (int j = 0; j < 64; j += 4) {
+                const float4 u = *reinterpret_cast<const float4*>(unit + j), g = *reinterpret_cast<const float4*>(gsum + j);
+                x[j] = j <= last ? x[j] * s * u.x * ex2(gi - g.x) : 0.f;
+                x[j + 1] = j + 1 <= last ? x[j + 1] * s * u.y * ex2(gi - g.y) : 0.f;
+                x[j + 2] = j + 2 <= last ? x[j + 2] * s * u.z * ex2(gi - g.z) : 0.f;
+                x[j + 3] = j + 3 <= last ? x[j + 3] * s * u.w * ex2(gi - g.w) : 0.f;
+            }
             if (tid < CH) {
+                float* dst = Lb + (i < 32 ? 0 : TB) + (i & 31) * LP;
 #pragma unroll
-                for (int j = 0; j < 64; j += 4) *reinterpret_cast<float4*>(Ls + i * LP + j) = make_float4(x[j], x[j + 1], x[j + 2], x[j + 3]);
+                for (int j = 0; j < 32; j += 4) *reinterpret_cast<float4*>(dst + j) = make_float4(x[j], x[j + 1], x[j + 2], x[j + 3]);
+                if (i >= 32) {
+#pragma unroll
+                    for (int j = 0; j < 32; j += 4)
+                        *reinterpret_cast<float4*>(dst + TB + j) = make_float4(x[32 + j], x[33 + j], x[34 + j], x[35 + j]);
+                }
             } else {
-                store_row_split(sA, sA + BLK, i, x);
+                store_row_split<8>(sA, sA + BLK, i, 0, x);
             }
         }
         __syncthreads();
-        // inverses of the two triangles on the diagonal: one column per lane, by substitution
-        if (warp < 2) {
-            const float* Lb = Ls + (warp * 32) * LP + warp * 32;
-            float x[32];
+        // inverses of the four 16 x 16 triangles on the diagonal, one per warp: a column per lane, by substitution
+        {
+            const int off = (warp >> 1) * 2 * TB + (warp & 1) * (16 * LP + 16);
+            const float* Lw = Lb + off;
+            float* Xw = Xb + off;
+            float x[16];
 #pragma unroll
-            for (int r = 0; r < 32; ++r) {
+            for (int r = 0; r < 16; ++r) {
                 float s0 = r == lane ? 1.f : 0.f, s1 = 0.f, s2 = 0.f, s3 = 0.f;
 #pragma unroll
                 for (int m = 0; m < r; m += 4) {
-                    const float4 l4 = *reinterpret_cast<const float4*>(Lb + r * LP + m);
+                    const float4 l4 = *reinterpret_cast<const float4*>(Lw + r * LP + m);
                     s0 = fmaf(-l4.x, x[m], s0);
                     if (m + 1 < r) s1 = fmaf(-l4.y, x[m + 1], s1);
                     if (m + 2 < r) s2 = fmaf(-l4.z, x[m + 2], s2);
                     if (m + 3 < r) s3 = fmaf(-l4.w, x[m + 3], s3);
                 }
                 x[r] = (s0 + s1) + (s2 + s3);
-                Xs[(warp * 32 + r) * LP + warp * 32 + lane] = x[r];
+                // lanes 16 .. 31 hold zeros: above the diagonal in an even block's rows, nothing in an odd block's
+                if (lane < 16 || !(warp & 1)) Xw[r * LP + lane] = x[r];
             }
-        } else {
-            for (int e = tid - 64; e < 32 * 32; e += 64) Xs[(e >> 5) * LP + 32 + (e & 31)] = 0.f;
         }
         __syncthreads();
-        // the block below the diagonal: X21 = -X22 (L21 X11); a thread makes eight numbers of a row
-        const int r = tid >> 2, c0 = (tid & 3) * 8;
-        auto block = [&](const float* Arow, const float* Bm, int pitch, float* acc) {
-#pragma unroll
-            for (int j = 0; j < 8; ++j) acc[j] = 0.f;
-#pragma unroll 8
-            for (int m = 0; m < 32; ++m) {
-                const float a = Arow[m];
-                const float4 b0 = *reinterpret_cast<const float4*>(Bm + m * pitch + c0), b1 = *reinterpret_cast<const float4*>(Bm + m * pitch + c0 + 4);
-                acc[0] = fmaf(a, b0.x, acc[0]); acc[1] = fmaf(a, b0.y, acc[1]); acc[2] = fmaf(a, b0.z, acc[2]); acc[3] = fmaf(a, b0.w, acc[3]);
-                acc[4] = fmaf(a, b1.x, acc[4]); acc[5] = fmaf(a, b1.y, acc[5]); acc[6] = fmaf(a, b1.z, acc[6]); acc[7] = fmaf(a, b1.w, acc[7]);
-            }
-        };
-        float acc[8];
-        block(Ls + (32 + r) * LP, Xs, LP, acc);
-#pragma unroll
-        for (int j = 0; j < 8; ++j) M1[r * 36 + c0 + j] = acc[j];
+        {                                              // below the diagonal of each 32 x 32 block: X21 = -X22 (L21 X11), 16 x 16
+            const int off = (tid >> 6) * 2 * TB, r = (tid & 63) >> 2, c0 = (tid & 3) * 4;
+            float acc[4];
+            block_row<16, 1>(Lb + off + (16 + r) * LP, Xb + off + c0, acc);
+            float* m = M1 + (tid >> 6) * 16 * LP;
+            *reinterpret_cast<float4*>(m + r * LP + c0) = make_float4(acc[0], acc[1], acc[2], acc[3]);
+            __syncthreads();
+            block_row<16, 1>(Xb + off + (16 + r) * LP + 16, m + c0, acc);
+            *reinterpret_cast<float4*>(Xb + off + (16 + r) * LP + c0) = make_float4(-acc[0], -acc[1], -acc[2], -acc[3]);
+        }
         __syncthreads();
-        block(Xs + (32 + r) * LP + 32, M1, 36, acc);
-#pragma unroll
-        for (int j = 0; j < 8; ++j) Xs[(32 + r) * LP + c0 + j] = -acc[j];
+        {                                              // and of the whole: 32 x 32, eight numbers of a row per thread
+            const int r = tid >> 2, c0 = (tid & 3) * 8;
+            float acc[8];
+            block_row<32, 2>(Lb + TB + r * LP, Xb + c0, acc);
+            *reinterpret_cast<float4*>(M1 + r * LP + c0) = make_float4(acc[0], acc[1], acc[2], acc[3]);
+            *reinterpret_cast<float4*>(M1 + r * LP + c0 + 4) = make_float4(acc[4], acc[5], acc[6], acc[7]);
+            __syncthreads();
+            block_row<32, 2>(Xb + 2 * TB + r * LP, M1 + c0, acc);
+            *reinterpret_cast<float4*>(Xb + TB + r * LP + c0) = make_float4(-acc[0], -acc[1], -acc[2], -acc[3]);
+            *reinterpret_cast<float4*>(Xb + TB + r * LP + c0 + 4) = make_float4(-acc[4], -acc[5], -acc[6], -acc[7]);
+        }
         __syncthreads();
         uint8_t* tt = p.tt + ((long long)slot * p.H + head) * TT_BYTES;
-        if (tid < CH) {                                // T = X diag(beta)
-            float x[64];
+        {                                              // T = X diag(beta): half a row per thread
+            const int r = tid >> 1, hf = tid & 1;
+            float x[32];
+            const float* src = Xb + (r < 32 ? 0 : (1 + hf) * TB) + (r & 31) * LP;
 #pragma unroll
-            for (int j = 0; j < 64; j += 4) {
-                const float4 t = *reinterpret_cast<const float4*>(Xs + i * LP + j);
-                x[j] = t.x * beta[j];
-                x[j + 1] = t.y * beta[j + 1];
-                x[j + 2] = t.z * beta[j + 2];
-                x[j + 3] = t.w * beta[j + 3];
+            for (int j = 0; j < 32; j += 4) {
+                float4 t = *reinterpret_cast<const float4*>(src + j);
+                const float4 be = *reinterpret_cast<const float4*>(beta + hf * 32 + j);
+                if (r < 32 && hf) t = make_float4(0.f, 0.f, 0.f, 0.f);
+                x[j] = t.x * be.x;
+                x[j + 1] = t.y * be.y;
+                x[j + 2] = t.z * be.z;
+                x[j + 3] = t.w * be.w;
             }
-            store_row_split(sT, sT + BLK, i, x);
+            store_row_split<4>(sT, sT + BLK, r, hf * 4, x);
         }
         tc::fence_proxy_async();
         tc::tc_fence_before();
         __syncthreads();
-        if (tid == 0) {
+        if (warp == 0) {
             tc::tc_fence_after();
             const uint32_t a = smem_u32(sA), t = smem_u32(sT), id = tc::instr_desc_f16(128, CH, 1, 1, 0, 1);
-            mma_steps<4, 32, 2048>(tmem + 64, a, 16, t, id, false);            // rows 64 .. 127 of the operand are not looked at
-            mma_steps<4, 32, 2048>(tmem + 64, a, 16, t + BLK, id, true);
-            mma_steps<4, 32, 2048>(tmem + 64, a + BLK, 16, t, id, true);
-            tc::tc_commit(&bars[1]);
+            // the operand's rows 64 .. 127 (what follows in shared memory) give rows that are not looked at
+            if (tc::elect_one()) {
+                mma_steps<4, 32, 2048>(tmem + 64, a, 16, t, id, false);
+                mma_steps<4, 32, 2048>(tmem + 64, a, 16, t + BLK, id, true);
+                mma_steps<4, 32, 2048>(tmem + 64, a + BLK, 16, t, id, true);
+                tc::tc_commit(&bars[1]);
+            }
+            __syncwarp();
         }
-        __syncwarp();
         for (int e = tid; e < BLK / 16; e += 128) {
             reinterpret_cast<uint4*>(tt)[e] = reinterpret_cast<const uint4*>(sT)[e];
             reinterpret_cast<uint4*>(tt + 2 * BLK)[e] = reinterpret_cast<const uint4*>(sT + BLK)[e];
@@ -285,17 +340,20 @@ delta_prepare_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_const
         float* sc = p.scal + ((long long)slot * p.H + head) * SCALARS;
         if (tid < CH) {
             const float gi = gsum[tid], gl = gsum[CH - 1];
-            sc[tid] = expf(gi) * unit[tid];
-            sc[CH + tid] = expf(gi) * unit[CH + tid];
-            sc[2 * CH + tid] = expf(gl - gi) * unit[tid];
-            if (tid == 0) sc[3 * CH] = gl > -0.5f ? 1.0f + expm1f(gl) : expf(gl);   // as the decays in csrc/delta.cu
+            sc[tid] = ex2(gi) * unit[tid];
+            sc[CH + tid] = ex2(gi) * unit[CH + tid];
+            sc[2 * CH + tid] = ex2(gl - gi) * unit[tid];
+            if (tid == 0) {                            // the state's own factor: to nearest, as the decays in csrc/delta.cu
+                const float x = gl * attn::LN2;
+                sc[3 * CH] = x > -0.5f ? 1.0f + expm1f(x) : expf(x);
+            }
         }
         if (tc::mbar_wait(&bars[1], 1, &abort_flag)) {
             tc::tc_fence_after();
             if (warp < 2) {
                 float x[64];
                 tmem_row64(tmem + 64 + lane_base, x);
-                store_row_split(tt + BLK, tt + 3 * BLK, i, x);
+                store_row_split<8>(tt + BLK, tt + 3 * BLK, i, 0, x);
             }
         } else if (lane == 0) {
             atomicMax(p.status, (int)KB_TIMEOUT_MMA);
@@ -318,7 +376,7 @@ struct Scan {
 };
 
 template <int D>
-__global__ void __launch_bounds__(128, 2)
+__global__ void __launch_bounds__(256, 2)
 delta_scan_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constant__ CUtensorMap tmQ, const ChunkParams p) {
     extern __shared__ __align__(1024) uint8_t smem[];
     using L = Scan<D>;
@@ -326,7 +384,10 @@ delta_scan_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constant
     uint64_t* bars = reinterpret_cast<uint64_t*>(smem + L::OFF_BAR);      // [K; Q] loaded, [T; A T] loaded, product done
     uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bars + 3);
     volatile int* abort_flag = reinterpret_cast<volatile int*>(tmem_slot + 1);
-    const int tid = threadIdx.x, warp = tid >> 5;
+    const int tid = threadIdx.x, warp = __shfl_sync(0xffffffffu, tid >> 5, 0);
+    // two threads per tile row, 32 columns each
+    const int row = (warp & 3) * 32 + (tid & 31), hf = warp >> 2;
+    const bool is_k = row < CH;                        // the rows of K (then R, U); the others are those of Q (then O)
     const int tile = blockIdx.x, head = blockIdx.y, b = blockIdx.z, kvh = head / (p.H / p.G);
     const int row0 = p.cu[b], n = p.cu[b + 1] - row0, chunks = (n + CH - 1) / CH;
     if (n <= 0) return;
@@ -334,17 +395,24 @@ delta_scan_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constant
         if (tid == 0) atomicMax(p.status, (int)KB_BAD_ARG);
         return;
     }
+    const int base = slot_base(p.cu, b);
+    const uint8_t* tt = p.tt + ((long long)base * p.H + head) * TT_BYTES;
+    const float* sc = p.scal + ((long long)base * p.H + head) * SCALARS;
+    if (tid == 0) {
+        for (int i = 0; i < 3; ++i) tc::mbar_init(bars + i, 1);
+        *abort_flag = 0;
+        tc::fence_barrier_init();
+        load_kq<D>(sKQ, &tmK, &tmQ, bars, kvh, row0);
+        tc::mbar_expect_tx(bars + 1, TT_BYTES);
+        bulk_load(sTT, tt, TT_BYTES, bars + 1);
+    }
+    __syncwarp();
     int slot = p.slots[b];
     if (slot >= p.num_states) {
         if (tid == 0) atomicMax(p.status, (int)KB_BAD_INDEX);
         slot = -1;
     }
     const bool fresh = slot < 0 || p.ctx[b] <= n;
-    if (tid == 0) {
-        for (int i = 0; i < 3; ++i) tc::mbar_init(bars + i, 1);
-        *abort_flag = 0;
-        tc::fence_barrier_init();
-    }
     if (warp == 0) {
         tc::tmem_alloc(tmem_slot, 256);
         tc::tmem_relinquish();
@@ -352,89 +420,91 @@ delta_scan_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constant
     tc::tc_fence_before();
     __syncthreads();
     tc::tc_fence_after();
-    const uint32_t tmem = *tmem_slot, lane_base = (uint32_t)(warp * 32) << 16;
-    const int base = slot_base(p.cu, b);
-    const uint8_t* tt = p.tt + ((long long)base * p.H + head) * TT_BYTES;
-    const float* sc = p.scal + ((long long)base * p.H + head) * SCALARS;
-    if (tid == 0) {
-        load_kq<D>(sKQ, &tmK, &tmQ, bars, kvh, row0);
-        tc::mbar_expect_tx(bars + 1, TT_BYTES);
-        bulk_load(sTT, tt, TT_BYTES, bars + 1);
-    }
-    __syncwarp();
-    // row tid of the state: 64 columns
-    float S[64];
-    float* st = p.state + (((long long)(slot < 0 ? 0 : slot) * p.H + head) * p.d + tid) * p.dvp + tile * 64;
-    const bool own = tid < p.d;
+    const uint32_t tmem0 = __shfl_sync(0xffffffffu, *tmem_slot, 0), tmem = tmem0 + ((uint32_t)((warp & 3) * 32) << 16) + hf * 32;
+    // this thread's half of row `row` of the state
+    const int col0 = tile * 64 + hf * 32;
+    float S[32];
+    float* st = p.state + (((long long)(slot < 0 ? 0 : slot) * p.H + head) * p.d + row) * p.dvp + col0;
+    const bool own = row < p.d;
 #pragma unroll
-    for (int c = 0; c < 64; c += 4) {
+    for (int c = 0; c < 32; c += 4) {
         float4 f = make_float4(0.f, 0.f, 0.f, 0.f);
-        if (own && !fresh && tile * 64 + c < p.dvp) f = *reinterpret_cast<const float4*>(st + c);
+        if (own && !fresh && col0 + c < p.dvp) f = *reinterpret_cast<const float4*>(st + c);
         S[c] = f.x; S[c + 1] = f.y; S[c + 2] = f.z; S[c + 3] = f.w;
     }
-    if (tid < D) store_row_split(sS, sS + L::S_HALF, tid, S);
-    const int i = tid & 63;
+    if (row < D) store_row_split<4>(sS, sS + L::S_HALF, row, hf * 4, S);
+    const int i = row & 63;
+    const long long vstride = (long long)p.H * p.dvt;
+    const bf16* vsrc = p.v + (long long)(row0 + i) * vstride + head * p.dvt + col0;
+    bf16* odst = p.o + (long long)(row0 + i) * vstride + head * p.dvt + col0;
     const uint32_t aKQ = smem_u32(sKQ), aTT = smem_u32(sTT), aS = smem_u32(sS), aRU = smem_u32(sRU);
     const uint32_t id_kb = tc::instr_desc_f16(128, 64, 1, 1, 0, 1), id_mb = tc::instr_desc_f16(128, 64, 1, 1, 1, 1);
+    // values and scalars of a chunk, fetched while the chunk in front of it is worked on
+    uint4 v[4];
+    float e, eu, decay;
+    auto fetch = [&](int c) {
+        const float* s = sc + (long long)c * p.H * SCALARS;
+        e = s[row];
+        eu = s[2 * CH + i];
+        decay = s[3 * CH];
+        if (is_k) {
+            const uint4* src = reinterpret_cast<const uint4*>(vsrc + (long long)c * CH * vstride);
+#pragma unroll
+            for (int j = 0; j < 4; ++j) v[j] = c * CH + i < n ? src[j] : make_uint4(0u, 0u, 0u, 0u);
+        }
+    };
+    fetch(0);
     uint32_t done = 0;                                 // parity of the product barrier
     bool failed = false;
     for (int c = 0; c < chunks; ++c) {
-        const int at = row0 + c * CH, valid = min(CH, n - c * CH);
         tc::fence_proxy_async();
         tc::tc_fence_before();
         if (__syncthreads_or(failed)) { failed = true; break; }
-        if (tid == 0) {                                // X = [K; Q] S
-            if (tc::mbar_wait(bars, c & 1, abort_flag)) {
-                tc::tc_fence_after();
-                mma_steps<D / 16, 32, 2048, true>(tmem, aKQ, 16, aS, id_kb, false);
-                mma_steps<D / 16, 32, 2048, true>(tmem, aKQ, 16, aS + L::S_HALF, id_kb, true);
+        // products are issued by one elected lane of a whole warp: their operands then stay in uniform registers
+        if (warp == 0) {                               // X = [K; Q] S
+            failed |= !tc::mbar_wait(bars, c & 1, abort_flag);
+            tc::tc_fence_after();
+            if (!__any_sync(0xffffffffu, failed) && tc::elect_one()) {
+                mma_steps<D / 16, 32, 2048, true>(tmem0, aKQ, 16, aS, id_kb, false);
+                mma_steps<D / 16, 32, 2048, true>(tmem0, aKQ, 16, aS + L::S_HALF, id_kb, true);
                 tc::tc_commit(bars + 2);
-            } else {
-                failed = true;
             }
-        }
-        __syncwarp();
-        const float* s = sc + (long long)c * p.H * SCALARS;
-        const float e = s[tid], eu = s[2 * CH + i], decay = s[3 * CH];
-        uint4 v[8];
-        if (tid < CH) {
-            const uint4* src = reinterpret_cast<const uint4*>(p.v + (long long)(at + i) * p.H * p.dvt + head * p.dvt + tile * 64);
-#pragma unroll
-            for (int j = 0; j < 8; ++j) v[j] = i < valid ? src[j] : make_uint4(0u, 0u, 0u, 0u);
+            __syncwarp();
         }
         failed |= !tc::mbar_wait(bars + 2, done, abort_flag);
         done ^= 1;
         tc::tc_fence_after();
-        float x[64];
-        tmem_row64(tmem + lane_base, x);
-        if (tid < CH) {                                // R = V - e^G r_k X
+        float x[32];
+        tmem_row32(tmem, x);
+        if (is_k) {                                    // R = V - e^G r_k X
 #pragma unroll
-            for (int j = 0; j < 8; ++j) {
+            for (int j = 0; j < 4; ++j) {
                 float f[8];
                 unpack8(*reinterpret_cast<const bf16x8*>(&v[j]), f);
 #pragma unroll
                 for (int q = 0; q < 8; ++q) x[j * 8 + q] = fmaf(-e, x[j * 8 + q], f[q]);
             }
-            store_row_split(sRU, sRU + BLK, i, x);
+            store_row_split<4>(sRU, sRU + BLK, i, hf * 4, x);
         } else {
 #pragma unroll
-            for (int j = 0; j < 64; ++j) x[j] *= e;
+            for (int j = 0; j < 32; ++j) x[j] *= e;
         }
         tc::fence_proxy_async();
         tc::tc_fence_before();
         if (__syncthreads_or(failed)) { failed = true; break; }
-        if (tid == 0) {                                // [U; A U] = [T; A T] R
-            if (tc::mbar_wait(bars + 1, c & 1, abort_flag)) {
-                tc::tc_fence_after();
-                mma_steps<4, 32, 2048>(tmem + 64, aTT, 16, aRU, id_kb, false);
-                mma_steps<4, 32, 2048>(tmem + 64, aTT, 16, aRU + BLK, id_kb, true);
-                mma_steps<4, 32, 2048>(tmem + 64, aTT + 2 * BLK, 16, aRU, id_kb, true);
+        if (warp == 0) {                               // [U; A U] = [T; A T] R
+            failed |= !tc::mbar_wait(bars + 1, c & 1, abort_flag);
+            tc::tc_fence_after();
+            if (!__any_sync(0xffffffffu, failed) && tc::elect_one()) {
+                mma_steps<4, 32, 2048>(tmem0 + 64, aTT, 16, aRU, id_kb, false);
+                mma_steps<4, 32, 2048>(tmem0 + 64, aTT, 16, aRU + BLK, id_kb, true);
+                mma_steps<4, 32, 2048>(tmem0 + 64, aTT + 2 * BLK, 16, aRU, id_kb, true);
                 tc::tc_commit(bars + 2);
-            } else {
-                failed = true;
             }
+            __syncwarp();
         }
-        __syncwarp();
+        const float scale_u = eu, scale_s = decay;
+        if (c + 1 < chunks) fetch(c + 1);
         failed |= !tc::mbar_wait(bars + 2, done, abort_flag);
         done ^= 1;
         tc::tc_fence_after();
@@ -443,43 +513,45 @@ delta_scan_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constant
             bulk_load(sTT, tt + (long long)(c + 1) * p.H * TT_BYTES, TT_BYTES, bars + 1);
         }
         __syncwarp();
-        {
-            float y[64];
-            tmem_row64(tmem + 64 + lane_base, y);
-            if (tid < CH) {                            // e^(G_64 - G) r_k U
+        float y[32];
+        tmem_row32(tmem + 64, y);
+        if (is_k) {                                    // e^(G_64 - G) r_k U
 #pragma unroll
-                for (int j = 0; j < 64; ++j) y[j] *= eu;
-                store_row_split(sRU, sRU + BLK, i, y);
-            } else if (i < valid) {
-                bf16* dst = p.o + (long long)(at + i) * p.H * p.dvt + head * p.dvt + tile * 64;
-#pragma unroll
-                for (int j = 0; j < 64; j += 8) {
-#pragma unroll
-                    for (int q = 0; q < 8; ++q) x[j + q] += y[j + q];
-                    store8(dst + j, x + j);
-                }
-            }
+            for (int j = 0; j < 32; ++j) y[j] *= scale_u;
+            store_row_split<4>(sRU, sRU + BLK, i, hf * 4, y);
         }
         tc::fence_proxy_async();
         tc::tc_fence_before();
         if (__syncthreads_or(failed)) { failed = true; break; }
-        if (tid == 0) {                                // K^T U
+        if (warp == 0) {                               // K^T U
             tc::tc_fence_after();
-            mma_steps<4, 2048, 2048>(tmem + 128, aKQ, 2 * BLK, aRU, id_mb, false);
-            mma_steps<4, 2048, 2048>(tmem + 128, aKQ, 2 * BLK, aRU + BLK, id_mb, true);
-            tc::tc_commit(bars + 2);
+            if (tc::elect_one()) {
+                mma_steps<4, 2048, 2048>(tmem0 + 128, aKQ, 2 * BLK, aRU, id_mb, false);
+                mma_steps<4, 2048, 2048>(tmem0 + 128, aKQ, 2 * BLK, aRU + BLK, id_mb, true);
+                tc::tc_commit(bars + 2);
+            }
+            __syncwarp();
+        }
+        if (!is_k && c * CH + i < n) {                 // O, while the product runs
+            bf16* dst = odst + (long long)c * CH * vstride;
+#pragma unroll
+            for (int j = 0; j < 32; j += 8) {
+#pragma unroll
+                for (int q = 0; q < 8; ++q) x[j + q] += y[j + q];
+                store8(dst + j, x + j);
+            }
         }
         __syncwarp();
         failed |= !tc::mbar_wait(bars + 2, done, abort_flag);
         done ^= 1;
         tc::tc_fence_after();
-        if (tid == 0 && c + 1 < chunks && !failed) load_kq<D>(sKQ, &tmK, &tmQ, bars, kvh, at + CH);
+        if (tid == 0 && c + 1 < chunks && !failed) load_kq<D>(sKQ, &tmK, &tmQ, bars, kvh, row0 + (c + 1) * CH);
         __syncwarp();
-        tmem_row64(tmem + 128 + lane_base, x);
-        if (tid < D) {
+        tmem_row32(tmem + 128, x);
+        if (row < D) {
 #pragma unroll
-            for (int j = 0; j < 64; ++j) S[j] = fmaf(decay, S[j], x[j]);
-            store_row_split(sS, sS + L::S_HALF, tid, S);
+            for (int j = 0; j < 32; ++j) S[j] = fmaf(scale_s, S[j], x[j]);
+            store_row_split<4>(sS, sS + L::S_HALF, row, hf * 4, S);
         }
     }
     if (failed) {
@@ -488,14 +560,14 @@ delta_scan_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constant
         while (global_timer_ns() - t0 < 2000000ull) {}
     } else if (own && slot >= 0) {
 #pragma unroll
-        for (int c = 0; c < 64; c += 4)
-            if (tile * 64 + c < p.dvp) *reinterpret_cast<float4*>(st + c) = make_float4(S[c], S[c + 1], S[c + 2], S[c + 3]);
+        for (int c = 0; c < 32; c += 4)
+            if (col0 + c < p.dvp) *reinterpret_cast<float4*>(st + c) = make_float4(S[c], S[c + 1], S[c + 2], S[c + 3]);
     }
     tc::tc_fence_before();
     __syncthreads();
     if (warp == 0) {
         tc::tc_fence_after();
-        tc::tmem_dealloc(tmem, 256);
+        tc::tmem_dealloc(tmem0, 256);
     }
 }
 
@@ -511,9 +583,9 @@ struct ConvParams {
     const int *cu, *ctx, *slots;
     bf16 *q, *k, *v;                                   // [N, G * D], [N, G * D], [N, H * dvt]
 };
-constexpr int CONV_TOKENS = 32;
+constexpr int CONV_TOKENS = 32, CONV_GROUP = 8;
 
-// A thread makes eight neighbouring channels of up to CONV_TOKENS neighbouring tokens.
+// A thread makes eight neighbouring channels of up to CONV_TOKENS neighbouring tokens; the inputs of CONV_GROUP tokens are fetched together.
 template <int TAPS>
 __global__ void __launch_bounds__(128) delta_conv_kernel(const ConvParams p) {
     const int vecs = (2 * p.G * p.d + p.H * p.dv) / 8, vec = blockIdx.y * 128 + threadIdx.x;
@@ -548,45 +620,56 @@ __global__ void __launch_bounds__(128) delta_conv_kernel(const ConvParams p) {
         const int m = (b + hi) >> 1;
         if (p.cu[m] <= t0) b = m; else hi = m;
     }
+    int next = b + 1 < p.B ? p.cu[b + 1] : p.N;
     bool enter = true;
-    for (int t = t0; t < t1; ++t) {
-        while (b + 1 < p.B && t >= p.cu[b + 1]) {
-            ++b;
-            enter = true;
-        }
-        if (enter) {
-            enter = false;
-            const int lo = p.cu[b], n = p.cu[b + 1] - lo, slot = p.slots[b];
-            const bool fresh = slot < 0 || slot >= p.num_states || p.ctx[b] <= n;
+    for (int tg = t0; tg < t1; tg += CONV_GROUP) {
+        uint4 in8[CONV_GROUP];
 #pragma unroll
-            for (int j = 1; j < TAPS; ++j) {
-                if (t - j >= lo) load8(p.rows + (long long)(t - j) * p.stride + col, past[j]);
-                else if (!fresh) {
-                    // row r of the ring is the input TAPS - 1 - r tokens in front of the pass
-                    const bf16* r = p.ring + (((long long)slot * p.H + ring_head) * p.ring_rows + (TAPS - 1 - (j - (t - lo)))) * (2 * p.d + p.dv) + ring_col;
+        for (int u = 0; u < CONV_GROUP; ++u)
+            if (tg + u < t1) in8[u] = *reinterpret_cast<const uint4*>(p.rows + (long long)(tg + u) * p.stride + col);
 #pragma unroll
-                    for (int e = 0; e < 8; ++e) past[j][e] = to_float(r[e]);
-                } else {
+        for (int u = 0; u < CONV_GROUP; ++u) {
+            const int t = tg + u;
+            if (t >= t1) break;
+            while (b + 1 < p.B && t >= next) {
+                ++b;
+                next = b + 1 < p.B ? p.cu[b + 1] : p.N;
+                enter = true;
+            }
+            if (enter) {
+                enter = false;
+                const int lo = p.cu[b], n = p.cu[b + 1] - lo, slot = p.slots[b];
+                const bool fresh = slot < 0 || slot >= p.num_states || p.ctx[b] <= n;
 #pragma unroll
-                    for (int e = 0; e < 8; ++e) past[j][e] = 0.f;
+                for (int j = 1; j < TAPS; ++j) {
+                    if (t - j >= lo) load8(p.rows + (long long)(t - j) * p.stride + col, past[j]);
+                    else if (!fresh) {
+                        // row r of the ring is the input TAPS - 1 - r tokens in front of the pass
+                        const bf16* r = p.ring + (((long long)slot * p.H + ring_head) * p.ring_rows + (TAPS - 1 - (j - (t - lo)))) * (2 * p.d + p.dv) + ring_col;
+#pragma unroll
+                        for (int e = 0; e < 8; ++e) past[j][e] = to_float(r[e]);
+                    } else {
+#pragma unroll
+                        for (int e = 0; e < 8; ++e) past[j][e] = 0.f;
+                    }
                 }
             }
+            unpack8(*reinterpret_cast<const bf16x8*>(&in8[u]), past[0]);
+            float z[8];
+#pragma unroll
+            for (int e = 0; e < 8; ++e) z[e] = past[TAPS - 1][e] * w[TAPS - 1][e];
+#pragma unroll
+            for (int j = TAPS - 2; j >= 0; --j)
+#pragma unroll
+                for (int e = 0; e < 8; ++e) z[e] = fmaf(past[j][e], w[j][e], z[e]);
+#pragma unroll
+            for (int e = 0; e < 8; ++e) z[e] = silu(z[e]);
+            store8(dst + (long long)t * dst_stride, z);
+#pragma unroll
+            for (int j = TAPS - 1; j > 0; --j)
+#pragma unroll
+                for (int e = 0; e < 8; ++e) past[j][e] = past[j - 1][e];
         }
-        load8(p.rows + (long long)t * p.stride + col, past[0]);
-        float z[8];
-#pragma unroll
-        for (int e = 0; e < 8; ++e) z[e] = past[TAPS - 1][e] * w[TAPS - 1][e];
-#pragma unroll
-        for (int j = TAPS - 2; j >= 0; --j)
-#pragma unroll
-            for (int e = 0; e < 8; ++e) z[e] = fmaf(past[j][e], w[j][e], z[e]);
-#pragma unroll
-        for (int e = 0; e < 8; ++e) z[e] = silu(z[e]);
-        store8(dst + (long long)t * dst_stride, z);
-#pragma unroll
-        for (int j = TAPS - 1; j > 0; --j)
-#pragma unroll
-            for (int e = 0; e < 8; ++e) past[j][e] = past[j - 1][e];
     }
 }
 
@@ -617,23 +700,38 @@ delta_finish_kernel(const bf16* __restrict__ o, int dvt, const bf16* __restrict_
     const long long tok = live ? item / H : 0;
     const int head = live ? (int)(item % H) : 0;
     const bf16* src = o + (tok * H + head) * dvt;
-    float x[8], ss = 0.f;
-    for (int c = sub * 8; live && c < dv; c += LPH * 8) {
-        load8(src + c, x);
+    const bf16* gsrc = gate + tok * gate_stride + head * dv;
+    bf16* dst = out + tok * out_stride + head * dv;
+    const int c0 = sub * 8;
+    const bool in = live && c0 < dv;
+    float x[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f}, g[8], w[8], ss = 0.f;
+    if (in) {
+        load8(src + c0, x);
+        load8(gsrc + c0, g);
+        load8(norm + c0, w);
+    }
 #pragma unroll
-        for (int j = 0; j < 8; ++j) ss += x[j] * x[j];
+    for (int j = 0; j < 8; ++j) ss += x[j] * x[j];
+    for (int c = c0 + LPH * 8; live && c < dv; c += LPH * 8) {
+        float y[8];
+        load8(src + c, y);
+#pragma unroll
+        for (int j = 0; j < 8; ++j) ss += y[j] * y[j];
     }
 #pragma unroll
     for (int k = LPH / 2; k > 0; k >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, k);
     const float r = 1.0f / sqrtf(ss / (float)dv + eps);
-    for (int c = sub * 8; live && c < dv; c += LPH * 8) {
-        float g[8], w[8];
+    if (!in) return;
+#pragma unroll
+    for (int j = 0; j < 8; ++j) x[j] = x[j] * r * w[j] * silu(g[j]);
+    store8(dst + c0, x);
+    for (int c = c0 + LPH * 8; c < dv; c += LPH * 8) {
         load8(src + c, x);
-        load8(gate + tok * gate_stride + head * dv + c, g);
+        load8(gsrc + c, g);
         load8(norm + c, w);
 #pragma unroll
         for (int j = 0; j < 8; ++j) x[j] = x[j] * r * w[j] * silu(g[j]);
-        store8(out + tok * out_stride + head * dv + c, x);
+        store8(dst + c, x);
     }
 }
 
@@ -668,7 +766,7 @@ int launch_chunks(const ChunkParams& p, const bf16* q, const bf16* k, cudaStream
     if (!r) r = rows_tmap(&tmQ, q, p.N, (long long)p.G * D);
     if (r) return r;
     delta_prepare_kernel<D><<<dim3(p.N / CH + p.B, p.H), 128, PREP_SMEM, st>>>(tmK, tmQ, p);
-    delta_scan_kernel<D><<<dim3(p.dvt / 64, p.H, p.B), 128, Scan<D>::SMEM, st>>>(tmK, tmQ, p);
+    delta_scan_kernel<D><<<dim3(p.dvt / 64, p.H, p.B), 256, Scan<D>::SMEM, st>>>(tmK, tmQ, p);
     return kb_launch_status();
 }
 
