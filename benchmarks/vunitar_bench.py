@@ -14,18 +14,17 @@ from __future__ import annotations
 import argparse
 import json
 import os
-import statistics
 import sys
-import time
 
 import torch
 
 ROOT = os.path.dirname(os.path.dirname(os.path.abspath(__file__)))
 sys.path.insert(0, ROOT)
+sys.path.insert(0, os.path.join(ROOT, "benchmarks"))
+from compare_common import engine_arm, peaks, timed  # noqa: E402
 from kotodama_b200.config import ModelConfig  # noqa: E402
 from kotodama_b200.models.llama import KotodamaModel  # noqa: E402
 from kotodama_b200.models.vunitar import VunitarConfig, VunitarModel  # noqa: E402
-from kotodama_b200.serve.engine import SamplingParams, ServingEngine  # noqa: E402
 
 VOCAB = 49152
 # name -> width, heads, kv_rank, layers, experts, top, expert ff, shared ff, dense ff (layer 0; all layers when experts = 0), KV heads of the Llama arm
@@ -34,15 +33,6 @@ SIZES = {
     "3072-moe": dict(width=3072, heads=24, rank=512, layers=6, experts=64, top=8, ff=1024, shared=2048, dense=10240, kv=8),
     "4096-dense": dict(width=4096, heads=32, rank=512, layers=6, experts=0, top=0, ff=0, shared=0, dense=16384, kv=8),
 }
-
-
-def peaks() -> dict:
-    try:
-        with open(os.path.join(ROOT, "MEASURED_PEAKS.json")) as fh:
-            d = json.load(fh)
-        return {"gbs": d["hbm_gbs"], "tflops": d["bf16_tflops"], "of": "measured"}
-    except OSError:
-        return {"gbs": 6650.0, "tflops": 1590.0, "of": "fallback"}
 
 
 def vunitar_config(z: dict) -> VunitarConfig:
@@ -61,29 +51,6 @@ def llama_config(z: dict) -> ModelConfig:
     inter = (active * 2 // 3 + 127) // 128 * 128
     return ModelConfig(hidden_size=z["width"], num_layers=z["layers"], num_attention_heads=z["heads"], num_kv_heads=z["kv"],
                        head_dim=128, intermediate_size=inter, vocab_size=VOCAB, max_position_embeddings=8192, tie_word_embeddings=True)
-
-
-def timed(calls: list, reps: int = 5) -> float:
-    """Mean device time of one call in ms: the calls (over different buffers) captured in one graph, replayed.  The
-    decode kernels of both models are launched as in serving, as programmatic dependents of one another."""
-    for c in calls[:2]:
-        c()
-    torch.cuda.synchronize()
-    g = torch.cuda.CUDAGraph()
-    from kotodama_b200.ops import get_ops
-    with torch.cuda.graph(g), get_ops("cuda").dependent_launch(True):
-        keep = [c() for c in calls]
-    for _ in range(2):
-        g.replay()
-    e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
-    torch.cuda.synchronize()
-    e0.record()
-    for _ in range(reps):
-        g.replay()
-    e1.record()
-    torch.cuda.synchronize()
-    del keep
-    return e0.elapsed_time(e1) / (reps * len(calls))
 
 
 def kernels(name: str, z: dict, batch: int = 64, ctx: int = 1280, tokens: int = 8192) -> list[dict]:
@@ -230,50 +197,15 @@ def kernels(name: str, z: dict, batch: int = 64, ctx: int = 1280, tokens: int = 
     return out
 
 
-def engine_arm(model, z: dict, requests: int, prompt: int, new: int) -> dict:
-    """Prefill of `requests` prompts of `prompt` tokens each, then `new` greedy tokens for all of them."""
-    cfg = model.config
-    eng = ServingEngine(model, device="cuda", dtype=torch.bfloat16, max_batch=requests, max_ctx=prompt + new + 16)
-    if isinstance(model, KotodamaModel):
-        eng.arena.init_weights(cfg.num_layers, 0)
-    gen = torch.Generator().manual_seed(0)
-    prompts = [torch.randint(0, cfg.vocab_size, (prompt,), generator=gen).tolist() for _ in range(requests)]
-    res = {}
-    for _ in range(2):                                  # the second pass is reported
-        before = eng.stats["prefill_s"]
-        for p in prompts:
-            eng.add_request(p, SamplingParams(max_new_tokens=new, temperature=0.0))
-        torch.cuda.synchronize()
-        eng.step()
-        torch.cuda.synchronize()
-        prefill_s = eng.stats["prefill_s"] - before
-        eng.graph_ms = []
-        steps = []
-        while eng.has_work():
-            torch.cuda.synchronize()
-            t = time.perf_counter()
-            eng.step()
-            torch.cuda.synchronize()
-            steps.append(time.perf_counter() - t)
-        res = dict(prefill_tok_s=round(requests * prompt / prefill_s), decode_tok_s=round(requests / statistics.median(steps)),
-                   decode_step_ms=round(1e3 * statistics.median(steps), 3), decode_graph_ms=round(statistics.median(eng.graph_ms), 3))
-        eng.graph_ms = None
-    eng.ops.check_status()
-    res["launches"] = eng.ops.launches
-    del eng
-    torch.cuda.empty_cache()
-    return res
-
-
 def engines(name: str, z: dict, requests: int = 64, prompt: int = 1024, new: int = 48) -> dict:
     vc, lc = vunitar_config(z), llama_config(z)
     out = dict(size=name, requests=requests, prompt_tokens=prompt, new_tokens=new, vunitar_params=vc.param_count(),
                llama_params=lc.param_count())
-    out["vunitar"] = engine_arm(VunitarModel.random_init(vc, 0, device="cuda"), z, requests, prompt, new)
+    out["vunitar"] = engine_arm(VunitarModel.random_init(vc, 0, device="cuda"), requests, prompt, new)
     torch.cuda.empty_cache()
     with torch.device("meta"):
         m = KotodamaModel(lc)
-    out["llama"] = engine_arm(m, z, requests, prompt, new)
+    out["llama"] = engine_arm(m, requests, prompt, new)
     return out
 
 

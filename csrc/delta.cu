@@ -17,7 +17,7 @@ struct DeltaParams {
     const void* rows;              // projections of the packed tokens
     long long stride;
     int col_q, col_k, col_v, col_g, col_b, col_a;
-    const float* conv;             // [2 G d + H dv, taps]
+    const float* conv;             // [taps, 2 G d + H dv]
     const float *a_log, *dt_bias, *norm;
     int taps, H, G, d, dv, dvp;
     float eps;
@@ -86,12 +86,12 @@ delta_step_kernel(const DeltaParams p) {
         const float g = decay(neg_a * softplus(to_float(row[p.col_a + head]) + bias));
         for (int c = tid; c < C; c += THREADS) {
             const int col = column(c);
-            const float* w = p.conv + (long long)(c < p.d ? kvh * p.d + c : c < 2 * p.d ? (p.G + kvh) * p.d + c - p.d
-                                                                                      : 2 * p.G * p.d + head * p.dv + c - 2 * p.d) * p.taps;
+            const int channels = 2 * p.G * p.d + p.H * p.dv;
+            const float* w = p.conv + (c < p.d ? kvh * p.d + c : c < 2 * p.d ? (p.G + kvh) * p.d + c - p.d : 2 * p.G * p.d + head * p.dv + c - 2 * p.d);
             float z = 0.f;
             for (int j = 0; j < p.taps; ++j) {
                 const int i = t - past + j;            // the tap's token
-                z = fmaf(w[j], i >= lo ? to_float(rows[(long long)i * p.stride + col]) : hist[(past + i - lo) * C + c], z);
+                z = fmaf(w[(long long)j * channels], i >= lo ? to_float(rows[(long long)i * p.stride + col]) : hist[(past + i - lo) * C + c], z);
             }
             cur[c] = silu(z);
         }

@@ -51,9 +51,6 @@ struct ChunkParams {
 // Chunk c of sequence b has slot cu[b] / 64 + b + c: slots of different sequences never meet, and N / 64 + B of them suffice.
 __device__ __forceinline__ int slot_base(const int* cu, int b) { return cu[b] / CH + b; }
 
-// results are rounded to bf16 where this is used
-__device__ __forceinline__ float silu(float z) { return __fdividef(z, 1.0f + __expf(-z)); }
-
 // 8 * CHUNKS numbers of a row as two bf16 numbers each, from 16-byte chunk `c0` on, to row `row` of two 128-byte-swizzled tiles
 template <int CHUNKS>
 __device__ __forceinline__ void store_row_split(uint8_t* hi, uint8_t* lo, int row, int c0, const float* x) {
@@ -62,31 +59,42 @@ __device__ __forceinline__ void store_row_split(uint8_t* hi, uint8_t* lo, int ro
         uint32_t h[4], l[4];
 #pragma unroll
         for (int j = 0; j < 4; ++j) {
-            const float a = x[c * 8 + 2 * j], b = x[c * 8 + 2 * j + 1];
-            const __nv_bfloat162 u = __floats2bfloat162_rn(a, b);
-            const float2 f = __bfloat1622float2(u);
-            h[j] = *reinterpret_cast<const uint32_t*>(&u);
-            l[j] = attn::pack_bf16(a - f.x, b - f.y);
+            // the upper half is cut off, the rest (exact) is rounded: integer instructions, where the conversions share the
+            // special-function unit
+            const uint32_t a = __float_as_uint(x[c * 8 + 2 * j]), b = __float_as_uint(x[c * 8 + 2 * j + 1]);
+            h[j] = __byte_perm(a, b, 0x7632);
+            const float ra = __uint_as_float(a) - __uint_as_float(a & 0xffff0000u), rb = __uint_as_float(b) - __uint_as_float(b & 0xffff0000u);
+            l[j] = __byte_perm(__float_as_uint(ra) + 0x8000u, __float_as_uint(rb) + 0x8000u, 0x7632);
         }
         const int at = row * 128 + (((c0 + c) ^ (row & 7)) << 4);
         *reinterpret_cast<uint4*>(hi + at) = make_uint4(h[0], h[1], h[2], h[3]);
         *reinterpret_cast<uint4*>(lo + at) = make_uint4(l[0], l[1], l[2], l[3]);
     }
 }
-__device__ __forceinline__ void tmem_row64(uint32_t taddr, float* x) {
-    tc::tmem_ld32(taddr, reinterpret_cast<uint32_t*>(x));
-    tc::tmem_ld32(taddr + 32, reinterpret_cast<uint32_t*>(x + 32));
-    tc::tmem_ld_wait();
-}
 __device__ __forceinline__ void tmem_row32(uint32_t taddr, float* x) {
     tc::tmem_ld32(taddr, reinterpret_cast<uint32_t*>(x));
     tc::tmem_ld_wait();
+}
+// 32 columns of the sum of two results 64 columns apart
+__device__ __forceinline__ void tmem_sum32(uint32_t taddr, float* x) {
+    float y[32];
+    tc::tmem_ld32(taddr, reinterpret_cast<uint32_t*>(x));
+    tc::tmem_ld32(taddr + 64, reinterpret_cast<uint32_t*>(y));
+    tc::tmem_ld_wait();
+#pragma unroll
+    for (int j = 0; j < 32; ++j) x[j] += y[j];
 }
 // 2^x by the special-function unit (relative error 2^-22)
 __device__ __forceinline__ float ex2(float x) {
     float y;
     asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
     return y;
+}
+// z sigmoid(z) where the result is rounded to bf16
+__device__ __forceinline__ float silu(float z) {
+    float r;
+    asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(1.0f + ex2(-attn::LOG2E * z)));
+    return z * r;
 }
 __device__ __forceinline__ void bulk_load(void* dst, const void* src, uint32_t bytes, uint64_t* bar) {
     asm volatile("cp.async.bulk.shared::cta.global.mbarrier::complete_tx::bytes [%0], [%1], %2, [%3];" ::"r"(smem_u32(dst)),
@@ -103,10 +111,12 @@ __device__ __forceinline__ void load_kq(uint8_t* dst, const CUtensorMap* tmK, co
         tc::tma_load_3d(dst + h * 2 * BLK + BLK, tmQ, bar, kvh * D + h * 64, row0, 0);
     }
 }
-// d (+)= A B over `STEPS` contraction steps; per step the operands advance by the given bytes (A K-major over 64-column blocks when A_BLK)
+// d (+)= A B over `STEPS` contraction steps; per step the operands advance by the given bytes (A_BLK, B_BLK: K-major over 64-column
+// blocks).  The two halves of an fp32 operand may be one B of 128 columns, `b_lbo` bytes apart; the 64-column results are then added
+// when they are read back.
 template <int STEPS, int A_STEP, int B_STEP, bool A_BLK = false, bool B_BLK = false>
-__device__ __forceinline__ void mma_steps(uint32_t d, uint32_t a_addr, uint32_t a_lbo, uint32_t b_addr, uint32_t idesc, bool acc) {
-    const tc::DescHalves a = tc::smem_desc_halves(a_addr, a_lbo, 1024), b = tc::smem_desc_halves(b_addr, 16, 1024);
+__device__ __forceinline__ void mma_steps(uint32_t d, uint32_t a_addr, uint32_t a_lbo, uint32_t b_addr, uint32_t b_lbo, uint32_t idesc, bool acc) {
+    const tc::DescHalves a = tc::smem_desc_halves(a_addr, a_lbo, 1024), b = tc::smem_desc_halves(b_addr, b_lbo, 1024);
 #pragma unroll
     for (int k = 0; k < STEPS; ++k) {
         const uint32_t ao = (A_BLK ? (k >> 2) * 2 * BLK + (k & 3) * A_STEP : k * A_STEP) >> 4;
@@ -119,26 +129,43 @@ __device__ __forceinline__ void mma_steps(uint32_t d, uint32_t a_addr, uint32_t 
 // A (16 KB); [K; Q] (32 KB), which gives way to the fp32 blocks of L and X and then to T
 constexpr int PREP_SMEM = 6 * BLK + 1024;
 
-// acc[0 .. 4 Q) = a row of a product of two blocks: sum over m < M of A[m] B[m][0 .. 4 Q)
-template <int M, int Q>
+// acc = four numbers of a row of a product: sum over m < 16 of A[m] B[m][0 .. 4)
 __device__ __forceinline__ void block_row(const float* A, const float* B, float* acc) {
 #pragma unroll
-    for (int j = 0; j < 4 * Q; ++j) acc[j] = 0.f;
+    for (int j = 0; j < 4; ++j) acc[j] = 0.f;
 #pragma unroll
-    for (int m = 0; m < M; m += 4) {
+    for (int m = 0; m < 16; m += 4) {
         const float4 a4 = *reinterpret_cast<const float4*>(A + m);
         const float a[4] = {a4.x, a4.y, a4.z, a4.w};
 #pragma unroll
-        for (int e = 0; e < 4; ++e)
-#pragma unroll
-            for (int q = 0; q < Q; ++q) {
-                const float4 b = *reinterpret_cast<const float4*>(B + (m + e) * LP + 4 * q);
-                acc[4 * q] = fmaf(a[e], b.x, acc[4 * q]);
-                acc[4 * q + 1] = fmaf(a[e], b.y, acc[4 * q + 1]);
-                acc[4 * q + 2] = fmaf(a[e], b.z, acc[4 * q + 2]);
-                acc[4 * q + 3] = fmaf(a[e], b.w, acc[4 * q + 3]);
-            }
+        for (int e = 0; e < 4; ++e) {
+            const float4 b = *reinterpret_cast<const float4*>(B + (m + e) * LP);
+            acc[0] = fmaf(a[e], b.x, acc[0]); acc[1] = fmaf(a[e], b.y, acc[1]); acc[2] = fmaf(a[e], b.z, acc[2]); acc[3] = fmaf(a[e], b.w, acc[3]);
+        }
     }
+}
+// C = s A B for 32 x 32 blocks: thread t < 64 makes a 4 x 4 tile
+__device__ __forceinline__ void block_tile(const float* A, const float* B, float* C, float s, int t) {
+    const int r0 = (t >> 3) * 4, c0 = (t & 7) * 4;
+    float acc[4][4] = {};
+#pragma unroll 1
+    for (int m = 0; m < 32; m += 4) {
+        float a[4][4];
+#pragma unroll
+        for (int r = 0; r < 4; ++r) *reinterpret_cast<float4*>(a[r]) = *reinterpret_cast<const float4*>(A + (r0 + r) * LP + m);
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+            const float4 b = *reinterpret_cast<const float4*>(B + (m + e) * LP + c0);
+#pragma unroll
+            for (int r = 0; r < 4; ++r) {
+                acc[r][0] = fmaf(a[r][e], b.x, acc[r][0]); acc[r][1] = fmaf(a[r][e], b.y, acc[r][1]);
+                acc[r][2] = fmaf(a[r][e], b.z, acc[r][2]); acc[r][3] = fmaf(a[r][e], b.w, acc[r][3]);
+            }
+        }
+    }
+#pragma unroll
+    for (int r = 0; r < 4; ++r)
+        *reinterpret_cast<float4*>(C + (r0 + r) * LP + c0) = make_float4(s * acc[r][0], s * acc[r][1], s * acc[r][2], s * acc[r][3]);
 }
 
 template <int D>
@@ -202,7 +229,7 @@ delta_prepare_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_const
     if (warp == 0 && __all_sync(0xffffffffu, ok)) {
         const uint32_t a = smem_u32(sKQ);
         if (tc::elect_one()) {
-            mma_steps<D / 16, 32, 32, true, true>(tmem, a, 16, a, tc::instr_desc_f16(128, CH, 1, 1, 0, 0), false);
+            mma_steps<D / 16, 32, 32, true, true>(tmem, a, 16, a, 16, tc::instr_desc_f16(128, CH, 1, 1, 0, 0), false);
             tc::tc_commit(&bars[1]);
         }
         __syncwarp();
@@ -228,31 +255,31 @@ delta_prepare_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_const
     } else {
         tc::tc_fence_after();
         const int i = tid & 63;
-        {
-            float x[64];
-            tmem_row64(tmem + lane_base, x);
+        // (loops are kept rolled where they can be: four blocks per SM at different places share the instruction cache)
+#pragma unroll 1
+        for (int h = 0; h < 64; h += 32) {
+            float x[32];
+            tmem_row32(tmem + lane_base + h, x);
             const float gi = gsum[i], s = tid < CH ? unit[i] * beta[i] : unit[tid];
-            const int last = tid < CH ? i - 1 : i;     // columns up to here
+            const int last = (tid < CH ? i - 1 : i) - h;                   // columns up to here
 #pragma unroll
-            for (int j = 0; j < 64; j += 4) {
-                const float4 u = *reinterpret_cast<const float4*>(unit + j), g = *reinterpret_cast<const float4*>(gsum + j);
+            for (int j = 0; j < 32; j += 4) {
+                const float4 u = *reinterpret_cast<const float4*>(unit + h + j), g = *reinterpret_cast<const float4*>(gsum + h + j);
                 x[j] = j <= last ? x[j] * s * u.x * ex2(gi - g.x) : 0.f;
                 x[j + 1] = j + 1 <= last ? x[j + 1] * s * u.y * ex2(gi - g.y) : 0.f;
                 x[j + 2] = j + 2 <= last ? x[j + 2] * s * u.z * ex2(gi - g.z) : 0.f;
                 x[j + 3] = j + 3 <= last ? x[j + 3] * s * u.w * ex2(gi - g.w) : 0.f;
             }
             if (tid < CH) {
-                float* dst = Lb + (i < 32 ? 0 : TB) + (i & 31) * LP;
+                if (h == 0 || i >= 32) {
+                    float* dst = Lb + (i < 32 ? 0 : h ? 2 * TB : TB) + (i & 31) * LP;
 #pragma unroll
-                for (int j = 0; j < 32; j += 4) *reinterpret_cast<float4*>(dst + j) = make_float4(x[j], x[j + 1], x[j + 2], x[j + 3]);
-                if (i >= 32) {
-#pragma unroll
-                    for (int j = 0; j < 32; j += 4)
-                        *reinterpret_cast<float4*>(dst + TB + j) = make_float4(x[32 + j], x[33 + j], x[34 + j], x[35 + j]);
+                    for (int j = 0; j < 32; j += 4) *reinterpret_cast<float4*>(dst + j) = make_float4(x[j], x[j + 1], x[j + 2], x[j + 3]);
                 }
             } else {
-                store_row_split<8>(sA, sA + BLK, i, 0, x);
+                store_row_split<4>(sA, sA + BLK, i, h >> 3, x);
             }
+            __syncwarp();
         }
         __syncthreads();
         // inverses of the four 16 x 16 triangles on the diagonal, one per warp: a column per lane, by substitution
@@ -281,25 +308,18 @@ delta_prepare_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_const
         {                                              // below the diagonal of each 32 x 32 block: X21 = -X22 (L21 X11), 16 x 16
             const int off = (tid >> 6) * 2 * TB, r = (tid & 63) >> 2, c0 = (tid & 3) * 4;
             float acc[4];
-            block_row<16, 1>(Lb + off + (16 + r) * LP, Xb + off + c0, acc);
+            block_row(Lb + off + (16 + r) * LP, Xb + off + c0, acc);
             float* m = M1 + (tid >> 6) * 16 * LP;
             *reinterpret_cast<float4*>(m + r * LP + c0) = make_float4(acc[0], acc[1], acc[2], acc[3]);
             __syncthreads();
-            block_row<16, 1>(Xb + off + (16 + r) * LP + 16, m + c0, acc);
+            block_row(Xb + off + (16 + r) * LP + 16, m + c0, acc);
             *reinterpret_cast<float4*>(Xb + off + (16 + r) * LP + c0) = make_float4(-acc[0], -acc[1], -acc[2], -acc[3]);
         }
         __syncthreads();
-        {                                              // and of the whole: 32 x 32, eight numbers of a row per thread
-            const int r = tid >> 2, c0 = (tid & 3) * 8;
-            float acc[8];
-            block_row<32, 2>(Lb + TB + r * LP, Xb + c0, acc);
-            *reinterpret_cast<float4*>(M1 + r * LP + c0) = make_float4(acc[0], acc[1], acc[2], acc[3]);
-            *reinterpret_cast<float4*>(M1 + r * LP + c0 + 4) = make_float4(acc[4], acc[5], acc[6], acc[7]);
-            __syncthreads();
-            block_row<32, 2>(Xb + 2 * TB + r * LP, M1 + c0, acc);
-            *reinterpret_cast<float4*>(Xb + TB + r * LP + c0) = make_float4(-acc[0], -acc[1], -acc[2], -acc[3]);
-            *reinterpret_cast<float4*>(Xb + TB + r * LP + c0 + 4) = make_float4(-acc[4], -acc[5], -acc[6], -acc[7]);
-        }
+        // and of the whole, 32 x 32: a 4 x 4 tile per thread of two warps
+        if (tid < 64) block_tile(Lb + TB, Xb, M1, 1.f, tid);
+        __syncthreads();
+        if (tid < 64) block_tile(Xb + 2 * TB, M1, Xb + TB, -1.f, tid);
         __syncthreads();
         uint8_t* tt = p.tt + ((long long)slot * p.H + head) * TT_BYTES;
         {                                              // T = X diag(beta): half a row per thread
@@ -323,12 +343,11 @@ delta_prepare_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_const
         __syncthreads();
         if (warp == 0) {
             tc::tc_fence_after();
-            const uint32_t a = smem_u32(sA), t = smem_u32(sT), id = tc::instr_desc_f16(128, CH, 1, 1, 0, 1);
+            const uint32_t a = smem_u32(sA), t = smem_u32(sT);
             // the operand's rows 64 .. 127 (what follows in shared memory) give rows that are not looked at
             if (tc::elect_one()) {
-                mma_steps<4, 32, 2048>(tmem + 64, a, 16, t, id, false);
-                mma_steps<4, 32, 2048>(tmem + 64, a, 16, t + BLK, id, true);
-                mma_steps<4, 32, 2048>(tmem + 64, a + BLK, 16, t, id, true);
+                mma_steps<4, 32, 2048>(tmem, a, 16, t, BLK, tc::instr_desc_f16(128, 128, 1, 1, 0, 1), false);
+                mma_steps<4, 32, 2048>(tmem, a + BLK, 16, t, 16, tc::instr_desc_f16(128, 64, 1, 1, 0, 1), true);
                 tc::tc_commit(&bars[1]);
             }
             __syncwarp();
@@ -351,9 +370,12 @@ delta_prepare_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_const
         if (tc::mbar_wait(&bars[1], 1, &abort_flag)) {
             tc::tc_fence_after();
             if (warp < 2) {
-                float x[64];
-                tmem_row64(tmem + 64 + lane_base, x);
-                store_row_split<8>(tt + BLK, tt + 3 * BLK, i, 0, x);
+#pragma unroll 1
+                for (int h = 0; h < 2; ++h) {
+                    float x[32];
+                    tmem_sum32(tmem + lane_base + h * 32, x);
+                    store_row_split<4>(tt + BLK, tt + 3 * BLK, i, h * 4, x);
+                }
             }
         } else if (lane == 0) {
             atomicMax(p.status, (int)KB_TIMEOUT_MMA);
@@ -438,7 +460,7 @@ delta_scan_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constant
     const bf16* vsrc = p.v + (long long)(row0 + i) * vstride + head * p.dvt + col0;
     bf16* odst = p.o + (long long)(row0 + i) * vstride + head * p.dvt + col0;
     const uint32_t aKQ = smem_u32(sKQ), aTT = smem_u32(sTT), aS = smem_u32(sS), aRU = smem_u32(sRU);
-    const uint32_t id_kb = tc::instr_desc_f16(128, 64, 1, 1, 0, 1), id_mb = tc::instr_desc_f16(128, 64, 1, 1, 1, 1);
+    const uint32_t id_k = tc::instr_desc_f16(128, 64, 1, 1, 0, 1), id_m = tc::instr_desc_f16(128, 64, 1, 1, 1, 1);
     // values and scalars of a chunk, fetched while the chunk in front of it is worked on
     uint4 v[4];
     float e, eu, decay;
@@ -465,8 +487,8 @@ delta_scan_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constant
             failed |= !tc::mbar_wait(bars, c & 1, abort_flag);
             tc::tc_fence_after();
             if (!__any_sync(0xffffffffu, failed) && tc::elect_one()) {
-                mma_steps<D / 16, 32, 2048, true>(tmem0, aKQ, 16, aS, id_kb, false);
-                mma_steps<D / 16, 32, 2048, true>(tmem0, aKQ, 16, aS + L::S_HALF, id_kb, true);
+                mma_steps<D / 16, 32, 2048, true>(tmem0, aKQ, 16, aS, 16, id_k, false);
+                mma_steps<D / 16, 32, 2048, true>(tmem0, aKQ, 16, aS + L::S_HALF, 16, id_k, true);
                 tc::tc_commit(bars + 2);
             }
             __syncwarp();
@@ -496,9 +518,9 @@ delta_scan_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constant
             failed |= !tc::mbar_wait(bars + 1, c & 1, abort_flag);
             tc::tc_fence_after();
             if (!__any_sync(0xffffffffu, failed) && tc::elect_one()) {
-                mma_steps<4, 32, 2048>(tmem0 + 64, aTT, 16, aRU, id_kb, false);
-                mma_steps<4, 32, 2048>(tmem0 + 64, aTT, 16, aRU + BLK, id_kb, true);
-                mma_steps<4, 32, 2048>(tmem0 + 64, aTT + 2 * BLK, 16, aRU, id_kb, true);
+                mma_steps<4, 32, 2048>(tmem0 + 64, aTT, 16, aRU, 16, id_k, false);
+                mma_steps<4, 32, 2048>(tmem0 + 64, aTT, 16, aRU + BLK, 16, id_k, true);
+                mma_steps<4, 32, 2048>(tmem0 + 64, aTT + 2 * BLK, 16, aRU, 16, id_k, true);
                 tc::tc_commit(bars + 2);
             }
             __syncwarp();
@@ -526,8 +548,8 @@ delta_scan_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constant
         if (warp == 0) {                               // K^T U
             tc::tc_fence_after();
             if (tc::elect_one()) {
-                mma_steps<4, 2048, 2048>(tmem0 + 128, aKQ, 2 * BLK, aRU, id_mb, false);
-                mma_steps<4, 2048, 2048>(tmem0 + 128, aKQ, 2 * BLK, aRU + BLK, id_mb, true);
+                mma_steps<4, 2048, 2048>(tmem0 + 128, aKQ, 2 * BLK, aRU, 16, id_m, false);
+                mma_steps<4, 2048, 2048>(tmem0 + 128, aKQ, 2 * BLK, aRU + BLK, 16, id_m, true);
                 tc::tc_commit(bars + 2);
             }
             __syncwarp();
@@ -576,7 +598,7 @@ struct ConvParams {
     const bf16* rows;
     long long stride;
     int col_q, col_k, col_v;
-    const float* conv;                                 // [2 G d + H dv, taps]
+    const float* conv;                                 // [taps, 2 G d + H dv]
     int N, B, H, G, d, dv, D, dvt;
     bf16* ring;                                        // [num_states, H, ring_rows, 2 d + dv]
     int ring_rows, num_states;
@@ -587,7 +609,7 @@ constexpr int CONV_TOKENS = 32, CONV_GROUP = 8;
 
 // A thread makes eight neighbouring channels of up to CONV_TOKENS neighbouring tokens; the inputs of CONV_GROUP tokens are fetched together.
 template <int TAPS>
-__global__ void __launch_bounds__(128) delta_conv_kernel(const ConvParams p) {
+__global__ void __launch_bounds__(128, 4) delta_conv_kernel(const ConvParams p) {
     const int vecs = (2 * p.G * p.d + p.H * p.dv) / 8, vec = blockIdx.y * 128 + threadIdx.x;
     if (vec >= vecs) return;
     const int ch = vec * 8, nq = p.G * p.d;
@@ -611,9 +633,7 @@ __global__ void __launch_bounds__(128) delta_conv_kernel(const ConvParams p) {
     }
     float w[TAPS][8], past[TAPS][8];                   // past[j]: the input j tokens back
 #pragma unroll
-    for (int j = 0; j < TAPS; ++j)
-#pragma unroll
-        for (int e = 0; e < 8; ++e) w[j][e] = p.conv[(long long)(ch + e) * TAPS + TAPS - 1 - j];
+    for (int j = 0; j < TAPS; ++j) load8(p.conv + (long long)(TAPS - 1 - j) * (2 * nq + p.H * p.dv) + ch, w[j]);
     const int t0 = blockIdx.x * CONV_TOKENS, t1 = min(p.N, t0 + CONV_TOKENS);
     int b = 0, hi = p.B;
     while (hi - b > 1) {
@@ -621,54 +641,63 @@ __global__ void __launch_bounds__(128) delta_conv_kernel(const ConvParams p) {
         if (p.cu[m] <= t0) b = m; else hi = m;
     }
     int next = b + 1 < p.B ? p.cu[b + 1] : p.N;
-    bool enter = true;
+    // the inputs in front of token t, which is the first of this thread's or of its sequence
+    auto enter = [&](int t) {
+        const int lo = p.cu[b], n = p.cu[b + 1] - lo, slot = p.slots[b];
+        const bool fresh = slot < 0 || slot >= p.num_states || p.ctx[b] <= n;
+#pragma unroll
+        for (int j = 1; j < TAPS; ++j) {
+            if (t - j >= lo) load8(p.rows + (long long)(t - j) * p.stride + col, past[j]);
+            else if (!fresh) {
+                // row r of the ring is the input TAPS - 1 - r tokens in front of the pass
+                const bf16* r = p.ring + (((long long)slot * p.H + ring_head) * p.ring_rows + (TAPS - 1 - (j - (t - lo)))) * (2 * p.d + p.dv) + ring_col;
+#pragma unroll
+                for (int e = 0; e < 8; ++e) past[j][e] = to_float(r[e]);
+            } else {
+#pragma unroll
+                for (int e = 0; e < 8; ++e) past[j][e] = 0.f;
+            }
+        }
+    };
+    auto token = [&](int t, const uint4& in) {
+        unpack8(*reinterpret_cast<const bf16x8*>(&in), past[0]);
+        float z[8];
+#pragma unroll
+        for (int e = 0; e < 8; e += 2) {
+            float2 a = __fmul2_rn(make_float2(past[TAPS - 1][e], past[TAPS - 1][e + 1]), make_float2(w[TAPS - 1][e], w[TAPS - 1][e + 1]));
+#pragma unroll
+            for (int j = TAPS - 2; j >= 0; --j) a = __ffma2_rn(make_float2(past[j][e], past[j][e + 1]), make_float2(w[j][e], w[j][e + 1]), a);
+            z[e] = silu(a.x);
+            z[e + 1] = silu(a.y);
+        }
+        store8(dst + (long long)t * dst_stride, z);
+#pragma unroll
+        for (int j = TAPS - 1; j > 0; --j)
+#pragma unroll
+            for (int e = 0; e < 8; ++e) past[j][e] = past[j - 1][e];
+    };
+    enter(t0);
     for (int tg = t0; tg < t1; tg += CONV_GROUP) {
         uint4 in8[CONV_GROUP];
 #pragma unroll
         for (int u = 0; u < CONV_GROUP; ++u)
             if (tg + u < t1) in8[u] = *reinterpret_cast<const uint4*>(p.rows + (long long)(tg + u) * p.stride + col);
+        if (tg + CONV_GROUP <= min(next, t1)) {        // inside one sequence
 #pragma unroll
-        for (int u = 0; u < CONV_GROUP; ++u) {
-            const int t = tg + u;
-            if (t >= t1) break;
-            while (b + 1 < p.B && t >= next) {
-                ++b;
-                next = b + 1 < p.B ? p.cu[b + 1] : p.N;
-                enter = true;
-            }
-            if (enter) {
-                enter = false;
-                const int lo = p.cu[b], n = p.cu[b + 1] - lo, slot = p.slots[b];
-                const bool fresh = slot < 0 || slot >= p.num_states || p.ctx[b] <= n;
+            for (int u = 0; u < CONV_GROUP; ++u) token(tg + u, in8[u]);
+        } else {
 #pragma unroll
-                for (int j = 1; j < TAPS; ++j) {
-                    if (t - j >= lo) load8(p.rows + (long long)(t - j) * p.stride + col, past[j]);
-                    else if (!fresh) {
-                        // row r of the ring is the input TAPS - 1 - r tokens in front of the pass
-                        const bf16* r = p.ring + (((long long)slot * p.H + ring_head) * p.ring_rows + (TAPS - 1 - (j - (t - lo)))) * (2 * p.d + p.dv) + ring_col;
-#pragma unroll
-                        for (int e = 0; e < 8; ++e) past[j][e] = to_float(r[e]);
-                    } else {
-#pragma unroll
-                        for (int e = 0; e < 8; ++e) past[j][e] = 0.f;
+            for (int u = 0; u < CONV_GROUP; ++u) {
+                if (tg + u >= t1) break;
+                if (tg + u >= next) {
+                    while (b + 1 < p.B && tg + u >= next) {
+                        ++b;
+                        next = b + 1 < p.B ? p.cu[b + 1] : p.N;
                     }
+                    enter(tg + u);
                 }
+                token(tg + u, in8[u]);
             }
-            unpack8(*reinterpret_cast<const bf16x8*>(&in8[u]), past[0]);
-            float z[8];
-#pragma unroll
-            for (int e = 0; e < 8; ++e) z[e] = past[TAPS - 1][e] * w[TAPS - 1][e];
-#pragma unroll
-            for (int j = TAPS - 2; j >= 0; --j)
-#pragma unroll
-                for (int e = 0; e < 8; ++e) z[e] = fmaf(past[j][e], w[j][e], z[e]);
-#pragma unroll
-            for (int e = 0; e < 8; ++e) z[e] = silu(z[e]);
-            store8(dst + (long long)t * dst_stride, z);
-#pragma unroll
-            for (int j = TAPS - 1; j > 0; --j)
-#pragma unroll
-                for (int e = 0; e < 8; ++e) past[j][e] = past[j - 1][e];
         }
     }
 }

@@ -892,6 +892,10 @@ class CudaOps(TorchOps):
 
     def paged_attention(self, q, k_pages, v_pages, page_table, ctx_lens, cu_seqlens, max_ctx, scale, softcap, chunk, gate, vdim, cols):
         N, H, kd = q.shape
+        B = page_table.shape[0]
+        if ctx_lens.numel() != B or (cu_seqlens.numel() - 1 if cu_seqlens is not None else N) != B:
+            raise KernelError(f"paged attention: {B} page lists, {ctx_lens.numel()} lengths, {N} rows, boundaries "
+                              f"{None if cu_seqlens is None else tuple(cu_seqlens.shape)}")
         out = torch.empty(N, H * cols, device=q.device, dtype=q.dtype)
         self._call("kb_paged_attn_plain", _p(q), _p(k_pages), _p(v_pages), _I(k_pages.shape[1]), _I(kd), _I(v_pages.shape[3]), _p(page_table),
                    _I(page_table.shape[1]), _I(k_pages.shape[0]), _p(ctx_lens), _p(cu_seqlens), _I(page_table.shape[0]), _p(gate),
@@ -907,7 +911,10 @@ class CudaOps(TorchOps):
         cols = [0]
         for n in (G * d, G * d, H * dv, H * dv, H):
             cols.append(cols[-1] + up8(n))
-        width, taps, B, dev = up8(H * dv), conv.shape[1], slots.numel(), rows.device
+        width, taps, B, dev = up8(H * dv), conv.shape[0], slots.numel(), rows.device
+        if ctx_lens.numel() != B or (cu_seqlens.numel() - 1 if cu_seqlens is not None else N) != B:
+            raise KernelError(f"delta rule: {B} state slots, {ctx_lens.numel()} lengths, {N} rows, boundaries "
+                              f"{None if cu_seqlens is None else tuple(cu_seqlens.shape)}")
         out = (torch.empty if width == H * dv else torch.zeros)(N, width, device=dev, dtype=rows.dtype)
         if (rows.dtype == torch.bfloat16 and cu_seqlens is not None and max_q > self.delta_short
                 and self.lib.kb_delta_chunk_ok(_I(H), _I(G), _I(d), _I(dv), _I(taps))):

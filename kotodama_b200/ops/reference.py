@@ -875,7 +875,7 @@ class TorchOps:
 
     def delta_rule(self, rows, H, G, d, dv, conv, a_log, dt_bias, norm, eps, state, ring, slots, cu_seqlens, ctx_lens, max_q):
         """Gated delta rule over packed tokens.  ``rows[N, *]`` hold ``q [G, d] | k [G, d] | v [H, dv] | gate [H, dv] | b [H] |
-        a [H]``, each part starting at a multiple of eight columns; ``conv[2 G d + H dv, taps]`` are the short convolutions of q, k and v.  Sequence
+        a [H]``, each part starting at a multiple of eight columns; ``conv[taps, 2 G d + H dv]`` are the short convolutions of q, k and v.  Sequence
         ``i`` owns rows ``cu_seqlens[i:i+2]`` (None: row ``i``), the last of its ``ctx_lens[i]`` tokens, and continues from
         ``state[slots[i]]`` (``[H, d, dv'>=dv]`` fp32) and ``ring[slots[i]]`` (``[H, taps - 1, 2 d + dv]``, the convolutions' last inputs);
         both are replaced.  A sequence that starts here starts from zero; a negative slot keeps nothing.  Per head
@@ -884,7 +884,8 @@ class TorchOps:
 
         with ``g = exp(-exp(a_log) softplus(a + dt_bias))``, ``beta = sigmoid(b)`` and unit vectors ``k``, ``q sqrt(d)``.  Returns
         ``rms(o) * norm * silu(gate)``, ``[N, H * dv]`` with rows padded to a multiple of eight."""
-        N, taps = rows.shape[0], conv.shape[1]
+        N, taps = rows.shape[0], conv.shape[0]
+        conv = conv.t()
         up8 = lambda n: (n + 7) // 8 * 8
         rep = H // G
         starts = [0]
@@ -893,8 +894,8 @@ class TorchOps:
         part = lambda i, n: _f(rows[:, starts[i]: starts[i] + n])
         heads = lambda z: z.reshape(-1, G, d).repeat_interleave(rep, 1)
         raw = torch.cat([heads(part(0, G * d)), heads(part(1, G * d)), part(2, H * dv).reshape(N, H, dv)], -1)      # [N, H, 2 d + dv]
-        w = torch.cat([conv[: G * d].view(G, d, taps).repeat_interleave(rep, 0), conv[G * d: 2 * G * d].view(G, d, taps).repeat_interleave(rep, 0),
-                       conv[2 * G * d:].view(H, dv, taps)], 1)                                                      # [H, 2 d + dv, taps]
+        w = torch.cat([conv[: G * d].reshape(G, d, taps).repeat_interleave(rep, 0), conv[G * d: 2 * G * d].reshape(G, d, taps).repeat_interleave(rep, 0),
+                       conv[2 * G * d:].reshape(H, dv, taps)], 1)                                                      # [H, 2 d + dv, taps]
         gate, beta = part(3, H * dv).reshape(N, H, dv), torch.sigmoid(part(4, H))
         g = torch.exp(-torch.exp(a_log) * F.softplus(part(5, H) + dt_bias))
         out = torch.zeros(N, up8(H * dv), device=rows.device, dtype=rows.dtype)

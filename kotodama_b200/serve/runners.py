@@ -328,7 +328,7 @@ class HybridRunner:
                 lw["wo"] = dw(o.reshape(Dp, m.heads * lw["cols"]))
             else:
                 lw["win"] = dw(fuse([x("q"), x("k"), x("v"), x("g"), x("b"), x("a")]))
-                lw["conv"] = torch.cat([f32(x(n + ".conv")) for n in "qkv"])
+                lw["conv"] = torch.cat([f32(x(n + ".conv")) for n in "qkv"]).t().contiguous()
                 lw.update(a_log=f32(x("A_log")), dt=f32(x("dt_bias")), norm=f32(x("norm")))
                 lw["wo"] = dw(pad(put(x("o")), Dp, _up(m.heads * m.vdim, 8)))
             if layer.mlp is not None:
