@@ -371,10 +371,12 @@ paged_decode_stream_kernel(const bf16* __restrict__ q, long long q_stride, const
     }
 }
 
-// Merge the splits: out[req][head][d] = sum_s e^{m_s - M} o_s[d] / sum_s e^{m_s - M} l_s
+// Merge the splits: out[req][head][d] = sum_s e^{m_s - M} o_s[d] / sum_s e^{m_s - M} l_s, with a gate times its sigmoid; `cols`
+// leading columns per head are written
 template <int HD>
 __global__ void paged_merge_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml,
-                                   bf16* __restrict__ out, long long out_stride, int n_kv, int G, int nsplit) {
+                                   bf16* __restrict__ out, long long out_stride, int n_kv, int G, int nsplit,
+                                   const bf16* __restrict__ gate, long long gate_stride, int cols) {
     kb_dep_trigger();
     kb_dep_wait();
     const int req = blockIdx.x, head = blockIdx.y;
@@ -394,7 +396,8 @@ __global__ void paged_merge_kernel(const float* __restrict__ part_o, const float
         den += w * l;
         if (d < HD) num += w * part_o[(pb * G + g) * HD + d];
     }
-    if (d < HD) out[(size_t)req * out_stride + (size_t)head * HD + d] = __float2bfloat16(den > 0.f ? num / den : 0.f);
+    if (gate) num /= 1.f + __expf(-__bfloat162float(gate[(size_t)req * gate_stride + head]));
+    if (d < cols) out[(size_t)req * out_stride + (size_t)head * cols + d] = __float2bfloat16(den > 0.f ? num / den : 0.f);
 }
 
 // Bulk-copy variant of the streaming kernel (the default for head_dim 128): with the head-major page layout
@@ -631,6 +634,20 @@ constexpr int MMA_PAGE = 2 * MMA_HALF;               // one staged (page, head) 
 constexpr int MMA_NST = 2;                           // pages in flight per warp
 constexpr int MMA_SMEM = 4 * MMA_NST * 2 * MMA_PAGE + 1024;
 
+// Attention with more to it than the plain causal form (EXT below): only keys of the query's own chunk of the sequence
+// (`chunk` tokens, counted from position 0; 0: all), scores through softcap * tanh(score / softcap) (0: none), several groups of
+// G query heads per KV head (`groups`); scores are scaled after the product, in fp32.
+struct DecodeExt {
+    int chunk, groups;
+    float softcap;
+};
+__device__ __forceinline__ float cap_log2(float s, float scale, float cap) {      // capped score in log2 units
+    const float L2E = 1.4426950408889634f;
+    s *= scale;
+    if (cap > 0.f) s = cap * (1.0f - __fdividef(2.0f, 1.0f + exp2f(fminf(s / cap * (2.0f * L2E), 100.f))));
+    return s * L2E;
+}
+
 __device__ __forceinline__ void tma_load_2d_dec(void* dst, const CUtensorMap* m, uint64_t* bar, int x, int y) {
     asm volatile(
         "cp.async.bulk.tensor.2d.shared::cta.global.tile.mbarrier::complete_tx::bytes [%0], [%1, {%3, %4}], [%2];"
@@ -681,14 +698,14 @@ __device__ __forceinline__ void merge_by_last_cta(const float* part_o, const flo
     }
 }
 
-template <int G>
+template <int G, int HD = 128, bool EXT = false>
 __global__ void __launch_bounds__(128, 3)
 paged_decode_mma_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constant__ CUtensorMap tmV,
                         const bf16* __restrict__ q, long long q_stride, const int* __restrict__ page_table, int max_pages,
                         const int* __restrict__ ctx_lens, int n_kv, int split_tokens, float scale,
                         float* part_o, float* part_ml, int nsplit, bf16* __restrict__ out, long long out_stride,
-                        unsigned* merge_counters) {
-    constexpr int HD = 128;
+                        unsigned* merge_counters, const DecodeExt ext) {
+    constexpr int MMA_PAGE = HD / 64 * MMA_HALF;         // one staged (page, head) block of K or V
     extern __shared__ uint8_t ring_unaligned[];
     uint8_t* ring_raw = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(ring_unaligned) + 1023) & ~uintptr_t(1023));
     __shared__ __align__(16) bf16 qs[G][HD];
@@ -699,7 +716,14 @@ paged_decode_mma_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_co
     const int kvh = blockIdx.x, req = blockIdx.y, sp = blockIdx.z;
     kb_dep_trigger();
     kb_dep_wait();                      // the rows appended to the pages and the queries come from the kernels before
-    const int ctx = ctx_lens[req];
+    const int page_head = EXT ? kvh / ext.groups : kvh, page_heads = EXT ? n_kv / ext.groups : n_kv;
+    int ctx = ctx_lens[req], page0 = 0, skip = 0;        // keys begin `skip` tokens into page `page0`
+    if (EXT && ext.chunk > 0) {
+        const int begin = (ctx - 1) / ext.chunk * ext.chunk;
+        page0 = begin / PAGE;
+        skip = begin % PAGE;
+        ctx -= page0 * PAGE;
+    }
     const int t0 = sp * split_tokens;
     const int nt = min(split_tokens, ctx - t0);
     const size_t pbase = ((size_t)(req * n_kv + kvh) * nsplit + sp);
@@ -708,17 +732,17 @@ paged_decode_mma_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_co
             part_ml[(pbase * G + threadIdx.x) * 2] = -INFINITY;
             part_ml[(pbase * G + threadIdx.x) * 2 + 1] = 0.f;
         }
-        if (merge_counters) merge_by_last_cta<G>(part_o, part_ml, out, out_stride, merge_counters, req, kvh, n_kv, nsplit);
+        if (!EXT && merge_counters) merge_by_last_cta<G>(part_o, part_ml, out, out_stride, merge_counters, req, kvh, n_kv, nsplit);
         return;
     }
     const int npages = (nt + PAGE - 1) / PAGE;
-    const float qscale = scale * 1.4426950408889634f;
+    const float qscale = EXT ? 1.f : scale * 1.4426950408889634f;
     for (int i = threadIdx.x; i < G * HD; i += blockDim.x) {
         const int g = i / HD, d = i % HD;
         qs[g][d] = __float2bfloat16(__bfloat162float(q[(size_t)req * q_stride + (size_t)(kvh * G + g) * HD + d]) * qscale);
     }
     for (int i = threadIdx.x; i < npages; i += blockDim.x)
-        spage[i] = page_table[(size_t)req * max_pages + t0 / PAGE + i];
+        spage[i] = page_table[(size_t)req * max_pages + page0 + t0 / PAGE + i];
     if (threadIdx.x == 0) {
         for (int w = 0; w < 4; ++w)
             for (int s = 0; s < MMA_NST; ++s) tc::mbar_init(&full[w][s], 1);
@@ -733,27 +757,28 @@ paged_decode_mma_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_co
         if (lane == 0) {
             const int st = i % MMA_NST;
             uint8_t* dst = ring + (size_t)(st * 2) * MMA_PAGE;
-            const int row0 = (spage[warp + 4 * i] * n_kv + kvh) * PAGE;     // row of the [pages * heads * 16, 128] view
+            const int row0 = (spage[warp + 4 * i] * page_heads + page_head) * PAGE;     // row of the [pages * heads * 16, HD] view
             tc::mbar_expect_tx(&full[warp][st], 2 * MMA_PAGE);
-            tma_load_2d_dec(dst, &tmK, &full[warp][st], 0, row0);
-            tma_load_2d_dec(dst + MMA_HALF, &tmK, &full[warp][st], 64, row0);
-            tma_load_2d_dec(dst + MMA_PAGE, &tmV, &full[warp][st], 0, row0);
-            tma_load_2d_dec(dst + MMA_PAGE + MMA_HALF, &tmV, &full[warp][st], 64, row0);
+#pragma unroll
+            for (int h = 0; h < HD / 64; ++h) {
+                tma_load_2d_dec(dst + h * MMA_HALF, &tmK, &full[warp][st], h * 64, row0);
+                tma_load_2d_dec(dst + MMA_PAGE + h * MMA_HALF, &tmV, &full[warp][st], h * 64, row0);
+            }
         }
     };
     for (int i = 0; i < MMA_NST && i < my_pages; ++i) issue(i);
 
     // Q fragments: row g = lane / 4 of the A operand (zero for g >= G), k = 16 ks + 2 (lane % 4) [+ 8]
     const int g_row = lane >> 2, qd = lane & 3;
-    uint32_t qa0[8], qa2[8];
+    uint32_t qa0[HD / 16], qa2[HD / 16];
 #pragma unroll
-    for (int ks = 0; ks < 8; ++ks) {
+    for (int ks = 0; ks < HD / 16; ++ks) {
         qa0[ks] = g_row < G ? *reinterpret_cast<const uint32_t*>(&qs[g_row < G ? g_row : 0][ks * 16 + 2 * qd]) : 0u;
         qa2[ks] = g_row < G ? *reinterpret_cast<const uint32_t*>(&qs[g_row < G ? g_row : 0][ks * 16 + 8 + 2 * qd]) : 0u;
     }
-    float o[16][4];
+    float o[HD / 8][4];
 #pragma unroll
-    for (int j = 0; j < 16; ++j) o[j][0] = o[j][1] = o[j][2] = o[j][3] = 0.f;
+    for (int j = 0; j < HD / 8; ++j) o[j][0] = o[j][1] = o[j][2] = o[j][3] = 0.f;
     float m = -INFINITY, l = 0.f;
     bool ok = true;
     // ldmatrix lane addressing: K matrices are (tokens 0-7 | 8-15) x (k 0-7 | 8-15) of a 16-wide k step, V
@@ -769,7 +794,7 @@ paged_decode_mma_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_co
         const uint32_t kb = smem_u32(ring + (size_t)(st * 2) * MMA_PAGE), vb = kb + MMA_PAGE;
         float s0[4] = {0.f, 0.f, 0.f, 0.f}, s1[4] = {0.f, 0.f, 0.f, 0.f};
 #pragma unroll
-        for (int ks = 0; ks < 8; ++ks) {
+        for (int ks = 0; ks < HD / 16; ++ks) {
             uint32_t b00, b01, b10, b11;
             ldsm_x4(kb + swz_off(k_row, ks * 2 + k_sub), b00, b01, b10, b11);
             mma_16816(s0, qa0[ks], qa2[ks], b00, b01);
@@ -777,21 +802,28 @@ paged_decode_mma_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_co
         }
         // online softmax on row g_row: this lane holds tokens 2 qd, 2 qd + 1, 8 + 2 qd, 9 + 2 qd of the page
         const int tok0 = (warp + 4 * i) * PAGE + 2 * qd;
+        if (EXT) {
+            const int out = skip - t0;                   // tokens in front of this one belong to another chunk
+            s0[0] = tok0 < out ? -INFINITY : cap_log2(s0[0], scale, ext.softcap);
+            s0[1] = tok0 + 1 < out ? -INFINITY : cap_log2(s0[1], scale, ext.softcap);
+            s1[0] = tok0 + 8 < out ? -INFINITY : cap_log2(s1[0], scale, ext.softcap);
+            s1[1] = tok0 + 9 < out ? -INFINITY : cap_log2(s1[1], scale, ext.softcap);
+        }
         const float v00 = tok0 < nt ? s0[0] : -INFINITY, v01 = tok0 + 1 < nt ? s0[1] : -INFINITY;
         const float v10 = tok0 + 8 < nt ? s1[0] : -INFINITY, v11 = tok0 + 9 < nt ? s1[1] : -INFINITY;
         float mx = fmaxf(fmaxf(v00, v01), fmaxf(v10, v11));
         mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 1));
         mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 2));
-        const float mn = fmaxf(m, mx);                   // finite: the first token of a staged page is always valid
+        const float mn = fmaxf(m, mx);                   // finite: a staged page has a valid token
         const float f = exp2f(m - mn);
         m = mn;
         const float p00 = exp2f(v00 - mn), p01 = exp2f(v01 - mn), p10 = exp2f(v10 - mn), p11 = exp2f(v11 - mn);
         l = l * f + (p00 + p01) + (p10 + p11);
         const uint32_t pa0 = pack2_bf16(p00, p01), pa2 = pack2_bf16(p10, p11);
 #pragma unroll
-        for (int j = 0; j < 16; ++j) { o[j][0] *= f; o[j][1] *= f; }
+        for (int j = 0; j < HD / 8; ++j) { o[j][0] *= f; o[j][1] *= f; }
 #pragma unroll
-        for (int j = 0; j < 8; ++j) {
+        for (int j = 0; j < HD / 16; ++j) {
             uint32_t b0, b1, b2, b3;
             ldsm_x4_trans(vb + swz_off(v_row, j * 2 + v_sub), b0, b1, b2, b3);
             mma_16816(o[2 * j], pa0, pa2, b0, b1);
@@ -821,7 +853,7 @@ paged_decode_mma_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_co
     float* wo_w = reinterpret_cast<float*>(ring);
     if (g_row < G) {
 #pragma unroll
-        for (int j = 0; j < 16; ++j) {
+        for (int j = 0; j < HD / 8; ++j) {
             wo_w[g_row * HD + 8 * j + 2 * qd] = m == -INFINITY ? 0.f : o[j][0];
             wo_w[g_row * HD + 8 * j + 2 * qd + 1] = m == -INFINITY ? 0.f : o[j][1];
         }
@@ -852,7 +884,7 @@ paged_decode_mma_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_co
         part_ml[(pbase * G + g) * 2] = mxx == -INFINITY ? -INFINITY : mxx * 0.6931471805599453f;
         part_ml[(pbase * G + g) * 2 + 1] = sum;
     }
-    if (merge_counters) merge_by_last_cta<G>(part_o, part_ml, out, out_stride, merge_counters, req, kvh, n_kv, nsplit);
+    if (!EXT && merge_counters) merge_by_last_cta<G>(part_o, part_ml, out, out_stride, merge_counters, req, kvh, n_kv, nsplit);
 }
 
 // Reads the decode status word and clears it, so that one timeout is reported once.
@@ -869,8 +901,8 @@ KB_API int kb_decode_status() {
 typedef CUresult (*EncodeTiledFnDec)(CUtensorMap*, CUtensorMapDataType, cuuint32_t, void*, const cuuint64_t*,
                                      const cuuint64_t*, const cuuint32_t*, const cuuint32_t*, CUtensorMapInterleave,
                                      CUtensorMapSwizzle, CUtensorMapL2promotion, CUtensorMapFloatOOBfill);
-// pages [num_pages][n_kv][16][128] bf16 seen as rows of 128 elements; a box is half a (page, head) block
-static int make_page_tmap(CUtensorMap* m, const void* base, long long rows) {
+// pages [num_pages][n_kv][16][hd] bf16 seen as rows of hd elements; a box is 64 columns of a (page, head) block
+static int make_page_tmap(CUtensorMap* m, const void* base, long long rows, int hd = 128) {
     static EncodeTiledFnDec enc = nullptr;
     if (!enc) {
         void* ptr = nullptr;
@@ -880,8 +912,8 @@ static int make_page_tmap(CUtensorMap* m, const void* base, long long rows) {
             return 100;
         enc = reinterpret_cast<EncodeTiledFnDec>(ptr);
     }
-    cuuint64_t dims[2] = {128, (cuuint64_t)rows};
-    cuuint64_t strides[1] = {256};
+    cuuint64_t dims[2] = {(cuuint64_t)hd, (cuuint64_t)rows};
+    cuuint64_t strides[1] = {(cuuint64_t)hd * 2};
     cuuint32_t box[2] = {64, PAGE};
     cuuint32_t estr[2] = {1, 1};
     const CUresult r = enc(m, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, const_cast<void*>(base), dims, strides, box, estr,
@@ -937,7 +969,7 @@ static int paged_decode_impl(const void* q, long long q_stride, const void* k_pa
         if (tr) return tr;                                                                                     \
         const int lr = kb_launch_dep(paged_decode_mma_kernel<G_>, grid, dim3(128), MMA_SMEM, st,               \
             tmK, tmV, (const bf16*)q, q_stride, page_table, max_pages, ctx_lens,                               \
-            n_kv, split_tokens, scale, part_o, part_ml, nsplit, (bf16*)out, out_stride, merge_counters);       \
+            n_kv, split_tokens, scale, part_o, part_ml, nsplit, (bf16*)out, out_stride, merge_counters, DecodeExt{0, 1, 0.f}); \
         if (lr) return lr;                                                                                     \
         merged = merge_counters != nullptr;                                                                    \
     } else if (streaming >= 2 && (HD_) == 128 && (G_) <= 4) {                                                         \
@@ -976,7 +1008,7 @@ static int paged_decode_impl(const void* q, long long q_stride, const void* k_pa
         if (kb_launch_status()) return KB_LAUNCH_FAILED;
         if (merged) return 0;
         return kb_launch_dep(paged_merge_kernel<128>, dim3(B, n_q), dim3(128), 0, st, (const float*)part_o, (const float*)part_ml,
-                             (bf16*)out, out_stride, n_kv, G, nsplit);
+                             (bf16*)out, out_stride, n_kv, G, nsplit, (const bf16*)nullptr, 0ll, 128);
     } else if (hd == 64) {
         switch (G) {
             case 1: DEC(64, 1); break;
@@ -988,7 +1020,7 @@ static int paged_decode_impl(const void* q, long long q_stride, const void* k_pa
         }
         if (kb_launch_status()) return KB_LAUNCH_FAILED;
         return kb_launch_dep(paged_merge_kernel<64>, dim3(B, n_q), dim3(64), 0, st, (const float*)part_o, (const float*)part_ml,
-                             (bf16*)out, out_stride, n_kv, G, nsplit);
+                             (bf16*)out, out_stride, n_kv, G, nsplit, (const bf16*)nullptr, 0ll, 64);
     } else {
         return 5;
     }
@@ -1011,6 +1043,64 @@ KB_API int kb_paged_decode_merged(const void* q, long long q_stride, const void*
                                   cudaStream_t st) {
     return paged_decode_impl(q, q_stride, k_pages, v_pages, page_table, max_pages, ctx_lens, B, n_q, n_kv, hd, max_ctx,
                              split_tokens, scale, part_o, part_ml, out, out_stride, num_pages, merge_counters, st);
+}
+
+// Decode attention with chunked visibility, soft-capped scores and gated outputs (DecodeExt) for any number of query heads per KV
+// head.  hd 64 or 128; q [B, n_q, hd], out [B, n_q * cols]; gate (may be null) [B, n_q] in rows gate_stride apart.  `visible`: most keys a query
+// sees, counted from the start of its first page; workspaces: B * n_q * nsplit * hd and B * n_q * nsplit * 2 floats.
+KB_API int kb_paged_decode_ext(const void* q, const void* k_pages, const void* v_pages, const int* page_table, int max_pages,
+                               const int* ctx_lens, int B, int n_q, int n_kv, int hd, int visible, int split_tokens, float scale, float softcap,
+                               int chunk, const void* gate, long long gate_stride, float* part_o, float* part_ml, void* out, int cols, int num_pages,
+                               cudaStream_t st) {
+    if (B < 1 || B > 65535 || n_kv < 1 || n_q % n_kv || split_tokens % PAGE || split_tokens < PAGE || split_tokens > 2048 || visible < 1 ||
+        num_pages < 1 || cols < 1 || cols > hd || (hd != 64 && hd != 128))
+        return 5;
+    int G = 8;                                           // query heads per block: the largest divisor up to eight
+    const int rep = n_q / n_kv;
+    while (rep % G) --G;
+    const int heads = n_q / G, nsplit = (visible + split_tokens - 1) / split_tokens;
+    if (nsplit > 65535) return 5;
+    CUtensorMap tmK, tmV;
+    const long long page_rows = (long long)num_pages * n_kv * PAGE;
+    int r = make_page_tmap(&tmK, k_pages, page_rows, hd);
+    if (!r) r = make_page_tmap(&tmV, v_pages, page_rows, hd);
+    if (r) return r;
+    const DecodeExt ext{chunk, rep / G, softcap};
+#define DEC_EXT(G_, HD_)                                                                                                     \
+    {                                                                                                                        \
+        static bool flags[64] = {};                                                                                          \
+        bool* done = kb_device_flag(flags);                                                                                  \
+        if (!done) return 7;                                                                                                 \
+        if (!*done) {                                                                                                        \
+            if (cudaFuncSetAttribute(paged_decode_mma_kernel<G_, HD_, true>, cudaFuncAttributeMaxDynamicSharedMemorySize,    \
+                                     MMA_SMEM) != cudaSuccess) return 7;                                                     \
+            *done = true;                                                                                                    \
+        }                                                                                                                    \
+        r = kb_launch_dep(paged_decode_mma_kernel<G_, HD_, true>, dim3(heads, B, nsplit), dim3(128),                         \
+                          HD_ == 128 ? MMA_SMEM : MMA_SMEM / 2 + 512, st, tmK, tmV, (const bf16*)q, (long long)n_q * hd,     \
+                          page_table, max_pages, ctx_lens, heads, split_tokens, scale, part_o, part_ml, nsplit, (bf16*)out,  \
+                          (long long)n_q * cols, (unsigned*)nullptr, ext);                                                   \
+    }
+#define DEC_EXT_G(HD_)                                                                                  \
+    switch (G) {                                                                                        \
+        case 1: DEC_EXT(1, HD_) break;                                                                  \
+        case 2: DEC_EXT(2, HD_) break;                                                                  \
+        case 3: DEC_EXT(3, HD_) break;                                                                  \
+        case 4: DEC_EXT(4, HD_) break;                                                                  \
+        case 5: DEC_EXT(5, HD_) break;                                                                  \
+        case 6: DEC_EXT(6, HD_) break;                                                                  \
+        case 7: DEC_EXT(7, HD_) break;                                                                  \
+        default: DEC_EXT(8, HD_) break;                                                                 \
+    }
+    if (hd == 128) DEC_EXT_G(128) else DEC_EXT_G(64)
+#undef DEC_EXT_G
+#undef DEC_EXT
+    if (r) return r;
+    if (hd == 128)
+        return kb_launch_dep(paged_merge_kernel<128>, dim3(B, n_q), dim3(128), 0, st, (const float*)part_o, (const float*)part_ml, (bf16*)out,
+                             (long long)n_q * cols, heads, G, nsplit, (const bf16*)gate, gate_stride, cols);
+    return kb_launch_dep(paged_merge_kernel<64>, dim3(B, n_q), dim3(64), 0, st, (const float*)part_o, (const float*)part_ml, (bf16*)out,
+                         (long long)n_q * cols, heads, G, nsplit, (const bf16*)gate, gate_stride, cols);
 }
 
 // Greedy sampling: out[row] = argmax_j logits[row][j] (first index on ties).

@@ -897,6 +897,21 @@ class CudaOps(TorchOps):
             raise KernelError(f"paged attention: {B} page lists, {ctx_lens.numel()} lengths, {N} rows, boundaries "
                               f"{None if cu_seqlens is None else tuple(cu_seqlens.shape)}")
         out = torch.empty(N, H * cols, device=q.device, dtype=q.dtype)
+        G, size = k_pages.shape[1], k_pages.shape[3]
+        if q.dtype == torch.bfloat16 and cu_seqlens is None and size in (64, 128) and v_pages.shape[3] == size:
+            # decoding: the tensor-core kernel over splits of the visible keys, short enough to fill the GPU
+            visible = min(max_ctx, chunk + 15) if chunk else max_ctx
+            split = 512
+            while split > 64 and B * G * ((visible + split - 1) // split) < 296:
+                split //= 2
+            nsplit = (visible + split - 1) // split
+            part_o = torch.empty(B * H * nsplit * size, device=q.device, dtype=torch.float32)
+            part_ml = torch.empty(B * H * nsplit * 2, device=q.device, dtype=torch.float32)
+            self._call("kb_paged_decode_ext", _p(q), _p(k_pages), _p(v_pages), _p(page_table), _I(page_table.shape[1]), _p(ctx_lens), _I(B), _I(H),
+                       _I(G), _I(size), _I(visible), _I(split), _F(scale), _F(softcap), _I(chunk), _p(gate),
+                       _LL(gate.stride(0) if gate is not None else 0), _p(part_o), _p(part_ml), _p(out), _I(cols), _I(k_pages.shape[0]), _st())
+            self.launches += 1
+            return out
         self._call("kb_paged_attn_plain", _p(q), _p(k_pages), _p(v_pages), _I(k_pages.shape[1]), _I(kd), _I(v_pages.shape[3]), _p(page_table),
                    _I(page_table.shape[1]), _I(k_pages.shape[0]), _p(ctx_lens), _p(cu_seqlens), _I(page_table.shape[0]), _p(gate),
                    _LL(gate.stride(0) if gate is not None else 0), _p(out), _I(N), _I(H), _I(vdim), _I(cols), _F(scale), _F(softcap), _I(chunk),
