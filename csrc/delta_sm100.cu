@@ -12,8 +12,8 @@
 //   conv      short convolutions + SiLU of q, k and v, to bf16; and the inputs that the next pass's convolutions look back on
 //   prepare   one CTA per (chunk, head), all chunks at once: [K; Q] K^T by tcgen05.mma, the unit norms' scalars, L, the inverse (fp32, two
 //             32 x 32 triangles by substitution and the block between them), A T by tcgen05.mma; T and A T go to global memory
-//   scan      one CTA per (64 value columns, head, sequence) walks the chunks: three tcgen05 products per chunk, [K; Q] S, [T; A T] R
-//             and K^T U, each with all 128 rows of the tile in use; the state stays in registers (fp32)
+//   scan      one CTA per (128 value columns, head, sequence) walks the chunks: three tcgen05 products per chunk; the state stays in
+//             registers (fp32)
 //   finish    output norm and gate
 //
 // Precision: q, k and v are bf16 after their convolutions and enter the products exactly; their unit norms, like all other
@@ -390,206 +390,287 @@ delta_prepare_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_const
 }
 
 // ------------------------------------------------------------------------------------------------ scan
+// The products are taken transposed, with the value columns as the 128 rows of the tile: what a product needs of the state, of R and
+// of U is then in the very lanes of tensor memory where the product before left it, and goes back there as its A operand (two bf16
+// halves); shared memory holds only what the copy engine brings ([K; Q], [T; A T], V and the scalars of two chunks).
+//
+//   MMA1  X^T = S^T [K; Q]^T     128 x 128 (tokens of K | tokens of Q)
+//   MMA2  [U; A U]^T = R^T [T; A T]^T
+//   MMA3  U^T K                  128 x D, added to the decayed state
+//
+// Sixteen warps, each a quarter of the lanes and of the columns: 16 tokens in K's part of X and U (where R and U are made), the same
+// 16 tokens in Q's part (where O is made), 32 rows of the state.  Warp 0 also issues the products, warp 15 the copies.  O leaves
+// through shared memory.
 template <int D>
 struct Scan {
-    static constexpr int KQ = (D / 64) * 2 * BLK, S_HALF = D * 128;
-    static constexpr int OFF_TT = KQ, OFF_S = OFF_TT + TT_BYTES, OFF_RU = OFF_S + 2 * S_HALF, OFF_BAR = OFF_RU + 2 * BLK;
-    static constexpr int SMEM = OFF_BAR + 64;
+    static constexpr int KQ = (D / 64) * 2 * BLK, OFF_TT = KQ, OFF_V = OFF_TT + TT_BYTES, OFF_SC = OFF_V + 2 * BLK;
+    static constexpr int STAGE = OFF_SC + 1024, OFF_O = 2 * STAGE, OFF_BAR = OFF_O + 2 * BLK, SMEM = OFF_BAR + 1024 + 128;
 };
+constexpr int SCAN_WARPS = 16;
+
+// 2 P numbers as two bf16 numbers each into P + P columns of packed pairs (an A operand in tensor memory)
+template <int P>
+__device__ __forceinline__ void tmem_store_split(uint32_t hi, uint32_t lo, const float* x) {
+    uint32_t h[P], l[P];
+#pragma unroll
+    for (int j = 0; j < P; ++j) {
+        const uint32_t a = __float_as_uint(x[2 * j]), b = __float_as_uint(x[2 * j + 1]);
+        h[j] = __byte_perm(a, b, 0x7632);
+        const float ra = __uint_as_float(a) - __uint_as_float(a & 0xffff0000u), rb = __uint_as_float(b) - __uint_as_float(b & 0xffff0000u);
+        l[j] = __byte_perm(__float_as_uint(ra) + 0x8000u, __float_as_uint(rb) + 0x8000u, 0x7632);
+    }
+    if constexpr (P == 16) {
+        tc::tmem_st16(hi, h);
+        tc::tmem_st16(lo, l);
+    } else {
+        tc::tmem_st8(hi, h);
+        tc::tmem_st8(lo, l);
+    }
+}
+__device__ __forceinline__ void scale16(float* x, const float* f) {
+#pragma unroll
+    for (int j = 0; j < 16; j += 4) {
+        const float4 a = *reinterpret_cast<const float4*>(f + j);
+        x[j] *= a.x; x[j + 1] *= a.y; x[j + 2] *= a.z; x[j + 3] *= a.w;
+    }
+}
+// d (+)= A B with A in tensor memory (8 columns per step of 16) and B stepped by the given bytes (B_BLK: K-major over 64-column blocks)
+template <int STEPS, int B_STEP, bool B_BLK = false>
+__device__ __forceinline__ void mma_ts_steps(uint32_t d, uint32_t a_tmem, uint32_t b_addr, uint32_t b_lbo, uint32_t idesc, bool acc) {
+    const tc::DescHalves b = tc::smem_desc_halves(b_addr, b_lbo, 1024);
+#pragma unroll
+    for (int k = 0; k < STEPS; ++k) {
+        const uint32_t bo = (B_BLK ? (k >> 2) * 2 * BLK + (k & 3) * B_STEP : k * B_STEP) >> 4;
+        tc::mma_f16_ts_h(d, a_tmem + 8 * k, b.lo + bo, b.hi, idesc, acc || k > 0);
+    }
+}
 
 template <int D>
-__global__ void __launch_bounds__(256, 2)
-delta_scan_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constant__ CUtensorMap tmQ, const ChunkParams p) {
-    extern __shared__ __align__(1024) uint8_t smem[];
+__global__ void __launch_bounds__(SCAN_WARPS * 32, 1)
+delta_scan_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmV,
+                  const __grid_constant__ CUtensorMap tmO, const ChunkParams p) {
+    extern __shared__ uint8_t smem_raw[];
+    uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
     using L = Scan<D>;
-    uint8_t *sKQ = smem, *sTT = smem + L::OFF_TT, *sS = smem + L::OFF_S, *sRU = smem + L::OFF_RU;
-    uint64_t* bars = reinterpret_cast<uint64_t*>(smem + L::OFF_BAR);      // [K; Q] loaded, [T; A T] loaded, product done
-    uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bars + 3);
+    uint64_t* full = reinterpret_cast<uint64_t*>(smem + L::OFF_BAR);      // [2] a chunk's data is there
+    uint64_t *ready = full + 2, *done = full + 3;      // the next product's operand is there; a product is done
+    uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(full + 4);
     volatile int* abort_flag = reinterpret_cast<volatile int*>(tmem_slot + 1);
     const int tid = threadIdx.x, warp = __shfl_sync(0xffffffffu, tid >> 5, 0);
-    // two threads per tile row, 32 columns each
-    const int row = (warp & 3) * 32 + (tid & 31), hf = warp >> 2;
-    const bool is_k = row < CH;                        // the rows of K (then R, U); the others are those of Q (then O)
     const int tile = blockIdx.x, head = blockIdx.y, b = blockIdx.z, kvh = head / (p.H / p.G);
     const int row0 = p.cu[b], n = p.cu[b + 1] - row0, chunks = (n + CH - 1) / CH;
     if (n <= 0) return;
-    if (smem_u32(smem) & 1023) {                       // uniform: the swizzled tiles need this alignment
-        if (tid == 0) atomicMax(p.status, (int)KB_BAD_ARG);
-        return;
-    }
     const int base = slot_base(p.cu, b);
     const uint8_t* tt = p.tt + ((long long)base * p.H + head) * TT_BYTES;
     const float* sc = p.scal + ((long long)base * p.H + head) * SCALARS;
-    if (tid == 0) {
-        for (int i = 0; i < 3; ++i) tc::mbar_init(bars + i, 1);
-        *abort_flag = 0;
-        tc::fence_barrier_init();
-        load_kq<D>(sKQ, &tmK, &tmQ, bars, kvh, row0);
-        tc::mbar_expect_tx(bars + 1, TT_BYTES);
-        bulk_load(sTT, tt, TT_BYTES, bars + 1);
+    const int boxes = tile * 128 + 64 < p.dvt ? 2 : 1;
+    auto load = [&](int c) {                           // one thread
+        uint8_t* st = smem + (c & 1) * L::STAGE;
+        uint64_t* bar = full + (c & 1);
+        const int at = row0 + c * CH;
+        tc::mbar_expect_tx(bar, (D / 64) * 2 * BLK + TT_BYTES + boxes * BLK + SCALARS * 4);
+#pragma unroll
+        for (int h = 0; h < D / 64; ++h) {
+            tc::tma_load_3d(st + h * 2 * BLK, &tmK, bar, kvh * D + h * 64, at, 0);
+            tc::tma_load_3d(st + h * 2 * BLK + BLK, &tmQ, bar, kvh * D + h * 64, at, 0);
+        }
+        bulk_load(st + L::OFF_TT, tt + (long long)c * p.H * TT_BYTES, TT_BYTES, bar);
+        for (int h = 0; h < boxes; ++h) tc::tma_load_3d(st + L::OFF_V + h * BLK, &tmV, bar, head * p.dvt + tile * 128 + h * 64, at, 0);
+        bulk_load(st + L::OFF_SC, sc + (long long)c * p.H * SCALARS, SCALARS * 4, bar);
+    };
+    if (warp == 0) {
+        if (tc::elect_one()) {
+            tc::mbar_init(full, 1);
+            tc::mbar_init(full + 1, 1);
+            tc::mbar_init(ready, SCAN_WARPS);
+            tc::mbar_init(done, 1);
+            *abort_flag = 0;
+            tc::fence_barrier_init();
+            load(0);
+            if (chunks > 1) load(1);
+        }
+        __syncwarp();
+        tc::tmem_alloc(tmem_slot, 256);
+        tc::tmem_relinquish();
     }
-    __syncwarp();
     int slot = p.slots[b];
     if (slot >= p.num_states) {
         if (tid == 0) atomicMax(p.status, (int)KB_BAD_INDEX);
         slot = -1;
     }
     const bool fresh = slot < 0 || p.ctx[b] <= n;
-    if (warp == 0) {
-        tc::tmem_alloc(tmem_slot, 256);
-        tc::tmem_relinquish();
-    }
     tc::tc_fence_before();
     __syncthreads();
     tc::tc_fence_after();
-    const uint32_t tmem0 = __shfl_sync(0xffffffffu, *tmem_slot, 0), tmem = tmem0 + ((uint32_t)((warp & 3) * 32) << 16) + hf * 32;
-    // this thread's half of row `row` of the state
-    const int col0 = tile * 64 + hf * 32;
+    // columns 0 .. 127 results; 128 .. 255 the state's two halves as an operand, which R's and U's lie over
+    const uint32_t tmem = __shfl_sync(0xffffffffu, *tmem_slot, 0);
+    const uint32_t op_hi = tmem + 128, s_lo = op_hi + D / 2, ru_lo = op_hi + 32;
+    bool ok = true;
+    const int lane = tid & 31, dvi = (warp & 3) * 32 + lane, g = warp >> 2, col = tile * 128 + dvi;
+    const bool owns = g * 32 < D;
+    const uint32_t lanes = (uint32_t)((warp & 3) * 32) << 16;
+    const uint32_t res_k = tmem + lanes + g * 16, res_q = res_k + CH, res_s = tmem + lanes + g * 32;
+    const uint32_t s_hi_w = op_hi + lanes + g * 16, s_lo_w = s_lo + lanes + g * 16, ru_hi_w = op_hi + lanes + g * 8, ru_lo_w = ru_lo + lanes + g * 8;
+    const uint32_t id1 = tc::instr_desc_f16(128, 128, 1, 1, 0, 0), id3 = tc::instr_desc_f16(128, D, 1, 1, 0, 1);
+    uint8_t* sO = smem + L::OFF_O;                     // [2][64 tokens][64 columns]
+    uint16_t* o_out = reinterpret_cast<uint16_t*>(sO + (dvi >> 6) * BLK) + g * 16 * 64 + (dvi & 63);
+    // S^T: this thread holds value column `col`, rows g * 32 .. of the state
     float S[32];
-    float* st = p.state + (((long long)(slot < 0 ? 0 : slot) * p.H + head) * p.d + row) * p.dvp + col0;
-    const bool own = row < p.d;
+    float* st = p.state + ((long long)(slot < 0 ? 0 : slot) * p.H + head) * p.d * p.dvp + col;
 #pragma unroll
-    for (int c = 0; c < 32; c += 4) {
-        float4 f = make_float4(0.f, 0.f, 0.f, 0.f);
-        if (own && !fresh && col0 + c < p.dvp) f = *reinterpret_cast<const float4*>(st + c);
-        S[c] = f.x; S[c + 1] = f.y; S[c + 2] = f.z; S[c + 3] = f.w;
+    for (int j = 0; j < 32; ++j) {
+        const int i = g * 32 + j;
+        S[j] = !fresh && i < p.d && col < p.dvp ? st[(long long)i * p.dvp] : 0.f;
     }
-    if (row < D) store_row_split<4>(sS, sS + L::S_HALF, row, hf * 4, S);
-    const int i = row & 63;
-    const long long vstride = (long long)p.H * p.dvt;
-    const bf16* vsrc = p.v + (long long)(row0 + i) * vstride + head * p.dvt + col0;
-    bf16* odst = p.o + (long long)(row0 + i) * vstride + head * p.dvt + col0;
-    const uint32_t aKQ = smem_u32(sKQ), aTT = smem_u32(sTT), aS = smem_u32(sS), aRU = smem_u32(sRU);
-    const uint32_t id_k = tc::instr_desc_f16(128, 64, 1, 1, 0, 1), id_m = tc::instr_desc_f16(128, 64, 1, 1, 1, 1);
-    // values and scalars of a chunk, fetched while the chunk in front of it is worked on
-    uint4 v[4];
-    float e, eu, decay;
-    auto fetch = [&](int c) {
-        const float* s = sc + (long long)c * p.H * SCALARS;
-        e = s[row];
-        eu = s[2 * CH + i];
-        decay = s[3 * CH];
-        if (is_k) {
-            const uint4* src = reinterpret_cast<const uint4*>(vsrc + (long long)c * CH * vstride);
-#pragma unroll
-            for (int j = 0; j < 4; ++j) v[j] = c * CH + i < n ? src[j] : make_uint4(0u, 0u, 0u, 0u);
-        }
+    uint32_t par_ready = 0, par_done = 0;
+    auto hand_over = [&]() {                           // what this warp wrote to tensor memory may be multiplied
+        tc::tmem_st_wait();
+        tc::tc_fence_before();
+        __syncwarp();
+        if (lane == 0) tc::mbar_arrive(ready);
     };
-    fetch(0);
-    uint32_t done = 0;                                 // parity of the product barrier
-    bool failed = false;
+    auto operand = [&]() {                             // warp 0: every warp has handed over
+        ok = tc::mbar_wait(ready, par_ready, abort_flag) && ok;
+        par_ready ^= 1;
+        tc::tc_fence_after();
+    };
+    auto issuer = [&]() -> bool {                      // one lane issues; the operands stay in uniform registers
+        return __all_sync(0xffffffffu, ok) && tc::elect_one();
+    };
+    auto result = [&]() {
+        __syncwarp();
+        ok = tc::mbar_wait(done, par_done, abort_flag) && ok;
+        par_done ^= 1;
+        tc::tc_fence_after();
+    };
+    auto store_o = [&](int c) {                        // one thread: the chunk's rows of O (all 64 of them) leave shared memory
+        for (int h = 0; h < boxes; ++h)
+            asm volatile("cp.async.bulk.tensor.3d.global.shared::cta.tile.bulk_group [%0, {%2, %3, %4}], [%1];" ::"l"(reinterpret_cast<uint64_t>(&tmO)),
+                         "r"(smem_u32(sO + h * BLK)), "r"(head * p.dvt + tile * 128 + h * 64), "r"(row0 + c * CH), "r"(0)
+                         : "memory");
+        asm volatile("cp.async.bulk.commit_group;" ::: "memory");
+    };
+    if (owns) tmem_store_split<16>(s_hi_w, s_lo_w, S);
+    hand_over();
     for (int c = 0; c < chunks; ++c) {
-        tc::fence_proxy_async();
-        tc::tc_fence_before();
-        if (__syncthreads_or(failed)) { failed = true; break; }
-        // products are issued by one elected lane of a whole warp: their operands then stay in uniform registers
-        if (warp == 0) {                               // X = [K; Q] S
-            failed |= !tc::mbar_wait(bars, c & 1, abort_flag);
-            tc::tc_fence_after();
-            if (!__any_sync(0xffffffffu, failed) && tc::elect_one()) {
-                mma_steps<D / 16, 32, 2048, true>(tmem0, aKQ, 16, aS, 16, id_k, false);
-                mma_steps<D / 16, 32, 2048, true>(tmem0, aKQ, 16, aS + L::S_HALF, 16, id_k, true);
-                tc::tc_commit(bars + 2);
+        const uint8_t* sm = smem + (c & 1) * L::STAGE;
+        const uint32_t aKQ = smem_u32(smem) + (c & 1) * L::STAGE, aTT = aKQ + L::OFF_TT;
+        const float* scal = reinterpret_cast<const float*>(sm + L::OFF_SC);
+        ok = tc::mbar_wait(full + (c & 1), (c >> 1) & 1, abort_flag) && ok;
+        float x[16], y[16];
+        uint32_t v[8];                                 // V, transposed on the way: one number per token, two of them per register
+        {
+            const uint16_t* src = reinterpret_cast<const uint16_t*>(sm + L::OFF_V + (dvi >> 6) * BLK) + g * 16 * 64 + (dvi & 63);
+#pragma unroll
+            for (int j = 0; j < 8; ++j) v[j] = (uint32_t)src[2 * j * 64] | (uint32_t)src[(2 * j + 1) * 64] << 16;
+        }
+        if (warp == 0) {                               // X^T
+            operand();
+            if (issuer()) {
+                mma_ts_steps<D / 16, 32, true>(tmem, op_hi, aKQ, 16, id1, false);
+                mma_ts_steps<D / 16, 32, true>(tmem, s_lo, aKQ, 16, id1, true);
+                tc::tc_commit(done);
+            }
+            __syncwarp();
+            if (lane == 0 && c > 0 && ok) store_o(c - 1);
+        }
+        result();
+        tc::tmem_ld16(res_k, reinterpret_cast<uint32_t*>(x));
+        tc::tmem_ld16(res_q, reinterpret_cast<uint32_t*>(y));
+        tc::tmem_ld_wait();
+#pragma unroll
+        for (int j = 0; j < 16; j += 4) {              // R = V - e^G r_k X
+            const float4 f = *reinterpret_cast<const float4*>(scal + g * 16 + j);
+            x[j] = fmaf(-f.x, x[j], __uint_as_float(v[j / 2] << 16));
+            x[j + 1] = fmaf(-f.y, x[j + 1], __uint_as_float(v[j / 2] & 0xffff0000u));
+            x[j + 2] = fmaf(-f.z, x[j + 2], __uint_as_float(v[j / 2 + 1] << 16));
+            x[j + 3] = fmaf(-f.w, x[j + 3], __uint_as_float(v[j / 2 + 1] & 0xffff0000u));
+        }
+        tmem_store_split<8>(ru_hi_w, ru_lo_w, x);
+        hand_over();
+        if (warp == 0) {                               // [U; A U]^T
+            operand();
+            if (lane == 0) asm volatile("cp.async.bulk.wait_group.read 0;" ::: "memory");     // O's buffer is free when this product is done
+            __syncwarp();
+            if (issuer()) {
+                mma_ts_steps<4, 32>(tmem, op_hi, aTT, 16, id1, false);
+                mma_ts_steps<4, 32>(tmem, ru_lo, aTT, 16, id1, true);
+                mma_ts_steps<4, 32>(tmem, op_hi, aTT + 2 * BLK, 16, id1, true);
+                tc::tc_commit(done);
+            }
+        } else if (warp == SCAN_WARPS - 1) {           // the chunk before this one is done with its stage
+            if (lane == 0 && c > 0 && c + 1 < chunks && ok) load(c + 1);
+        }
+        scale16(y, scal + CH + g * 16);                // e^G r_q X
+        result();
+        tc::tmem_ld16(res_k, reinterpret_cast<uint32_t*>(x));
+        float z[16];
+        tc::tmem_ld16(res_q, reinterpret_cast<uint32_t*>(z));
+        tc::tmem_ld_wait();
+        scale16(x, scal + 2 * CH + g * 16);            // e^(G_64 - G) r_k U
+        tmem_store_split<8>(ru_hi_w, ru_lo_w, x);
+        hand_over();
+        if (warp == 0) {                               // U^T K
+            operand();
+            if (issuer()) {
+                mma_ts_steps<4, 2048>(tmem, op_hi, aKQ, 2 * BLK, id3, false);
+                mma_ts_steps<4, 2048>(tmem, ru_lo, aKQ, 2 * BLK, id3, true);
+                tc::tc_commit(done);
             }
             __syncwarp();
         }
-        failed |= !tc::mbar_wait(bars + 2, done, abort_flag);
-        done ^= 1;
-        tc::tc_fence_after();
-        float x[32];
-        tmem_row32(tmem, x);
-        if (is_k) {                                    // R = V - e^G r_k X
+        // O = e^G r_q X + A U, while the product runs
+        const int valid = n - c * CH;
+        if (valid >= CH) {
 #pragma unroll
-            for (int j = 0; j < 4; ++j) {
-                float f[8];
-                unpack8(*reinterpret_cast<const bf16x8*>(&v[j]), f);
+            for (int j = 0; j < 16; ++j) o_out[j * 64] = __bfloat16_as_ushort(__float2bfloat16(y[j] + z[j]));
+            tc::fence_proxy_async();
+        } else if (col < p.dvt) {                      // the rows behind the sequence's end are another's
+            bf16* dst = p.o + (long long)(row0 + c * CH) * p.H * p.dvt + head * p.dvt + col;
 #pragma unroll
-                for (int q = 0; q < 8; ++q) x[j * 8 + q] = fmaf(-e, x[j * 8 + q], f[q]);
+            for (int j = 0; j < 16; ++j)
+                if (g * 16 + j < valid) dst[(long long)(g * 16 + j) * p.H * p.dvt] = __float2bfloat16(y[j] + z[j]);
+        }
+        const float decay = scal[3 * CH];
+        result();
+        if (owns) {
+            tc::tmem_ld16(res_s, reinterpret_cast<uint32_t*>(x));
+            tc::tmem_ld16(res_s + 16, reinterpret_cast<uint32_t*>(y));
+            tc::tmem_ld_wait();
+#pragma unroll
+            for (int j = 0; j < 16; ++j) {
+                S[j] = fmaf(decay, S[j], x[j]);
+                S[16 + j] = fmaf(decay, S[16 + j], y[j]);
             }
-            store_row_split<4>(sRU, sRU + BLK, i, hf * 4, x);
-        } else {
-#pragma unroll
-            for (int j = 0; j < 32; ++j) x[j] *= e;
+            tmem_store_split<16>(s_hi_w, s_lo_w, S);
         }
-        tc::fence_proxy_async();
-        tc::tc_fence_before();
-        if (__syncthreads_or(failed)) { failed = true; break; }
-        if (warp == 0) {                               // [U; A U] = [T; A T] R
-            failed |= !tc::mbar_wait(bars + 1, c & 1, abort_flag);
-            tc::tc_fence_after();
-            if (!__any_sync(0xffffffffu, failed) && tc::elect_one()) {
-                mma_steps<4, 32, 2048>(tmem0 + 64, aTT, 16, aRU, 16, id_k, false);
-                mma_steps<4, 32, 2048>(tmem0 + 64, aTT, 16, aRU + BLK, 16, id_k, true);
-                mma_steps<4, 32, 2048>(tmem0 + 64, aTT + 2 * BLK, 16, aRU, 16, id_k, true);
-                tc::tc_commit(bars + 2);
-            }
-            __syncwarp();
-        }
-        const float scale_u = eu, scale_s = decay;
-        if (c + 1 < chunks) fetch(c + 1);
-        failed |= !tc::mbar_wait(bars + 2, done, abort_flag);
-        done ^= 1;
-        tc::tc_fence_after();
-        if (tid == 0 && c + 1 < chunks && !failed) {
-            tc::mbar_expect_tx(bars + 1, TT_BYTES);
-            bulk_load(sTT, tt + (long long)(c + 1) * p.H * TT_BYTES, TT_BYTES, bars + 1);
-        }
-        __syncwarp();
-        float y[32];
-        tmem_row32(tmem + 64, y);
-        if (is_k) {                                    // e^(G_64 - G) r_k U
-#pragma unroll
-            for (int j = 0; j < 32; ++j) y[j] *= scale_u;
-            store_row_split<4>(sRU, sRU + BLK, i, hf * 4, y);
-        }
-        tc::fence_proxy_async();
-        tc::tc_fence_before();
-        if (__syncthreads_or(failed)) { failed = true; break; }
-        if (warp == 0) {                               // K^T U
-            tc::tc_fence_after();
-            if (tc::elect_one()) {
-                mma_steps<4, 2048, 2048>(tmem0 + 128, aKQ, 2 * BLK, aRU, 16, id_m, false);
-                mma_steps<4, 2048, 2048>(tmem0 + 128, aKQ, 2 * BLK, aRU + BLK, 16, id_m, true);
-                tc::tc_commit(bars + 2);
-            }
-            __syncwarp();
-        }
-        if (!is_k && c * CH + i < n) {                 // O, while the product runs
-            bf16* dst = odst + (long long)c * CH * vstride;
-#pragma unroll
-            for (int j = 0; j < 32; j += 8) {
-#pragma unroll
-                for (int q = 0; q < 8; ++q) x[j + q] += y[j + q];
-                store8(dst + j, x + j);
-            }
-        }
-        __syncwarp();
-        failed |= !tc::mbar_wait(bars + 2, done, abort_flag);
-        done ^= 1;
-        tc::tc_fence_after();
-        if (tid == 0 && c + 1 < chunks && !failed) load_kq<D>(sKQ, &tmK, &tmQ, bars, kvh, row0 + (c + 1) * CH);
-        __syncwarp();
-        tmem_row32(tmem + 128, x);
-        if (row < D) {
-#pragma unroll
-            for (int j = 0; j < 32; ++j) S[j] = fmaf(scale_s, S[j], x[j]);
-            store_row_split<4>(sS, sS + L::S_HALF, row, hf * 4, S);
-        }
+        hand_over();
+        if (!__all_sync(0xffffffffu, ok)) break;
     }
-    if (failed) {
+    if (warp == 0 && __all_sync(0xffffffffu, ok)) {    // the last arrivals, before the block ends
+        operand();
+        if (lane == 0 && ok) {
+            if (n % CH == 0) store_o(chunks - 1);
+            asm volatile("cp.async.bulk.wait_group 0;" ::: "memory");
+        }
+        __syncwarp();
+    }
+    if (ok && slot >= 0 && col < p.dvp) {
+#pragma unroll
+        for (int j = 0; j < 32; ++j)
+            if (g * 32 + j < p.d) st[(long long)(g * 32 + j) * p.dvp] = S[j];
+    }
+    if (!ok) {
         atomicMax(p.status, (int)KB_TIMEOUT_MMA);
         const uint64_t t0 = global_timer_ns();         // copies in flight land before the block's memory is given up
         while (global_timer_ns() - t0 < 2000000ull) {}
-    } else if (own && slot >= 0) {
-#pragma unroll
-        for (int c = 0; c < 32; c += 4)
-            if (col0 + c < p.dvp) *reinterpret_cast<float4*>(st + c) = make_float4(S[c], S[c + 1], S[c + 2], S[c + 3]);
     }
+    __syncwarp();
     tc::tc_fence_before();
     __syncthreads();
     if (warp == 0) {
         tc::tc_fence_after();
-        tc::tmem_dealloc(tmem0, 256);
+        tc::tmem_dealloc(tmem, 256);
     }
 }
 
@@ -764,15 +845,15 @@ delta_finish_kernel(const bf16* __restrict__ o, int dvt, const bf16* __restrict_
     }
 }
 
-// [rows, cols] bf16, box 64 columns x 64 rows, 128-byte swizzle
-int rows_tmap(CUtensorMap* m, const void* base, long long rows, long long cols) {
+// [rows, cols] bf16, box 64 columns x 64 rows
+int rows_tmap(CUtensorMap* m, const void* base, long long rows, long long cols, CUtensorMapSwizzle swizzle) {
     attn::EncodeTiledFn enc = attn::get_encode();
     if (!enc) return 100;
     cuuint64_t dims[3] = {(cuuint64_t)cols, (cuuint64_t)rows, 1};
     cuuint64_t strides[2] = {(cuuint64_t)cols * 2, (cuuint64_t)rows * cols * 2};
     cuuint32_t box[3] = {64, CH, 1}, estr[3] = {1, 1, 1};
     const CUresult r = enc(m, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 3, const_cast<void*>(base), dims, strides, box, estr, CU_TENSOR_MAP_INTERLEAVE_NONE,
-                           CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
+                           swizzle, CU_TENSOR_MAP_L2_PROMOTION_L2_256B, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
     return r == CUDA_SUCCESS ? 0 : 200 + (int)r;
 }
 template <typename K>
@@ -790,12 +871,14 @@ int launch_chunks(const ChunkParams& p, const bf16* q, const bf16* k, cudaStream
     static bool f1[64] = {}, f2[64] = {};
     int r = allow_smem(delta_prepare_kernel<D>, PREP_SMEM, f1);
     if (!r) r = allow_smem(delta_scan_kernel<D>, Scan<D>::SMEM, f2);
-    CUtensorMap tmK, tmQ;
-    if (!r) r = rows_tmap(&tmK, k, p.N, (long long)p.G * D);
-    if (!r) r = rows_tmap(&tmQ, q, p.N, (long long)p.G * D);
+    CUtensorMap tmK, tmQ, tmV, tmO;
+    if (!r) r = rows_tmap(&tmK, k, p.N, (long long)p.G * D, CU_TENSOR_MAP_SWIZZLE_128B);
+    if (!r) r = rows_tmap(&tmQ, q, p.N, (long long)p.G * D, CU_TENSOR_MAP_SWIZZLE_128B);
+    if (!r) r = rows_tmap(&tmV, p.v, p.N, (long long)p.H * p.dvt, CU_TENSOR_MAP_SWIZZLE_NONE);
+    if (!r) r = rows_tmap(&tmO, p.o, p.N, (long long)p.H * p.dvt, CU_TENSOR_MAP_SWIZZLE_NONE);
     if (r) return r;
     delta_prepare_kernel<D><<<dim3(p.N / CH + p.B, p.H), 128, PREP_SMEM, st>>>(tmK, tmQ, p);
-    delta_scan_kernel<D><<<dim3(p.dvt / 64, p.H, p.B), 256, Scan<D>::SMEM, st>>>(tmK, tmQ, p);
+    delta_scan_kernel<D><<<dim3((p.dvt + 127) / 128, p.H, p.B), SCAN_WARPS * 32, Scan<D>::SMEM, st>>>(tmK, tmQ, tmV, tmO, p);
     return kb_launch_status();
 }
 
