@@ -213,26 +213,28 @@ def run_serve(args, rank, world, local):
     return serve_bench.run(a, rank, world, local)
 
 
-def run_vunitar(args) -> dict:
-    """Prefill and decode throughput of the Vunitar design at sizes that resemble a real model's layers, beside the Llama
-    family at equal width, heads and active parameters, and the kernels of both against their rooflines."""
+def run_design(args) -> dict:
+    """Prefill and decode throughput of one of the model designs at sizes that resemble a real model's layers, beside the
+    Llama family at equal size, and the kernels of both against their rooflines."""
+    import importlib
     sys.path.insert(0, os.path.join(ROOT, "benchmarks"))
-    import vunitar_bench
+    name = args.mode
+    bench = importlib.import_module(f"{name}_bench")
     sampler = ClockSampler(0)
     sampler.start()
-    res = vunitar_bench.run(args.sizes.split(",") if args.sizes else list(vunitar_bench.SIZES))
+    res = bench.run(args.sizes.split(",") if args.sizes else list(bench.SIZES))
     clocks = sampler.stop()
     e = res["engines"][0]
-    return {"metric": "vunitar_decode_tokens_per_sec", "value": e["vunitar"]["decode_tok_s"], "unit": "tokens/s", "n_gpus": 1,
-            "steps": e["new_tokens"], "warmup": 1, "ms_per_step": e["vunitar"]["decode_step_ms"], "higher_is_better": True,
+    return {"metric": f"{name}_decode_tokens_per_sec", "value": e[name]["decode_tok_s"], "unit": "tokens/s", "n_gpus": 1,
+            "steps": e["new_tokens"], "warmup": 1, "ms_per_step": e[name]["decode_step_ms"], "higher_is_better": True,
             "scaling": "weak", "vs_baseline": None, "dtype": "bf16",
             "data": "synthetic uniform-random prompts, random-init weights",
-            "config": {"model": f"Vunitar {e['size']}", "requests": e["requests"], "prompt_tokens": e["prompt_tokens"],
+            "config": {"model": f"{name.capitalize()} {e['size']}", "requests": e["requests"], "prompt_tokens": e["prompt_tokens"],
                        "new_tokens": e["new_tokens"], "parallelism": "1 GPU",
                        "timing": "engine: wall clock with a device synchronize around every step; kernels: CUDA events over graph "
                                  "replays on buffers larger than L2"},
-            "clocks": clocks, "gpu_launches": e["vunitar"]["launches"],
-            "e2e": {"value": e["vunitar"]["decode_tok_s"], "unit": "tokens/s", "h2d_bytes_per_step": e["requests"] * 28,
+            "clocks": clocks, "gpu_launches": e[name]["launches"],
+            "e2e": {"value": e[name]["decode_tok_s"], "unit": "tokens/s", "h2d_bytes_per_step": e["requests"] * 28,
                     "d2h_bytes_per_step": e["requests"] * 8},
             "impl": "native", "engines": res["engines"], "kernels": res["kernels"], "peaks": res["peaks"]}
 
@@ -266,11 +268,11 @@ def main() -> None:
     ap.add_argument("--attn-res-blocks", type=int, default=7)
     ap.add_argument("--backend", default="auto", choices=["auto", "native", "nccl"])
     ap.add_argument("--op-times", default="", help="write a per-op device-time table to this file")
-    ap.add_argument("--mode", default="dp", choices=["dp", "tp", "serve", "vunitar"],
+    ap.add_argument("--mode", default="dp", choices=["dp", "tp", "serve", "vunitar", "lisunex"],
                     help="dp: data parallel (the headline); tp: tensor + sequence parallel over all ranks, one global "
-                         "batch of --micro-batch sequences; serve: 64-request paged-KV serving; vunitar: "
-                         "prefill, decode and kernels of the Vunitar design beside the Llama family at equal size (1 GPU)")
-    ap.add_argument("--sizes", default="", help="--mode vunitar: comma-separated sizes of benchmarks/vunitar_bench.py (default: all)")
+                         "batch of --micro-batch sequences; serve: 64-request paged-KV serving; vunitar, lisunex: "
+                         "prefill, decode and kernels of that design beside the Llama family at equal size (1 GPU)")
+    ap.add_argument("--sizes", default="", help="--mode vunitar / lisunex: comma-separated sizes of benchmarks/<mode>_bench.py (default: all)")
     ap.add_argument("--fp8", action="store_true", help="block-scaled e4m3 projections (bf16 masters)")
     args = ap.parse_args()
     args.warmup = max(args.warmup, 3)
@@ -284,9 +286,9 @@ def main() -> None:
         os.environ["KOTODAMA_GEMM"] = "cublas"
         args.backend = "nccl"
     rank, world, local = dist_setup(args.gpus)
-    if args.mode == "vunitar":
+    if args.mode in ("vunitar", "lisunex"):
         if rank == 0:
-            print(json.dumps(run_vunitar(args)))
+            print(json.dumps(run_design(args)))
         if world > 1:
             dist.barrier()
             dist.destroy_process_group()

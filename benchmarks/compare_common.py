@@ -47,6 +47,24 @@ def timed(calls: list, reps: int = 5) -> float:
     return e0.elapsed_time(e1) / (reps * len(calls))
 
 
+def kernel_ms(calls: list, names: list[str]) -> dict[str, float]:
+    """Mean device time in ms of the kernels whose name contains each of ``names``, over the calls (profiler records; for
+    operations of several launches)."""
+    from torch.profiler import ProfilerActivity, profile
+    for c in calls:
+        c()
+    torch.cuda.synchronize()
+    with profile(activities=[ProfilerActivity.CUDA]) as prof:
+        for c in calls:
+            c()
+        torch.cuda.synchronize()
+    out = {}
+    for n in names:
+        rows = [e for e in prof.key_averages() if n in e.key]
+        out[n] = sum(e.self_device_time_total for e in rows) / max(1, sum(e.count for e in rows)) * 1e-3
+    return out
+
+
 def engine_arm(model, requests: int, prompt: int, new: int) -> dict:
     """Prefill of `requests` prompts of `prompt` tokens each, then `new` greedy tokens for all of them."""
     cfg = model.config

@@ -21,7 +21,7 @@ import torch
 ROOT = os.path.dirname(os.path.dirname(os.path.abspath(__file__)))
 sys.path.insert(0, ROOT)
 sys.path.insert(0, os.path.join(ROOT, "benchmarks"))
-from compare_common import engine_arm, peaks, timed  # noqa: E402
+from compare_common import engine_arm, kernel_ms, peaks, timed  # noqa: E402
 from kotodama_b200.config import ModelConfig  # noqa: E402
 from kotodama_b200.models.lisunex import LisunexConfig, LisunexModel  # noqa: E402
 from kotodama_b200.models.llama import KotodamaModel  # noqa: E402
@@ -97,11 +97,18 @@ def kernels(name: str, z: dict, batch: int = 64, ctx: int = 1280, tokens: int = 
     add("delta rule, one token", "decode attention", ms, B * (DH * 128 * 128 * 8 + DH * 384 * (2 * TAPS - 2) * 2 + W * 2 + DH * 256))
     n = tokens
     cu, ctxs = i32([0] + [(i + 1) * 1024 for i in range(n // 1024)]), i32([1024] * (n // 1024))
-    rows = [bf(n, W) for _ in range(2)]
+    rows = [bf(n, W) for _ in range(3)]
     # products of the chunked form, every operand counted once
     fl = n * DH * (2.0 * 128 * 64 * 128 + 2.0 * 128 * 128 * 128 + 2.0 * 128 * 64 * 128 * 2 + 2.0 * 64 ** 3) / 64
-    ms = timed([lambda r=r: ops.delta_rule(r, DH, DG, 128, 128, conv, al, dt, nw, 1e-5, st[0], rg[0], slots[: n // 1024], cu, ctxs, 1024) for r in rows])
-    add("delta rule, prompts of 1024 (conv, prepare, scan, finish)", "attention", ms, n * (W + DH * 128) * 2 + n // 1024 * DH * 128 * 128 * 4, fl)
+    calls = [lambda r=r: ops.delta_rule(r, DH, DG, 128, 128, conv, al, dt, nw, 1e-5, st[0], rg[0], slots[: n // 1024], cu, ctxs, 1024) for r in rows]
+    add("delta rule, prompts of 1024 (all launches)", "attention", timed(calls), n * (W + DH * 128) * 2 + n // 1024 * DH * 128 * 128 * 4, fl)
+    # its launches one by one, each against the bytes and products of its own inputs and outputs
+    part = kernel_ms(calls * 3, ["delta_conv", "delta_prepare", "delta_scan", "delta_finish"])
+    qk, vo, tt = n * 2 * DG * 256, n * DH * 256, n // 64 * DH * 32768
+    add("  delta conv + SiLU", "row kernel", part["delta_conv"], 2 * (qk + vo))
+    add("  delta prepare (triangular inverses)", "attention", part["delta_prepare"], qk + tt, n // 64 * DH * (2.0 * 128 * 64 * 128 + 2.0 * 64 ** 3))
+    add("  delta scan", "attention", part["delta_scan"], qk + 2 * vo + tt, n // 64 * DH * (2.0 * 128 * 128 * 128 + 2 * 2.0 * 128 * 64 * 128))
+    add("  delta output norm + gate", "row kernel", part["delta_finish"], 3 * vo)
     del st, rg
     # ---- decode products and row kernels
     a = bf(B, D)
