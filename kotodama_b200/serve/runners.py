@@ -131,6 +131,15 @@ def _up(n: int, a: int) -> int:
     return (n + a - 1) // a * a
 
 
+def _pad(t: torch.Tensor, *shape: int) -> torch.Tensor:
+    """Zeros behind ``t`` in every dimension, up to ``shape``."""
+    if tuple(t.shape) == shape:
+        return t
+    out = torch.zeros(shape, dtype=t.dtype, device=t.device)
+    out[tuple(slice(0, n) for n in t.shape)] = t
+    return out
+
+
 class LatentRunner:
     """Latent-attention decoder with dense / mixture-of-experts feed-forwards and output norms
     (``models/vunitar.py``).
@@ -161,8 +170,8 @@ class LatentRunner:
         self.short_portion = 16                 # most tokens per sequence for the latent form of the attention
         w = model.weights
         put = lambda t: t.to(self.device, self.dtype).contiguous()
-        vec = lambda t, n: self._pad(t.to(self.device, torch.float32), n)
-        lin = lambda t, n, k: self._pad(put(t), n, k)
+        vec = lambda t, n: _pad(t.to(self.device, torch.float32), n)
+        lin = lambda t, n, k: _pad(put(t), n, k)
         dw = self.ops.decode_weight
         Dp = self.Dp
         self.embed = lin(w["embed"], cfg.vocab_size, Dp)
@@ -177,11 +186,11 @@ class LatentRunner:
                 dp, dv = _up(m.dim, 8), _up(m.vdim, 8)
             R = _up(m.kv_rank, self.ops.latent_multiple(self.dtype))
             H = m.heads
-            uk = self._pad(put(w[p + "mix.uk"]).view(H, m.dim, m.kv_rank), H, dp, R)
-            uv = self._pad(put(w[p + "mix.uv"]).view(H, m.vdim, m.kv_rank), H, dv, R)
+            uk = _pad(put(w[p + "mix.uk"]).view(H, m.dim, m.kv_rank), H, dp, R)
+            uv = _pad(put(w[p + "mix.uv"]).view(H, m.vdim, m.kv_rank), H, dv, R)
             ukv = torch.cat([uk.reshape(H * dp, R), uv.reshape(H * dv, R)])
-            q = self._pad(put(w[p + "mix.q"]).view(H, m.dim, self.D), H, dp, Dp).reshape(H * dp, Dp)
-            o = self._pad(put(w[p + "mix.o"]).view(self.D, H, m.vdim), Dp, H, dv).reshape(Dp, H * dv)
+            q = _pad(put(w[p + "mix.q"]).view(H, m.dim, self.D), H, dp, Dp).reshape(H * dp, Dp)
+            o = _pad(put(w[p + "mix.o"]).view(self.D, H, m.vdim), Dp, H, dv).reshape(Dp, H * dv)
             lw: dict[str, Any] = dict(
                 H=H, dp=dp, dv=dv, R=R, rank=m.kv_rank, scale=m.scale, flash=fits,
                 wqc=dw(torch.cat([q, lin(w[p + "mix.dkv"], R, Dp)])), cnorm=vec(w[p + "mix.dkv.norm"], R),
@@ -209,14 +218,6 @@ class LatentRunner:
         self.head = lin(w["head"], cfg.vocab_size, Dp)
         self.cache: Any = None
         self.layer_trace: Optional[list] = None      # when a list: the residual stream after every layer is appended
-
-    @staticmethod
-    def _pad(t: torch.Tensor, *shape: int) -> torch.Tensor:
-        if tuple(t.shape) == shape:
-            return t
-        out = torch.zeros(shape, dtype=t.dtype, device=t.device)
-        out[tuple(slice(0, n) for n in t.shape)] = t
-        return out
 
     def first_visible(self, n: int) -> int:
         return 0
@@ -299,15 +300,14 @@ class HybridRunner:
         cfg = self.cfg = model.config
         self.D, self.short_portion = cfg.hidden_size, 16
         Dp = self.Dp = _up(self.D, 8)
-        pad = LatentRunner._pad
         w = model.weights
         f32 = lambda t: t.to(self.device, torch.float32).contiguous()
         put = lambda t: t.to(self.device, self.dtype)
-        vec = lambda t: pad(f32(t), Dp)
+        vec = lambda t: _pad(f32(t), Dp)
         dw = self.ops.decode_weight
         # one product for everything that reads the layer's input: the parts start at multiples of eight rows
-        fuse = lambda parts: torch.cat([pad(put(t), _up(t.shape[0], 8), Dp) for t in parts])
-        self.embed = pad(put(w["embed"]), cfg.vocab_size, Dp)
+        fuse = lambda parts: torch.cat([_pad(put(t), _up(t.shape[0], 8), Dp) for t in parts])
+        self.embed = _pad(put(w["embed"]), cfg.vocab_size, Dp)
         self.steps = [vec(t) for t in w["loop.step"]] if cfg.loop else []
         tables: dict[Any, tuple[torch.Tensor, torch.Tensor]] = {}
         self.layers: list[dict[str, Any]] = []
@@ -321,23 +321,23 @@ class HybridRunner:
                 if m.rot not in tables:
                     tables[m.rot] = tuple(t.to(self.device).contiguous() for t in m.rot.table(self.max_ctx))
                 lw["win"] = dw(fuse([x("q"), x("k"), x("v"), x("g")]))
-                lw["bias"] = torch.cat([pad(put(b), _up(b.shape[0], 8)) for b in (x("q.b"), x("k.b"), x("v.b"), torch.zeros(m.heads))])
+                lw["bias"] = torch.cat([_pad(put(b), _up(b.shape[0], 8)) for b in (x("q.b"), x("k.b"), x("v.b"), torch.zeros(m.heads))])
                 lw["cs"] = tables[m.rot]
                 lw["gate"] = _up(m.heads * m.dim, 8) + _up(m.kv_heads * m.dim, 8) + _up(m.kv_heads * m.vdim, 8)
-                o = pad(put(x("o")).view(self.D, m.heads, m.vdim), Dp, m.heads, lw["cols"])
+                o = _pad(put(x("o")).view(self.D, m.heads, m.vdim), Dp, m.heads, lw["cols"])
                 lw["wo"] = dw(o.reshape(Dp, m.heads * lw["cols"]))
             else:
                 lw["win"] = dw(fuse([x("q"), x("k"), x("v"), x("g"), x("b"), x("a")]))
                 lw["conv"] = torch.cat([f32(x(n + ".conv")) for n in "qkv"]).t().contiguous()
                 lw.update(a_log=f32(x("A_log")), dt=f32(x("dt_bias")), norm=f32(x("norm")))
-                lw["wo"] = dw(pad(put(x("o")), Dp, _up(m.heads * m.vdim, 8)))
+                lw["wo"] = dw(_pad(put(x("o")), Dp, _up(m.heads * m.vdim, 8)))
             if layer.mlp is not None:
                 fp = _up(layer.mlp.ff, 8)
                 lw.update(norm2=vec(w[p + "norm2"]), wgu=dw(fuse([w[p + "mlp.gate"], w[p + "mlp.up"]])),
-                          wd=dw(pad(put(w[p + "mlp.down"]), Dp, fp)))
+                          wd=dw(_pad(put(w[p + "mlp.down"]), Dp, fp)))
             self.layers.append(lw)
         self.final = vec(w["final.norm"])
-        self.head = pad(put(w["head"]), cfg.vocab_size, Dp)
+        self.head = _pad(put(w["head"]), cfg.vocab_size, Dp)
         self.runs = cfg.runs()
         self.chunks = {lw["m"].chunk for lw in self.layers if not lw["delta"]}
         self.context_buckets = 0 in self.chunks
